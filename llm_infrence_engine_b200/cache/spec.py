@@ -22,6 +22,7 @@ class FixedStateSpec:
     """A per-request tensor of fixed shape that a mixer reads and writes in place (32-bit floats)."""
 
     shape: Tuple[int, ...]
+    zeroed: bool = True   # starts from zero at a request's first token; False: whoever owns it never reads it there
 
 
 def flatten_specs(spec) -> tuple:

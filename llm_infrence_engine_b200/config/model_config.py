@@ -866,3 +866,132 @@ class MemilornConfig:
         for t in range(self.loop_times):
             order += [(i, t, t > 0 and i == self.loop_start) for i in range(self.loop_start, self.loop_stop)]
         return order + [(i, 0, False) for i in range(self.loop_stop, len(self.layers))]
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Sinorax: a decoder whose config.json lists its layers one by one; every sublayer lies between two Dynamic Tanhs. Mixers: grouped
+# softmax attention whose values turn with their positions, windowed attention with sigmoid weights and a penalty by distance.
+
+@dataclass(frozen=True)
+class LinearRotationConfig:
+    """``rot``: how many entries of a head turn, the base of the frequencies, and the factor (``scaling.factor``) that slows them down."""
+
+    dims: int
+    base: float
+    factor: float = 1.0
+
+    @classmethod
+    def from_dict(cls, r: Mapping[str, Any], where: str) -> "LinearRotationConfig":
+        dims = _pos_int(r, "dims", where)
+        if dims % 2:
+            raise ConfigError(f"config.json: {where}'dims' must be even, got {dims}")
+        base = _number(r, "base", where)
+        if not base > 0:
+            raise ConfigError(f"config.json: {where}'base' must be positive, got {base}")
+        sc = _opt_sub(r, "scaling", where)
+        factor = _number(sc, "factor", where + "scaling.") if sc else 1.0
+        if not factor > 0:
+            raise ConfigError(f"config.json: {where}scaling.'factor' must be positive, got {factor}")
+        return cls(dims, base, factor)
+
+
+@dataclass(frozen=True)
+class SinoraxAttentionConfig:
+    """``attention``: causal softmax attention with biases, queries, keys and values turned (``rot``). ``attention_2``: sigmoid weights, a
+    penalty by distance, a window of ``window`` positions, no biases and no rotation (``rot`` is None)."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rot: Optional[LinearRotationConfig] = None
+    window: Optional[int] = None
+
+    @classmethod
+    def from_dict(cls, m: Mapping[str, Any], where: str, turned: bool) -> "SinoraxAttentionConfig":
+        heads, kv_heads = _pos_int(m, "heads", where), _pos_int(m, "kv_heads", where)
+        if heads % kv_heads:
+            raise ConfigError(f"config.json: {where}{heads} heads cannot share {kv_heads} kv_heads")
+        dim = _pos_int(m, "dim", where)
+        vdim = _pos_int(m, "vdim", where) if "vdim" in m else dim
+        scale = _number(m, "scale", where)
+        if not turned:
+            if m.get("rot") is not None:
+                raise ConfigError(f"config.json: {where}'rot' is not part of this mixer")
+            mask = _opt_sub(m, "mask", where)
+            return cls(heads, kv_heads, dim, vdim, scale, None, _pos_int(mask, "size", where + "mask.") if mask else None)
+        if m.get("mask") is not None:
+            raise ConfigError(f"config.json: {where}'mask' is not part of this mixer")
+        rot = LinearRotationConfig.from_dict(_sub(m, "rot", where), where + "rot.")
+        if rot.dims > dim:
+            raise ConfigError(f"config.json: {where}rot.dims {rot.dims} is more than dim {dim}")
+        if vdim % 2:
+            raise ConfigError(f"config.json: {where}'vdim' must be even (values turn in pairs), got {vdim}")
+        return cls(heads, kv_heads, dim, vdim, scale, rot, None)
+
+
+@dataclass(frozen=True)
+class BigramConfig:
+    """``embedding.bigram``: row ``(previous * mul_prev + token * mul_cur) mod buckets`` of a table is added to a token's embedding."""
+
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+    @classmethod
+    def from_dict(cls, b: Mapping[str, Any], where: str) -> "BigramConfig":
+        for key in ("mul_prev", "mul_cur"):
+            if isinstance(b.get(key), bool) or not isinstance(b.get(key), int) or not 0 <= b[key] < 1 << 31:
+                raise ConfigError(f"config.json: {where}'{key}' must be a count, got {b.get(key)!r}")
+        return cls(_pos_int(b, "buckets", where), b["mul_prev"], b["mul_cur"])
+
+
+@dataclass(frozen=True)
+class SinoraxLayerConfig:
+    kind: str                  # "attention" or "attention_2"
+    mixer: SinoraxAttentionConfig
+    ff: Optional[int]          # width of the feed-forward; None: the layer is a mixer alone
+
+
+@dataclass(frozen=True)
+class SinoraxConfig:
+    """The whole of a Sinorax config.json: vocabulary, width, the bigram table, the factor and the bound of the logits, the layers.
+    ``norm.eps`` is read for completeness; Dynamic Tanh has no use for it."""
+
+    architecture = "Sinorax"
+
+    vocab: int
+    width: int
+    eps: float
+    bigram: Optional[BigramConfig]
+    logit_scale: float
+    logit_softcap: Optional[float]
+    layers: tuple
+
+    @classmethod
+    def from_dict(cls, d: Mapping[str, Any]) -> "SinoraxConfig":
+        if not isinstance(d.get("layers"), (list, tuple)) or not d["layers"]:
+            raise ConfigError("config.json: 'layers' must be a list with at least one layer")
+        layers = []
+        for i, layer in enumerate(d["layers"]):
+            where = f"layers[{i}]."
+            if not isinstance(layer, Mapping):
+                raise ConfigError(f"config.json: layers[{i}] must be an object")
+            kind = layer.get("type")
+            if kind not in ("attention", "attention_2"):
+                raise ConfigError(f"config.json: {where}type {kind!r} is not one of ['attention', 'attention_2']")
+            mixer = SinoraxAttentionConfig.from_dict(_sub(layer, "mixer", where), where + "mixer.", turned=kind == "attention")
+            mlp = layer.get("mlp")
+            if mlp is not None and (not isinstance(mlp, Mapping) or mlp.get("kind", "dense") != "dense"):
+                raise ConfigError(f"config.json: {where}mlp must be null or an object of kind 'dense'")
+            layers.append(SinoraxLayerConfig(kind, mixer, _pos_int(mlp, "ff", where + "mlp.") if mlp is not None else None))
+        norm = _opt_sub(d, "norm", "")
+        embedding = _opt_sub(d, "embedding", "")
+        bigram = _opt_sub(embedding, "bigram", "embedding.") if embedding else None
+        scale = _number(d, "logit_scale", "") if d.get("logit_scale") is not None else 1.0
+        cap = _number(d, "logit_softcap", "") if d.get("logit_softcap") is not None else None
+        if cap is not None and not cap > 0:
+            raise ConfigError(f"config.json: 'logit_softcap' must be positive, got {cap}")
+        return cls(_pos_int(d, "vocab", ""), _pos_int(d, "width", ""), _number(norm, "eps", "norm.") if norm and "eps" in norm else 0.0,
+                   BigramConfig.from_dict(bigram, "embedding.bigram.") if bigram else None, scale, cap, tuple(layers))

@@ -12,9 +12,14 @@
 //   * a sliding window, as in the generic kernel; with `keep_first` the first tokens of the request stay visible after the
 //     window has passed them (at their true positions);
 //   * chunks: with `chunk` > 0 a position sees only keys of its own run of `chunk` positions, counted from the request's start;
-//   * a soft cap: score <- cap * tanh(score / cap), applied to the scaled score.
+//   * a soft cap: score <- cap * tanh(score / cap), applied to the scaled score;
+//   * a penalty by the logarithm of the distance: r1[head] * ln(1 + r2[head] * (p - j)) is taken off the scaled score;
+//   * weights without a softmax: with `sig_bias` a visible key's weight is sigmoid(score + sig_bias[head]), and nothing is divided
+//     by a sum over the keys (no maximum, no sink);
+//   * values that were turned by their positions when they were cached: the finished sum of the token at position p is turned
+//     back, pair m by the angle whose cosine and sine are turn_cos[n][m], turn_sin[n][m] (pairs (m, m + dv / 2), or neighbours).
 //
-// Each extra is off when its pointer is null (or `temp_every` is 0). Sink and gate are applied where a (token, head) is
+// Each extra is off when its pointer is null (or `temp_every` is 0). Sink, turn and gate are applied where a (token, head) is
 // finished: in the block when there is one slice, in the merge kernel otherwise. With `slice_keys` > 0 the slices lie at
 // fixed places of the request, so every bit of a token's result depends on its own position alone.
 #pragma once
@@ -38,7 +43,24 @@ struct Extras {
     int keep_first = 0;       // keys below this position are seen even when the window has passed them
     int chunk = 0;            // > 0: only keys with floor(key / chunk) == floor(position / chunk) are seen
     float softcap = 0.f;      // > 0: the scaled score s becomes softcap * tanh(s / softcap)
+    const float* sig_bias = nullptr;   // [nq]: sigmoid weights
+    const float* log_r1 = nullptr;     // [nq], with log_r2: the penalty by distance
+    const float* log_r2 = nullptr;
+    const float* turn_cos = nullptr;   // [N, dv / 2], with turn_sin: results are turned back
+    const float* turn_sin = nullptr;
+    int turn_neighbours = 0;  // 1: pairs (2 m, 2 m + 1)
 };
+
+// Where the pair of result entry `dim` lies: its number m, and the other entry.
+__device__ __forceinline__ int turn_pair(int dim, int dv, int neighbours, int& other) {
+    if (neighbours) { other = dim ^ 1; return dim >> 1; }
+    const int half = dv >> 1;
+    other = dim < half ? dim + half : dim - half;
+    return dim < half ? dim : dim - half;
+}
+
+// Entry `dim` (value a, its pair's other entry b) turned back by the angle (c, s): (u, v) -> (u c + v s, v c - u s).
+__device__ __forceinline__ float turn_back(float a, float b, bool first, float c, float s) { return first ? fmaf(b, s, a * c) : fmaf(-b, s, a * c); }
 
 // First key that position p may see apart from the kept first tokens (window and chunk together).
 __device__ __forceinline__ int first_visible(int p, int window, const Extras& ex) {
@@ -55,6 +77,7 @@ __device__ __forceinline__ float sigmoidf_(float x) { return 1.0f / (1.0f + expf
 template <typename T>
 __device__ __forceinline__ float finish_scale(float M, float L, const Extras& ex, int head, const T* gate_row) {
     float f = 1.f;
+    if (ex.sig_bias) L = 1.f;
     if (ex.sink) {
         const float sk = ex.sink[head];
         const float M2 = fmaxf(M, sk);
@@ -127,7 +150,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attn_ext_kernel(
     float m[GC], l[GC], acc[GC][DPL];
 #pragma unroll
     for (int g = 0; g < GC; ++g) {
-        m[g] = -INFINITY;
+        m[g] = ex.sig_bias ? 0.f : -INFINITY;   // (sigmoid weights are never rescaled)
         l[g] = 0.f;
 #pragma unroll
         for (int i = 0; i < DPL; ++i) acc[g][i] = 0.f;
@@ -177,10 +200,21 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attn_ext_kernel(
                 for (int g = 0; g < GC; ++g)
                     if (g < ng) s[g] += ex.rel[(size_t)r * nq + kvh * G + g0 + g];
             }
+            if (ex.log_r1) {
+                const float dist = (float)(p - key);
+#pragma unroll
+                for (int g = 0; g < GC; ++g)
+                    if (g < ng) s[g] -= ex.log_r1[kvh * G + g0 + g] * log1pf(ex.log_r2[kvh * G + g0 + g] * dist);
+            }
         }
         float corr[GC];
 #pragma unroll
         for (int g = 0; g < GC; ++g) {
+            if (ex.sig_bias) {
+                corr[g] = 1.f;
+                ps[(warp * GC + g) * 32 + lane] = (valid && g < ng) ? sigmoidf_(s[g] + ex.sig_bias[kvh * G + g0 + g]) : 0.f;
+                continue;
+            }
             const float sv = valid ? s[g] : -INFINITY;
             const float m_new = fmaxf(m[g], warp_max(sv));
             const float pv = valid ? expf(sv - m_new) : 0.f;
@@ -229,14 +263,22 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attn_ext_kernel(
         float M = -INFINITY;
 #pragma unroll
         for (int w = 0; w < WARPS; ++w) M = fmaxf(M, m_s[w * GC + g]);
-        float L = 0.f, A = 0.f;
+        int other = dim;
+        const bool turned = ex.turn_cos && num_splits == 1;
+        const int pair = turned ? turn_pair(dim, dv, ex.turn_neighbours, other) : 0;
+        float L = 0.f, A = 0.f, B = 0.f;
         if (M > -INFINITY) {
 #pragma unroll
             for (int w = 0; w < WARPS; ++w) {
                 const float f = expf(m_s[w * GC + g] - M);
                 L = fmaf(l_s[w * GC + g], f, L);
                 A = fmaf(acc_s[(w * GC + g) * DMAX + dim], f, A);
+                if (turned) B = fmaf(acc_s[(w * GC + g) * DMAX + other], f, B);
             }
+        }
+        if (turned) {
+            const size_t at = (size_t)n * (dv >> 1) + pair;
+            A = turn_back(A, B, dim < other, ex.turn_cos[at], ex.turn_sin[at]);
         }
         const int head = kvh * G + g0 + g;
         if (num_splits == 1) {
@@ -256,6 +298,7 @@ __global__ void attn_ext_combine_kernel(const float* __restrict__ part_acc, cons
                                         int nq, int dv, int num_splits, Extras ex) {
     constexpr int KEPT = 128;
     __shared__ float w_s[KEPT];
+    __shared__ float a_s[512];   // the merged sums, for results that are turned back (dv <= 512)
     __shared__ float scale_s, max_s;
     const size_t th = blockIdx.x;  // token * nq + head
     const int n = (int)(th / nq), head = (int)(th % nq);
@@ -288,10 +331,55 @@ __global__ void attn_ext_combine_kernel(const float* __restrict__ part_acc, cons
             const float w = s < KEPT ? w_s[s] : (ml[2 * s] > -INFINITY ? expf(ml[2 * s] - M) : 0.f);
             A = fmaf(acc[(size_t)s * dv + dim], w, A);
         }
+        if (ex.turn_cos) { a_s[dim] = A; continue; }
         float o = A * g;
         if (gate_row) o *= sigmoidf_(to_f32(gate_row[dim]));
         out[th * dv + dim] = from_f32<T>(o);
     }
+    if (!ex.turn_cos) return;
+    __syncthreads();
+    for (int dim = threadIdx.x; dim < dv; dim += blockDim.x) {
+        int other;
+        const size_t at = (size_t)n * (dv >> 1) + turn_pair(dim, dv, ex.turn_neighbours, other);
+        float o = turn_back(a_s[dim], a_s[other], dim < other, ex.turn_cos[at], ex.turn_sin[at]) * g;
+        if (gate_row) o *= sigmoidf_(to_f32(gate_row[dim]));
+        out[th * dv + dim] = from_f32<T>(o);
+    }
+}
+
+// What the tensor-core kernels are compiled for (see there).
+enum { PLAIN = 0, MASKS = 1, SIGMOID = 2 };
+inline int kind_of(const Extras& ex) {
+    if (ex.sig_bias) return SIGMOID;
+    return (ex.keep_first > 0 || ex.chunk > 0 || ex.softcap > 0.f || ex.log_r1) ? MASKS : PLAIN;
+}
+
+// A row's terms of its scores in the tensor-core kernels, whose weights are rounded to 8 bits: the fast exponential, logarithm and
+// division (errors of about 1e-7 of their results) do not show. The sigmoid of scale s - r1 ln(1 + r2 d) + bias is
+// 1 / (1 + 2^x) with x = -log2(e) (scale s + bias) + r1 log2(1 + r2 d).
+struct RowTerms {
+    float r1, r2, a, b;
+    __device__ __forceinline__ RowTerms(const Extras& ex, int head, float factor, bool used) : r1(0.f), r2(0.f), a(0.f), b(0.f) {
+        if (!used) return;
+        if (ex.log_r1) { r1 = ex.log_r1[head]; r2 = ex.log_r2[head]; }
+        if (ex.sig_bias) {
+            a = -1.4426950408889634f * factor;
+            b = -1.4426950408889634f * ex.sig_bias[head];
+        }
+    }
+    __device__ __forceinline__ static float lg2(float v) { float y; asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(v)); return y; }
+    __device__ __forceinline__ static float ex2(float v) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(v)); return y; }
+    __device__ __forceinline__ float penalty(float dist) const { return r1 * 0.6931471805599453f * lg2(fmaf(r2, dist, 1.0f)); }
+    // (dist < 0, a key the row does not see, may give anything: the caller masks it)
+    __device__ __forceinline__ float sigmoid(float s, float dist) const {
+        return __fdividef(1.0f, 1.0f + ex2(fmaf(r1, lg2(fmaf(r2, dist, 1.0f)), fmaf(a, s, b))));
+    }
+};
+
+// True if the extras contradict each other or lack a pointer.
+inline bool bad_extras(const Extras& ex, int dv) {
+    return (ex.gate_mode && !ex.gate) || (ex.sig_bias && ex.sink) || ((ex.log_r1 == nullptr) != (ex.log_r2 == nullptr)) ||
+           ((ex.turn_cos == nullptr) != (ex.turn_sin == nullptr)) || (ex.turn_cos && dv % 2);
 }
 
 inline size_t smem_bytes(int GC, int DPL, int dk) {
@@ -320,7 +408,7 @@ int paged_attention_ext(const T* q, int q_stride, const T* k_pool, const T* v_po
     if (N <= 0) return 0;
     if (nkv <= 0 || nq % nkv || dk <= 0 || dv <= 0 || dv > 512 || dk > 4096 || page_size <= 0 || num_splits < 1 || slice_keys < 0 ||
         slice_keys % 32 || (num_splits > 1 && !scratch) || (!v_pool && dv > dk) || (ex.rel && (!ex.rows_of || ex.rel_rows < 1)) ||
-        (ex.gate_mode && !ex.gate))
+        bad_extras(ex, dv))
         return LLMIE_ERR_BAD_ARGUMENT;
     constexpr int VN = Vec16<T>::N;
     const int vec_ok = dk % VN == 0 && ((uintptr_t)k_pool % 16 == 0);

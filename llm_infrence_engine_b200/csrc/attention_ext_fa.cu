@@ -48,10 +48,12 @@ __device__ __forceinline__ uint32_t pack2(float a, float b) {
 }
 
 // KD: steps of 16 over the key entries (dk = 16 KD); NV: pairs of n8 tiles over the value entries (dv = 16 NV)
-// MASKS: kept first tokens, chunks and the soft cap are compiled in (else they are not looked at, and cost nothing)
-template <int KD, int NV, bool MASKS>
+// KIND: PLAIN, MASKS (kept first tokens, chunks, the soft cap and the penalty by distance are compiled in; else they are not looked at,
+// and cost nothing) or SIGMOID (weights without a softmax, with the penalty by distance: no maxima, no sums, nothing is rescaled)
+template <int KD, int NV, int KIND>
 __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
     extern __shared__ __align__(16) unsigned char smem_raw[];
+    constexpr bool MASKS = KIND == attn_ext::MASKS, SIG = KIND == attn_ext::SIGMOID;
     constexpr int dk = 16 * KD, dv = 16 * NV, ks = dk + 8, vs = dv + 8;
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);            // [ROWS][ks]: only until the queries are in registers
     bf16* Ks = Qs + ROWS * ks;                               // [2][KEYS][ks]
@@ -104,6 +106,7 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
         if (P.ex.temp_every > 0 && ok) f = P.scale * (1.0f + P.ex.temp_coef * logf((float)((row_pos[i] + 1) / P.ex.temp_every + 1)));
         row_factor[i] = f;
     }
+    const attn_ext::RowTerms terms0(P.ex, row_head[0], row_factor[0], SIG || MASKS), terms1(P.ex, row_head[1], row_factor[1], SIG || MASKS);
     const bool warp_live = warp * 16 < ntok * gh;   // a warp without rows only fetches
     // the span of my warp's positions: a chunk that all its rows see in full needs no mask arithmetic
     int w_min = row_pos[0] < 0 || row_pos[1] < 0 ? -1 : min(row_pos[0], row_pos[1]), w_lo = max(row_lo[0], row_lo[1]);
@@ -183,9 +186,29 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
                 }
             }
         }
+        uint32_t pf[4][4];   // the weights, rounded to bfloat16 as the products use them, as A operands
         // scale, bias, mask; element (tile t, e): row gid + 8 * (e >> 1), key base + t * 8 + 2 * tig + (e & 1)
-        float mx[2] = {-INFINITY, -INFINITY};
         const bool interior = c >= npre && w_min >= 0 && base + KEYS - 1 <= w_min && base + KEYS <= end && base >= lo && base >= w_lo;
+        if constexpr (SIG) {
+#pragma unroll
+            for (int t = 0; t < 8; ++t) {
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const attn_ext::RowTerms& rt = i ? terms1 : terms0;
+                    const int key = base + t * 8 + 2 * tig;
+                    float w[2];
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) w[e] = rt.sigmoid(s[t][2 * i + e], (float)(row_pos[i] - key - e));
+                    if (!interior) {
+#pragma unroll
+                        for (int e = 0; e < 2; ++e)
+                            if (key + e > row_pos[i] || key + e >= range_hi || key + e < range_lo || key + e < row_lo[i]) w[e] = 0.f;
+                    }
+                    pf[t >> 1][(t & 1) * 2 + i] = pack2(w[0], w[1]);
+                }
+            }
+        } else {
+        float mx[2] = {-INFINITY, -INFINITY};
         if (interior) {
 #pragma unroll
             for (int t = 0; t < 8; ++t)
@@ -204,6 +227,7 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
                             v += P.ex.rel[(size_t)br * P.nq + row_head[i]];
                         }
                     }
+                    if (MASKS && P.ex.log_r1) v -= (i ? terms1 : terms0).penalty((float)(row_pos[i] - (base + t * 8 + 2 * tig + (e & 1))));
                     s[t][e] = v;
                     mx[i] = fmaxf(mx[i], v);
                 }
@@ -230,6 +254,7 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
                                 v += P.ex.rel[(size_t)br * P.nq + row_head[i]];
                             }
                         }
+                        if (MASKS && P.ex.log_r1) v -= (i ? terms1 : terms0).penalty((float)(p - key));
                     }
                     s[t][e] = v;
                     mx[i] = fmaxf(mx[i], v);
@@ -245,8 +270,7 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
             corr[i] = expf(m_run[i] - m_use[i]);
             m_run[i] = m_new;
         }
-        // the weights, rounded to bfloat16 as the products use them (the sums are taken over the rounded weights), as A operands
-        uint32_t pf[4][4];
+        // (the sums are taken over the rounded weights)
 #pragma unroll
         for (int t = 0; t < 8; ++t) {
 #pragma unroll
@@ -266,6 +290,7 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
         }
 #pragma unroll
         for (int t = 0; t < 2 * NV; ++t) { acc[t][0] *= corr[0]; acc[t][1] *= corr[0]; acc[t][2] *= corr[1]; acc[t][3] *= corr[1]; }
+        }
         // ---- O += P V
         {
             const bf16* vb = Vs + stage * KEYS * vs + (lane & 15) * vs + (lane >> 4) * 8;
@@ -295,7 +320,31 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
                 f = expf(M - M2);
                 L = L * f + expf(sk - M2);
             }
-            const float inv = f / L;
+            const float inv = SIG ? 1.f : f / L;
+            if (P.ex.turn_cos) {   // both entries of every pair are this thread's
+                const float* tc = P.ex.turn_cos + (size_t)n * (dv / 2);
+                const float* ts = P.ex.turn_sin + (size_t)n * (dv / 2);
+#pragma unroll
+                for (int t = 0; t < NV; ++t) {
+                    if (P.ex.turn_neighbours) {
+#pragma unroll
+                        for (int u = 0; u < 2; ++u) {   // tiles 2 t and 2 t + 1: entries col, col + 1
+                            const int m = ((2 * t + u) * 8 + 2 * tig) >> 1;
+                            const float a = acc[2 * t + u][2 * i], b = acc[2 * t + u][2 * i + 1];
+                            acc[2 * t + u][2 * i] = attn_ext::turn_back(a, b, true, tc[m], ts[m]);
+                            acc[2 * t + u][2 * i + 1] = attn_ext::turn_back(b, a, false, tc[m], ts[m]);
+                        }
+                    } else {
+#pragma unroll
+                        for (int u = 0; u < 2; ++u) {   // entry t * 8 + 2 tig + u and its partner dv / 2 = 8 NV further on
+                            const int m = t * 8 + 2 * tig + u;
+                            const float a = acc[t][2 * i + u], b = acc[t + NV][2 * i + u];
+                            acc[t][2 * i + u] = attn_ext::turn_back(a, b, true, tc[m], ts[m]);
+                            acc[t + NV][2 * i + u] = attn_ext::turn_back(b, a, false, tc[m], ts[m]);
+                        }
+                    }
+                }
+            }
             const bf16* gate_row = P.ex.gate_mode ? reinterpret_cast<const bf16*>(P.ex.gate) + (size_t)n * P.ex.gate_stride : nullptr;
             float gh1 = 1.f;
             if (P.ex.gate_mode == 1) gh1 = attn_ext::sigmoidf_(to_f32(gate_row[head]));
@@ -316,7 +365,7 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
             float* pa = P.part_acc + slot * dv;
 #pragma unroll
             for (int t = 0; t < 2 * NV; ++t) *reinterpret_cast<float2*>(pa + t * 8 + 2 * tig) = make_float2(acc[t][2 * i], acc[t][2 * i + 1]);
-            if (tig == 0) { P.part_ml[slot * 2] = m_run[i]; P.part_ml[slot * 2 + 1] = l_run[i]; }
+            if (tig == 0) { P.part_ml[slot * 2] = SIG ? 0.f : m_run[i]; P.part_ml[slot * 2 + 1] = l_run[i]; }
         }
     }
 }
@@ -324,20 +373,23 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
 size_t smem_bytes(int dk, int dv) { return 2 * ((size_t)ROWS * (dk + 8) + 2 * KEYS * (dk + 8) + 2 * KEYS * (dv + 8)); }
 size_t bias_bytes(int rel_rows, int gh, int n_rows_of) { return sizeof(float) * (size_t)rel_rows * gh + 2 * (size_t)((n_rows_of + 1) & ~1); }
 
-template <int KD, int NV, bool MASKS>
+template <int KD, int NV, int KIND>
 int launch_as(const Params& P, dim3 grid, size_t smem, cudaStream_t s) {
     static bool set = false;
     if (!set) {
-        cudaFuncSetAttribute(attn_ext_fa_kernel<KD, NV, MASKS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
+        cudaFuncSetAttribute(attn_ext_fa_kernel<KD, NV, KIND>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024);
         set = true;
     }
-    return launch_kernel(attn_ext_fa_kernel<KD, NV, MASKS>, grid, dim3(THREADS), smem, s, P);
+    return launch_kernel(attn_ext_fa_kernel<KD, NV, KIND>, grid, dim3(THREADS), smem, s, P);
 }
 
 template <int KD, int NV>
 int launch(const Params& P, dim3 grid, size_t smem, cudaStream_t s) {
-    if (P.ex.keep_first > 0 || P.ex.chunk > 0 || P.ex.softcap > 0.f) return launch_as<KD, NV, true>(P, grid, smem, s);
-    return launch_as<KD, NV, false>(P, grid, smem, s);
+    switch (attn_ext::kind_of(P.ex)) {
+        case attn_ext::SIGMOID: return launch_as<KD, NV, attn_ext::SIGMOID>(P, grid, smem, s);
+        case attn_ext::MASKS: return launch_as<KD, NV, attn_ext::MASKS>(P, grid, smem, s);
+        default: return launch_as<KD, NV, attn_ext::PLAIN>(P, grid, smem, s);
+    }
 }
 
 }  // namespace
@@ -354,7 +406,8 @@ LLMIE_API int llmie_paged_attention_ext_fa(const bf16* q, int q_stride, const bf
                                            bf16* out, float* scratch, int N, int nq, int nkv, int dk, int dv, int page_size, float scale,
                                            int window, int num_splits, float temp_coef, int temp_every, const float* rel, const int* rows_of,
                                            int n_rows_of, int rel_rows, const float* sink, const bf16* gate, int gate_stride, int gate_mode,
-                                           int keep_first, int chunk, float softcap, cudaStream_t s) {
+                                           int keep_first, int chunk, float softcap, const float* sig_bias, const float* log_r1,
+                                           const float* log_r2, const float* turn_cos, const float* turn_sin, int turn_neighbours, cudaStream_t s) {
     if (N <= 0 || tiles <= 0) return 0;
     if (nkv <= 0 || nq % nkv || !llmie_attention_ext_fa_fits(dk, dv, v_pool != nullptr, nq / nkv) || !tile_info || page_size <= 0 ||
         num_splits < 1 || (num_splits > 1 && !scratch) || q_stride % 8 || ((uintptr_t)q % 16) || ((uintptr_t)k_pool % 16) ||
@@ -371,6 +424,9 @@ LLMIE_API int llmie_paged_attention_ext_fa(const bf16* q, int q_stride, const bf
     P.ex.temp_coef = temp_coef; P.ex.temp_every = temp_every; P.ex.rel = rel; P.ex.rows_of = rows_of; P.ex.n_rows_of = n_rows_of;
     P.ex.rel_rows = rel_rows; P.ex.sink = sink; P.ex.gate = gate; P.ex.gate_stride = gate_stride; P.ex.gate_mode = gate_mode;
     P.ex.keep_first = keep_first; P.ex.chunk = chunk; P.ex.softcap = softcap;
+    P.ex.sig_bias = sig_bias; P.ex.log_r1 = log_r1; P.ex.log_r2 = log_r2;
+    P.ex.turn_cos = turn_cos; P.ex.turn_sin = turn_sin; P.ex.turn_neighbours = turn_neighbours;
+    if (attn_ext::bad_extras(P.ex, dv) || (sig_bias && (rel || keep_first || chunk || softcap != 0.f))) return LLMIE_ERR_BAD_ARGUMENT;
     if ((long long)nkv * P.head_chunks > 65535 || num_splits > 65535) return LLMIE_ERR_BAD_ARGUMENT;
     size_t smem = smem_bytes(dk, dv);
     P.bias_in_smem = 0;

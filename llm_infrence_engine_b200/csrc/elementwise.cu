@@ -51,6 +51,58 @@ LLMIE_API int llmie_embed(const int* ids, const void* table, float* out, int N, 
 }
 
 // ------------------------------------------------------------------------------------------------
+// x[n, :] = table[ids[n], :] * scale + bigram[row(n), :], widened to float, with
+//   row(n) = (previous token * mul_prev + token * mul_cur) mod buckets, or `buckets` (the last row) for a request's first token.
+// The previous token of a request's first row in the step lies in last[slot] (the request's state slot); the block of that row
+// reads it and then leaves the request's last token of the step there, so nobody reads what another block writes.
+// starts: [R + 1] first row of each request. Products and sums of the row number are 64-bit.
+template <typename T>
+__global__ void embed_bigram_kernel(const int* __restrict__ ids, const T* __restrict__ table, const T* __restrict__ bigram, float* __restrict__ out,
+                                    const int* __restrict__ positions, const int* __restrict__ token_seq, const int* __restrict__ starts, int R,
+                                    int* __restrict__ last, long long buckets, long long mul_prev, long long mul_cur, int N, int H, float scale) {
+    __shared__ long long row_s;
+    pdl_trigger();
+    pdl_wait();
+    const int n = blockIdx.x;
+    if (threadIdx.x == 0) {
+        const int slot = token_seq[n];
+        const bool opens = n == 0 || token_seq[n - 1] != slot || positions[n] == 0;   // (padding rows share a slot; their position is 0)
+        int previous = -1;
+        if (positions[n] > 0) previous = opens ? last[slot] : ids[n - 1];
+        if (opens) {   // which request is it? the last one whose rows start at or before n
+            int lo = 0, hi = R - 1;
+            while (lo < hi) {
+                const int mid = (lo + hi + 1) >> 1;
+                if (starts[mid] <= n) lo = mid; else hi = mid - 1;
+            }
+            const int end = min(starts[lo + 1], N);
+            last[slot] = ids[max(end, n + 1) - 1];
+        }
+        long long row = buckets;
+        if (previous >= 0) row = ((long long)previous * mul_prev + (long long)ids[n] * mul_cur) % buckets;
+        row_s = row < 0 ? row + buckets : row;
+    }
+    __syncthreads();
+    const T* a = table + (size_t)ids[n] * H;
+    const T* b = bigram + (size_t)row_s * H;
+    float* o = out + (size_t)n * H;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = to_f32(a[i]) * scale + to_f32(b[i]);
+}
+
+LLMIE_API int llmie_embed_bigram(const int* ids, const void* table, const void* bigram, float* out, const int* positions, const int* token_seq,
+                                 const int* starts, int R, int* last, long long buckets, long long mul_prev, long long mul_cur, int N, int H,
+                                 int dtype, float scale, cudaStream_t s) {
+    if (N <= 0) return 0;
+    if (R < 1 || buckets < 1 || H < 1) return LLMIE_ERR_BAD_ARGUMENT;
+    const int threads = H >= 1024 ? 256 : 128;
+    if (dtype == DT_F32)
+        return launch_kernel(embed_bigram_kernel<float>, dim3(N), dim3(threads), 0, s, ids, (const float*)table, (const float*)bigram, out, positions,
+                             token_seq, starts, R, last, buckets, mul_prev, mul_cur, N, H, scale);
+    return launch_kernel(embed_bigram_kernel<bf16>, dim3(N), dim3(threads), 0, s, ids, (const bf16*)table, (const bf16*)bigram, out, positions,
+                         token_seq, starts, R, last, buckets, mul_prev, mul_cur, N, H, scale);
+}
+
+// ------------------------------------------------------------------------------------------------
 // ids[i] = previous[src[i]] where src[i] >= 0: a request's next token taken from the tokens the step before chose, which
 // are still on the device (the host has not read them yet)
 __global__ void feed_tokens_kernel(int* __restrict__ ids, const int* __restrict__ src, const int* __restrict__ previous, int N) {
@@ -527,22 +579,27 @@ LLMIE_API int llmie_kv_store(const void* z, int z_stride, int k_col, int v_col, 
 
 // ------------------------------------------------------------------------------------------------
 // out = act(in), elementwise in 32-bit. kind 0: the tanh form of GELU, 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)));
-// kind 1: a soft cap, param * tanh(z / param).
+// kind 1: a soft cap on a scaled input, param * tanh(scale z / param); kind 2: the exact GELU, 0.5 z (1 + erf(z / sqrt 2)); kind 3: scale z.
 // With `clear_in` the input is set to zero after it was read (a float32 accumulation buffer of a split-K product).
 template <typename TI, typename TO>
-__global__ void act_kernel(TI* __restrict__ in, TO* __restrict__ out, long long total, int kind, int clear_in, float param) {
+__global__ void act_kernel(TI* __restrict__ in, TO* __restrict__ out, long long total, int kind, int clear_in, float param, float scale) {
     pdl_trigger();
     pdl_wait();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
     const float z = to_f32(in[i]);
     if (clear_in) in[i] = from_f32<TI>(0.f);
-    const float y = kind == 1 ? param * tanhf(z / param) : 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    float y;
+    if (kind == 1) y = param * tanhf(scale * z / param);
+    else if (kind == 2) y = 0.5f * z * (1.0f + erff(0.7071067811865476f * z));
+    else if (kind == 3) y = scale * z;
+    else y = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
     out[i] = from_f32<TO>(y);
 }
 
 // bfloat16 in and out, 8 elements (16 bytes) per thread. The result is rounded to bfloat16 (8 bits), so the hyperbolic tangent is
-// the fast 32-bit form (tanh(a) = 1 - 2 / (exp(2a) + 1), errors of about 1e-7).
+// the fast 32-bit form (tanh(a) = 1 - 2 / (exp(2a) + 1), errors of about 1e-7). ERF: the exact GELU instead.
+template <bool ERF>
 __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict__ in, bf16* __restrict__ out, long long items) {
     pdl_trigger();
     pdl_wait();
@@ -558,6 +615,7 @@ __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict_
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
             const float v = z[2 * j + k];
+            if (ERF) { y[k] = 0.5f * v * (1.0f + erff(0.7071067811865476f * v)); continue; }
             const float a = 0.7978845608028654f * (v + 0.044715f * v * v * v);
             const float t = 1.0f - __fdividef(2.0f, __expf(2.0f * a) + 1.0f);
             y[k] = 0.5f * v * (1.0f + t);
@@ -568,15 +626,19 @@ __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict_
     *reinterpret_cast<uint4*>(out + i * 8) = packed;
 }
 
-LLMIE_API int llmie_act(void* in, void* out, long long total, int kind, int clear_in, float param, int in_dtype, int out_dtype, cudaStream_t s) {
+LLMIE_API int llmie_act(void* in, void* out, long long total, int kind, int clear_in, float param, float scale, int in_dtype,
+                        int out_dtype, cudaStream_t s) {
     if (total <= 0) return 0;
-    if (kind < 0 || kind > 1 || (kind == 1 && !(param > 0.f))) return LLMIE_ERR_BAD_ARGUMENT;
-    if (kind == 0 && in_dtype == DT_BF16 && out_dtype == DT_BF16 && !clear_in && total % 8 == 0 && ((uintptr_t)in % 16 == 0) && ((uintptr_t)out % 16 == 0))
-        return launch_kernel(act_bf16x8_kernel, dim3((unsigned)((total / 8 + 255) / 256)), dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
+    if (kind < 0 || kind > 3 || (kind == 1 && !(param > 0.f))) return LLMIE_ERR_BAD_ARGUMENT;
+    if ((kind == 0 || kind == 2) && in_dtype == DT_BF16 && out_dtype == DT_BF16 && !clear_in && total % 8 == 0 && ((uintptr_t)in % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
+        const dim3 blocks((unsigned)((total / 8 + 255) / 256));
+        if (kind == 2) return launch_kernel(act_bf16x8_kernel<true>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
+        return launch_kernel(act_bf16x8_kernel<false>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
+    }
     const dim3 grid((unsigned)((total + 255) / 256));
-    if (in_dtype == DT_F32 && out_dtype == DT_F32) return launch_kernel(act_kernel<float, float>, grid, dim3(256), 0, s, (float*)in, (float*)out, total, kind, clear_in, param);
-    if (in_dtype == DT_F32 && out_dtype == DT_BF16) return launch_kernel(act_kernel<float, bf16>, grid, dim3(256), 0, s, (float*)in, (bf16*)out, total, kind, clear_in, param);
-    if (in_dtype == DT_BF16 && out_dtype == DT_BF16) return launch_kernel(act_kernel<bf16, bf16>, grid, dim3(256), 0, s, (bf16*)in, (bf16*)out, total, kind, clear_in, param);
+    if (in_dtype == DT_F32 && out_dtype == DT_F32) return launch_kernel(act_kernel<float, float>, grid, dim3(256), 0, s, (float*)in, (float*)out, total, kind, clear_in, param, scale);
+    if (in_dtype == DT_F32 && out_dtype == DT_BF16) return launch_kernel(act_kernel<float, bf16>, grid, dim3(256), 0, s, (float*)in, (bf16*)out, total, kind, clear_in, param, scale);
+    if (in_dtype == DT_BF16 && out_dtype == DT_BF16) return launch_kernel(act_kernel<bf16, bf16>, grid, dim3(256), 0, s, (bf16*)in, (bf16*)out, total, kind, clear_in, param, scale);
     return LLMIE_ERR_BAD_ARGUMENT;
 }
 

@@ -17,7 +17,8 @@
 //
 // grid = (ceil(N / 128), ceil(M / TN), k_splits). Splitting K gives small matrices enough blocks to pull
 // the whole memory system; the partial sums meet in the float32 output by atomic addition, which is
-// also how a projection adds itself into the residual stream without a separate kernel.
+// also how a projection adds itself into the residual stream without a separate kernel. A bias per output is added once, by the
+// blocks of the first K range.
 //
 // Every wait on an mbarrier is bounded: after SPIN_LIMIT polls the block records an error in
 // `error_flag`, stops issuing work, lets the copies it started land (again bounded), frees its tensor
@@ -32,7 +33,7 @@ constexpr int BM = 128, BK = 64, STAGES = 4, UMMA_K = 16;
 template <int TN>
 __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x,
                                                       float* __restrict__ out, int ldo, int M, int N, int K, int kb_per_split,
-                                                      int accumulate, int* error_flag) {
+                                                      int accumulate, int* error_flag, const bf16* __restrict__ bias) {
     constexpr int W_BYTES = BM * BK * 2, X_BYTES = TN * BK * 2, STAGE_BYTES = W_BYTES + X_BYTES;
     constexpr int COLS = TN < 32 ? 32 : TN;  // tensor-memory columns: a power of two, at least 32
     extern __shared__ unsigned char raw[];
@@ -116,6 +117,7 @@ __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CU
     if (done) {
         const int n = n0 + warp * 32 + lane;
         const int rows = min(TN, M - m0);
+        const float add = (bias && n < N && blockIdx.z == 0) ? to_f32(bias[n]) : 0.f;
 #pragma unroll
         for (int c = 0; c < TN; c += 16) {
             uint32_t v[16];
@@ -127,8 +129,8 @@ __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CU
                     const int m = c + j;
                     if (m < rows) {
                         float* dst = out + (size_t)(m0 + m) * ldo + n;
-                        if (accumulate) atomicAdd(dst, __uint_as_float(v[j]));
-                        else *dst = __uint_as_float(v[j]);
+                        if (accumulate) atomicAdd(dst, __uint_as_float(v[j]) + add);
+                        else *dst = __uint_as_float(v[j]) + add;
                     }
                 }
             }
@@ -153,7 +155,7 @@ __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CU
 // ------------------------------------------------------------------------------------------------ host side
 template <int TN>
 int launch(const CUtensorMap& mw, const CUtensorMap& mx, float* out, int ldo, int M, int N, int K, int k_splits, int accumulate,
-           int* error_flag, cudaStream_t s) {
+           int* error_flag, const bf16* bias, cudaStream_t s) {
     constexpr size_t smem = (size_t)STAGES * (BM * BK * 2 + TN * BK * 2) + 1024 + 256;
     static bool set = false;
     if (!set) {
@@ -165,11 +167,11 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, float* out, int ldo, in
     const int per = (nkb + k_splits - 1) / k_splits;
     const int splits = (nkb + per - 1) / per;  // no empty split
     const dim3 grid((N + BM - 1) / BM, (M + TN - 1) / TN, splits);
-    return launch_kernel(gemm_tc_kernel<TN>, grid, dim3(128), smem, s, mw, mx, out, ldo, M, N, K, per, accumulate, error_flag);
+    return launch_kernel(gemm_tc_kernel<TN>, grid, dim3(128), smem, s, mw, mx, out, ldo, M, N, K, per, accumulate, error_flag, bias);
 }
 
 static int run(const bf16* x, const bf16* w, float* out, int ldo, int M, int N, int K, int k_splits, int accumulate, int* error_flag,
-               cudaStream_t s) {
+               const bf16* bias, cudaStream_t s) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0 || K % 8 || ((uintptr_t)w & 15) || ((uintptr_t)x & 15) || k_splits < 1 || (!accumulate && k_splits != 1) || !error_flag ||
         ldo < N)
@@ -180,16 +182,16 @@ static int run(const bf16* x, const bf16* w, float* out, int ldo, int M, int N, 
     if (rc) return rc;
     rc = tensor_map(x, M, K, TN, &mx);
     if (rc) return rc;
-    if (TN == 16) return launch<16>(mw, mx, out, ldo, M, N, K, k_splits, accumulate, error_flag, s);
-    if (TN == 32) return launch<32>(mw, mx, out, ldo, M, N, K, k_splits, accumulate, error_flag, s);
-    return launch<64>(mw, mx, out, ldo, M, N, K, k_splits, accumulate, error_flag, s);
+    if (TN == 16) return launch<16>(mw, mx, out, ldo, M, N, K, k_splits, accumulate, error_flag, bias, s);
+    if (TN == 32) return launch<32>(mw, mx, out, ldo, M, N, K, k_splits, accumulate, error_flag, bias, s);
+    return launch<64>(mw, mx, out, ldo, M, N, K, k_splits, accumulate, error_flag, bias, s);
 }
 
 }  // namespace
 
 // x [M, K] and w [N, K] bfloat16 row-major (K a multiple of 8, bases 16-byte aligned), out float32 with row stride ldo.
-// accumulate = 0 needs k_splits = 1 and stores; accumulate = 1 adds atomically into what `out` holds.
+// accumulate = 0 needs k_splits = 1 and stores; accumulate = 1 adds atomically into what `out` holds. bias: [N] bfloat16 or null.
 LLMIE_API int llmie_gemm_tc(const bf16* x, const bf16* w, float* out, int ldo, int M, int N, int K, int k_splits, int accumulate,
-                            int* error_flag, cudaStream_t s) {
-    return run(x, w, out, ldo, M, N, K, k_splits, accumulate, error_flag, s);
+                            int* error_flag, const bf16* bias, cudaStream_t s) {
+    return run(x, w, out, ldo, M, N, K, k_splits, accumulate, error_flag, bias, s);
 }

@@ -86,6 +86,8 @@ class CudaKernels:
         # sublayer, which adds and normalises in one pass: (stream, result, the post-norm's weight, eps, plain); ``plain``: the result
         # is only scaled element by element by the weight (a layer scale), not normed
         self._pending_post: Optional[tuple] = None
+        # ... and one that a Dynamic Tanh closes waits here: (stream, result, alpha, weight, bias)
+        self._pending_tanh: Optional[tuple] = None
         self._state_lists: dict = {}   # the addresses of a runner's state tensors on the device (zero_fresh_states)
         self._fresh: list = []   # zeroed tensors of ``zeros_like_rows`` that nothing has been added into yet
         # ``zeros_like_rows`` hands out views of one float32 buffer that is zero between uses: the stream kernels that read a
@@ -112,7 +114,8 @@ class CudaKernels:
                    "llmie_selective_scan", "llmie_weighted_pair", "llmie_moe_route", "llmie_moe_sort", "llmie_moe_gemm", "llmie_moe_combine",
                    "llmie_moe_tile_rows", "llmie_moe_router", "llmie_moe_gather", "llmie_moe_grouped_tc", "llmie_moe_grouped_tc_rows",
                    "llmie_embed_add", "llmie_mlstm_prepare", "llmie_mlstm_scan", "llmie_mlstm_finish", "llmie_paged_attention_talk",
-                   "llmie_attention_talk_slice", "llmie_attention_talk_mma_fits", "llmie_paged_attention_talk_mma"):
+                   "llmie_attention_talk_slice", "llmie_attention_talk_mma_fits", "llmie_paged_attention_talk_mma", "llmie_embed_bigram",
+                   "llmie_dynamic_tanh"):
             getattr(self.lib, fn).restype = ctypes.c_int
         # two forms of the gate/up kernel live in source files of their own, and the library also builds without them
         self._gate_up_cluster = self._gate_up_pair = self._gate_up_glu_pair = None
@@ -143,6 +146,7 @@ class CudaKernels:
         self._pending_add = None
         self._pending_streams = None
         self._pending_post = None
+        self._pending_tanh = None
         self._fresh = []
         self._dirty_qkv = None
         for t in [self._acc, self._acc_qkv, *self._zero_bufs, *self._retired_acc]:
@@ -190,6 +194,26 @@ class CudaKernels:
         out = torch.empty((N, H), dtype=torch.float32, device=table.device)
         self._check(self.lib.llmie_embed(_ptr(token_ids), _ptr(table), _ptr(out), N, H, self._dt(table, "table"), ctypes.c_float(scale),
                                         self._stream()), "embed")
+        return out
+
+    def embed_bigram(self, token_ids, table, bigram, buckets: int, mul_prev: int, mul_cur: int, positions, token_seq, seq_starts, num_seqs: int, last,
+                     scale: float = 1.0):
+        """``table[token] * scale + bigram[row]`` with ``row = (previous * mul_prev + token * mul_cur) mod buckets``, or the last row for a
+        request's first token. ``last`` (int32, one per state slot) holds every request's last token of the step before; the kernel
+        reads it for a portion's first row and leaves the portion's last token there."""
+        for name, t in (("token_ids", token_ids), ("positions", positions), ("token_seq", token_seq), ("seq_starts", seq_starts)):
+            self._need(t, name, torch.int32, 1)
+        self._need(last, "last", torch.int32)
+        self._need(table, "table", None, 2)
+        self._need(bigram, "bigram", table.dtype, 2)
+        N, H = token_ids.shape[0], table.shape[1]
+        if tuple(bigram.shape) != (buckets + 1, H) or seq_starts.shape[0] < num_seqs + 1:
+            raise KernelError("embed_bigram: the bigram table needs one row per bucket and one more, as wide as the embedding")
+        out = torch.empty((N, H), dtype=torch.float32, device=table.device)
+        self._check(self.lib.llmie_embed_bigram(_ptr(token_ids), _ptr(table), _ptr(bigram), _ptr(out), _ptr(positions), _ptr(token_seq), _ptr(seq_starts),
+                                                int(num_seqs), _ptr(last), ctypes.c_longlong(buckets), ctypes.c_longlong(mul_prev),
+                                                ctypes.c_longlong(mul_cur), N, H, self._dt(table, "table"), ctypes.c_float(scale), self._stream()),
+                    "embed_bigram")
         return out
 
     def embed_add(self, token_ids, table, residual, scale: float = 1.0):
@@ -297,6 +321,10 @@ class CudaKernels:
             x, y, w_post, eps, plain = self._pending_post
             self._pending_post = None
             self._layernorm(x, y, w_post, None, eps, None, None, "post_norm_add", post_plain=plain)
+        if self._pending_tanh is not None:
+            x, y, alpha, weight, bias = self._pending_tanh
+            self._pending_tanh = None
+            self._dynamic_tanh(x, (y, alpha, weight, bias), None, None, None, "post_tanh_add")
 
     def _take_pending(self, residual, out_dtype):
         """The put-off addend for ``residual`` if there is one that the norm kernel can add on its way (same dtype as its output)."""
@@ -333,8 +361,8 @@ class CudaKernels:
         grows all the same, the outgrown buffer is kept for the graphs that hold its address)."""
         self._transient(self.tc_max_rows, widest, torch.device(device))
 
-    def linear(self, x, w, out_dtype=None, add_to=None, transient=False):
-        """``x w^T`` for ``x [rows, K]`` and ``w [outputs, K]``.
+    def linear(self, x, w, out_dtype=None, add_to=None, transient=False, bias=None):
+        """``x w^T`` (``+ bias``, one number per output in the type of ``x``) for ``x [rows, K]`` and ``w [outputs, K]``.
 
         ``add_to``: a float32 ``[rows, outputs]`` tensor (the residual stream) that the product is added into;
         nothing is returned. ``transient``: the caller hands the result straight to ``rope_kv_write`` or ``silu_mul``
@@ -348,8 +376,9 @@ class CudaKernels:
                 self._need(w, "w", x.dtype, 2)
                 if x.shape[1] != w.shape[1]:
                     raise KernelError(f"linear: x has {x.shape[1]} columns, w has {w.shape[1]}")
+                self._check_bias(bias, x, w)
                 self.launches += 1
-                return torch.nn.functional.linear(x, w)
+                return torch.nn.functional.linear(x, w, bias)
             x = x.contiguous()
             self.launches += 1
         self._need(x, "x", None, 2)
@@ -358,6 +387,7 @@ class CudaKernels:
         self._need(w, "w", x.dtype, 2)
         if K != w.shape[1]:
             raise KernelError(f"linear: x has {K} columns, w has {w.shape[1]}")
+        self._check_bias(bias, x, w)
         bf16 = x.dtype == torch.bfloat16
         small = bf16 and self.use_tc_gemm and M <= self.tc_max_rows and K % 8 == 0
         if add_to is not None:
@@ -366,29 +396,35 @@ class CudaKernels:
             if tuple(add_to.shape) != (M, N):
                 raise KernelError(f"linear: add_to is {list(add_to.shape)}, the product is [{M}, {N}]")
             if small:
-                self.linear_tc(x, w, out=add_to, accumulate=True)
+                self.linear_tc(x, w, out=add_to, accumulate=True, bias=bias)
             elif bf16 and self.use_cublas and add_to.is_contiguous():
                 self.launches += 1
-                self._pending_add = (add_to, torch.nn.functional.linear(x, w))  # added by the norm that follows, or by flush()
+                self._pending_add = (add_to, torch.nn.functional.linear(x, w, bias))  # added by the norm that follows, or by flush()
             else:
-                self._check(self.lib.llmie_gemm_simt(_ptr(x), _ptr(w), _ptr(add_to), M, N, K, self._dt(x, "x"), 0, 1, self._stream()),
+                self._check(self.lib.llmie_gemm_simt(_ptr(x), _ptr(w), _ptr(add_to), M, N, K, self._dt(x, "x"), 0, 1, _ptr(bias), self._stream()),
                             "linear (accumulate)")
             return None
         out_dtype = out_dtype or x.dtype
         if small and transient:
-            return self.linear_tc(x, w, out=self._transient(M, N, w.device), accumulate=True)
+            return self.linear_tc(x, w, out=self._transient(M, N, w.device), accumulate=True, bias=bias)
         if small and out_dtype == torch.float32:
-            return self.linear_tc(x, w)
+            return self.linear_tc(x, w, bias=bias)
         if bf16 and out_dtype == torch.float32 and self.use_tc_gemm and K % 8 == 0 and N <= 128:
             # few outputs in 32-bit for many rows (a router's logits over a prompt portion): one tile of weight rows, a block per 64 rows
-            return self.linear_tc(x, w)
+            return self.linear_tc(x, w, bias=bias)
         if self.use_cublas and bf16 and out_dtype == torch.bfloat16:
             self.launches += 1
-            return torch.nn.functional.linear(x, w)
+            return torch.nn.functional.linear(x, w, bias)
         out = torch.empty((M, N), dtype=out_dtype, device=x.device)
         self._check(self.lib.llmie_gemm_simt(_ptr(x), _ptr(w), _ptr(out), M, N, K, self._dt(x, "x"), self._dt(out, "out"), 0,
-                                             self._stream()), "linear")
+                                             _ptr(bias), self._stream()), "linear")
         return out
+
+    def _check_bias(self, bias, x, w) -> None:
+        if bias is not None:
+            self._need(bias, "bias", x.dtype, 1)
+            if bias.shape[0] != w.shape[0]:
+                raise KernelError(f"linear: the bias has {bias.shape[0]} entries, w has {w.shape[0]} outputs")
 
     def _is_transient(self, t: torch.Tensor) -> bool:
         return self._acc is not None and t.dtype == torch.float32 and t.untyped_storage().data_ptr() == self._acc.untyped_storage().data_ptr()
@@ -403,7 +439,7 @@ class CudaKernels:
         cap = max(1, (4 << 20) // max(1, M * N))
         return max(1, min(want, nkb, cap))
 
-    def linear_tc(self, x, w, out=None, accumulate=False, k_splits=None):
+    def linear_tc(self, x, w, out=None, accumulate=False, k_splits=None, bias=None):
         """``out (+)= x w^T`` in float32 from bfloat16 operands on the tcgen05 tensor cores, for small batches.
         ``accumulate`` adds into ``out`` (which may be a strided view, e.g. the residual stream) atomically."""
         self._need(w, "w", torch.bfloat16, 2)
@@ -424,7 +460,7 @@ class CudaKernels:
             k_splits = self.tc_splits(M, N, K) if accumulate else 1
         self._need(x, "x", torch.bfloat16, 2)
         rc = self.lib.llmie_gemm_tc(_ptr(x), _ptr(w), _ptr(out), out.stride(0), M, N, K, int(k_splits), int(bool(accumulate)),
-                                    _ptr(self._error_flag), self._stream())
+                                    _ptr(self._error_flag), _ptr(bias), self._stream())
         self._check(rc, "linear_tc")
         return out
 
@@ -925,23 +961,25 @@ class CudaKernels:
     # ------------------------------------------------------------------ a product with an activation behind it
     def linear_act(self, x, w, activation, out_dtype=None):
         """``act(x w^T)``; the activation is computed in 32-bit on the product's sums where those are at hand (small batches)."""
-        if activation != "gelu_tanh":
+        kinds = {"gelu_tanh": 0, "gelu_erf": 2}
+        if activation not in kinds:
             raise KernelError(f"linear_act: activation '{activation}' is not built")
         out_dtype = out_dtype or x.dtype
         z = self.linear(x, w, transient=True)
         clear = self._is_transient(z)
         out = torch.empty(z.shape, dtype=out_dtype, device=z.device)
-        self._check(self.lib.llmie_act(_ptr(z), _ptr(out), ctypes.c_longlong(z.numel()), 0, int(clear), ctypes.c_float(0.0), self._dt(z, "z"),
+        self._check(self.lib.llmie_act(_ptr(z), _ptr(out), ctypes.c_longlong(z.numel()), kinds[activation], int(clear), ctypes.c_float(0.0), ctypes.c_float(1.0), self._dt(z, "z"),
                                        _DT[out_dtype], self._stream()), "act")
         return out
 
-    def softcap(self, x, cap: float):
-        """``cap * tanh(x / cap)`` of a float32 tensor, element by element."""
+    def softcap(self, x, cap: float, scale: float = 1.0):
+        """``cap * tanh(scale * x / cap)`` of a float32 tensor, element by element; ``cap`` None: ``scale * x``."""
         self._need(x, "x", torch.float32)
-        if not cap > 0:
+        if cap is not None and not cap > 0:
             raise KernelError("softcap: the cap must be positive")
         out = torch.empty_like(x)
-        self._check(self.lib.llmie_act(_ptr(x), _ptr(out), ctypes.c_longlong(x.numel()), 1, 0, ctypes.c_float(cap), 0, 0, self._stream()), "softcap")
+        self._check(self.lib.llmie_act(_ptr(x), _ptr(out), ctypes.c_longlong(x.numel()), 3 if cap is None else 1, 0, ctypes.c_float(cap or 0.0), ctypes.c_float(scale), 0, 0,
+                                       self._stream()), "softcap")
         return out
 
     # ------------------------------------------------------------------ attention with extras
@@ -960,14 +998,19 @@ class CudaKernels:
 
     def attention_ext(self, q, q_col, num_heads, num_kv_heads, head_dim, v_head_dim, k_pool, v_pool, block_table, token_seq, positions,
                       page_size, scale, window, max_context, temp=(0.0, 0), rel=None, rel_rows=None, sink=None, gate=None, gate_col=0,
-                      gate_per_head=False, batch=None, num_splits=None, keep_first=0, chunk=0, softcap=0.0, talk=None):
+                      gate_per_head=False, batch=None, num_splits=None, keep_first=0, chunk=0, softcap=0.0, talk=None,
+                      sigmoid_bias=None, log_distance=None, turn=None):
         """Paged attention with extras: the query heads are columns ``q_col ..`` of ``q``; ``v_pool=None`` reads the values out
         of the key rows (their first ``v_head_dim`` entries); ``temp=(coef, every)`` a query temperature by position;
         ``rel [rows, heads]`` with ``rel_rows`` (distance -> row) a bias by distance; ``sink [heads]`` joins the denominator;
         ``gate`` (columns from ``gate_col`` of a tensor with the tokens' rows) an output gate per head or per element;
         ``keep_first`` keys at the request's start stay visible when the ``window`` has passed them; ``chunk`` > 0 lets a position
         see only the keys of its own run of ``chunk`` positions; ``softcap`` > 0 bounds the scaled scores by ``cap * tanh(s / cap)``;
-        ``talk [heads, heads]`` (float32) mixes the heads' capped scores before mask and softmax, ``score'_h = sum_g talk[h, g] score_g``."""
+        ``talk [heads, heads]`` (float32) mixes the heads' capped scores before mask and softmax, ``score'_h = sum_g talk[h, g] score_g``;
+        ``log_distance = (r1, r2)`` (float32, one number per head each) takes ``r1 ln(1 + r2 (p - j))`` off the scaled score;
+        ``sigmoid_bias [heads]`` (float32): no softmax, a visible key's weight is ``sigmoid(score + bias)``;
+        ``turn = (cos, sin, neighbours)`` with ``[N, v_head_dim / 2]`` tables: every head's result is turned back by these angles (pairs half
+        the values apart, or neighbours), for values that were turned when they were cached."""
         self._need(q, "q", None, 2)
         dt = self._dt(q, "q")
         N = q.shape[0]
@@ -1004,15 +1047,33 @@ class CudaKernels:
             gate_mode = 1 if gate_per_head else 2
             if gate.shape[0] != N or gate_col + (num_heads if gate_per_head else num_heads * v_head_dim) > gate.shape[1]:
                 raise KernelError("attention_ext: the gate columns lie outside the rows")
+        for name, t in (("sigmoid_bias", sigmoid_bias), *((("log_distance", t) for t in log_distance) if log_distance is not None else ())):
+            if t is not None:
+                self._need(t, name, torch.float32, 1)
+                if t.shape[0] != num_heads:
+                    raise KernelError(f"attention_ext: {name} needs one number per head")
+        if sigmoid_bias is not None and sink is not None:
+            raise KernelError("attention_ext: sigmoid weights have no sink")
+        if turn is not None:
+            for name, t in (("turn cos", turn[0]), ("turn sin", turn[1])):
+                self._need(t, name, torch.float32, 2)
+                if v_head_dim % 2 or tuple(t.shape) != (N, v_head_dim // 2):
+                    raise KernelError("attention_ext: the turn's tables must be [tokens, v_head_dim / 2] with v_head_dim even")
+        more = (_ptr(sigmoid_bias), _ptr(log_distance[0] if log_distance is not None else None), _ptr(log_distance[1] if log_distance is not None else None),
+                _ptr(turn[0] if turn is not None else None), _ptr(turn[1] if turn is not None else None), int(bool(turn[2])) if turn is not None else 0)
         out = torch.empty((N, num_heads * v_head_dim), dtype=q.dtype, device=q.device)
         esize = q.element_size()
         if talk is not None:
+            if sigmoid_bias is not None or log_distance is not None or turn is not None:
+                raise KernelError("attention_ext: talking heads are not built together with sigmoid weights, a penalty by distance or turned values")
             return self._attention_talk(q, q_col, num_heads, num_kv_heads, head_dim, v_head_dim, k_pool, v_pool, block_table, token_seq, positions,
                                         page_size, scale, window, max_context, talk, sink, gate, gate_col, gate_mode, keep_first, chunk, softcap,
                                         temp, rel, out, batch)
         max_rows = 0
         tensor_cores = dt == 1 and self.use_mma_attention_ext and batch is not None and (q_col * esize) % 16 == 0 and q.shape[1] % 8 == 0
         masked = bool(keep_first or chunk or softcap)
+        if sigmoid_bias is not None and (masked or rel is not None):
+            tensor_cores = False   # (the tensor-core kernels know sigmoid weights under a causal mask and a window)
         if masked and not self.masked_attention_tensor_cores:
             tensor_cores = False
         if keep_first < 0 or chunk < 0 or softcap < 0 or (keep_first and not window):
@@ -1032,7 +1093,7 @@ class CudaKernels:
                 v_head_dim, page_size, ctypes.c_float(scale), int(window), splits, ctypes.c_float(temp[0]), int(temp[1]), _ptr(rel),
                 _ptr(rel_rows), 0 if rel_rows is None else rel_rows.shape[0], 0 if rel is None else rel.shape[0], _ptr(sink),
                 ctypes.c_void_p(0 if gate is None else gate.data_ptr() + gate_col * esize), 0 if gate is None else gate.shape[1], gate_mode,
-                int(keep_first), int(chunk), ctypes.c_float(softcap), self._stream()), "attention_ext (tensor cores, a warp to a row block)")
+                int(keep_first), int(chunk), ctypes.c_float(softcap), *more, self._stream()), "attention_ext (tensor cores, a warp to a row block)")
             if splits > 1:
                 self.launches += 1
             return out
@@ -1045,7 +1106,7 @@ class CudaKernels:
             group = num_heads // num_kv_heads
             heads_per_tile = min(group, 32)
             tile_rows = 32
-            while tile_rows < min(max_rows, self.attention_ext_tile_rows) and tile_rows < batch.max_seq_len * heads_per_tile:
+            while sigmoid_bias is None and tile_rows < min(max_rows, self.attention_ext_tile_rows) and tile_rows < batch.max_seq_len * heads_per_tile:
                 tile_rows *= 2
             if batch.max_seq_len == 1:
                 tiles, tile_info = N, None
@@ -1061,7 +1122,7 @@ class CudaKernels:
                 head_dim, v_head_dim, page_size, ctypes.c_float(scale), int(window), splits, ctypes.c_float(temp[0]), int(temp[1]), _ptr(rel),
                 _ptr(rel_rows), 0 if rel_rows is None else rel_rows.shape[0], 0 if rel is None else rel.shape[0], _ptr(sink),
                 ctypes.c_void_p(0 if gate is None else gate.data_ptr() + gate_col * esize), 0 if gate is None else gate.shape[1], gate_mode,
-                int(keep_first), int(chunk), ctypes.c_float(softcap), self._stream()), "attention_ext (tensor cores)")
+                int(keep_first), int(chunk), ctypes.c_float(softcap), *more, self._stream()), "attention_ext (tensor cores)")
             if splits > 1:
                 self.launches += 1
             return out
@@ -1075,7 +1136,7 @@ class CudaKernels:
                        ctypes.c_float(temp[0]), int(temp[1]), _ptr(rel), _ptr(rel_rows), 0 if rel_rows is None else rel_rows.shape[0],
                        0 if rel is None else rel.shape[0], _ptr(sink),
                        ctypes.c_void_p(0 if gate is None else gate.data_ptr() + gate_col * esize), 0 if gate is None else gate.shape[1],
-                       gate_mode, int(keep_first), int(chunk), ctypes.c_float(softcap), self._stream()), "attention_ext")
+                       gate_mode, int(keep_first), int(chunk), ctypes.c_float(softcap), *more, self._stream()), "attention_ext")
         if splits > 1:
             self.launches += 1
         return out
@@ -1251,6 +1312,61 @@ class CudaKernels:
         self._need(weight, "weight", torch.float32, 1)
         self._pending_post = (residual, y, weight, 0.0, True)
 
+    # ------------------------------------------------------------------ Dynamic Tanh in place of a norm
+    def _dynamic_tanh(self, x, post, pre, rows, out_dtype, what):
+        """``x += tanh(a y) * w + b`` for ``post = (y, a, w, b)``, then ``tanh(a x) * w + b`` for ``pre = (a, w, b)``; either may be None."""
+        self._need(x, "residual", torch.float32, 2)
+        N, H = x.shape
+        y = None
+        y_dt = 0
+        clear = False
+        if post is not None:
+            y = post[0]
+            self._need(y, "y", None, 2)
+            y_dt = self._dt(y, "y")
+            if tuple(y.shape) != (N, H):
+                raise KernelError(f"{what}: the sublayer's result is {list(y.shape)}, the stream is {list(x.shape)}")
+            clear = self._clears(y)
+        for part in (post[1:] if post is not None else None, pre):
+            if part is not None:
+                for t in part:
+                    self._need(t, "a Dynamic Tanh's tensor", torch.float32)
+                if part[0].numel() != 1 or part[1].numel() != H or part[2].numel() != H:
+                    raise KernelError(f"{what}: a Dynamic Tanh over rows of {H} needs one alpha and {H} weights and biases")
+        if rows is not None:
+            self._need(rows, "rows", torch.int32, 1)
+        n_rows = N if rows is None else rows.shape[0]
+        out = torch.empty((n_rows, H), dtype=out_dtype, device=x.device) if pre is not None else None
+        out_dt = _DT[out_dtype] if pre is not None else y_dt
+        fast = y_dt == 1 or out_dt == 1
+        pa, pw, pb = post[1:] if post is not None else (None, None, None)
+        qa, qw, qb = pre if pre is not None else (None, None, None)
+        self._check(self.lib.llmie_dynamic_tanh(_ptr(x), _ptr(y), y_dt, _ptr(pa), _ptr(pw), _ptr(pb), int(clear), _ptr(qa), _ptr(qw), _ptr(qb), _ptr(out),
+                                                out_dt, _ptr(rows), n_rows, H, int(fast), 12 * self.num_sms, self._stream()), what)
+        if clear and rows is not None:
+            y.zero_()   # only the chosen rows were read; the buffer must be zero for its next user
+            self.launches += 1
+        return out
+
+    def dynamic_tanh(self, residual, alpha, weight, bias, out_dtype, rows=None):
+        """``tanh(alpha x) * weight + bias`` of the stream's rows (or of ``rows``), in ``out_dtype``; ``alpha`` is one number on the device.
+        A sublayer's result whose own closing Dynamic Tanh still waits (``post_tanh_add``) is added by the same kernel."""
+        post = None
+        if (self._pending_tanh is not None and self._pending_tanh[0] is residual and self._pending_add is None and self._pending_streams is None
+                and self._pending_post is None):
+            post, self._pending_tanh = self._pending_tanh[1:], None
+        else:
+            self.flush()
+        return self._dynamic_tanh(residual, post, (alpha, weight, bias), rows, out_dtype, "dynamic_tanh")
+
+    def post_tanh_add(self, residual, y, alpha, weight, bias):
+        """``residual += tanh(alpha y) * weight + bias``: put off until the next ``dynamic_tanh`` of the same stream (one pass does both) or
+        until ``flush``. ``y`` is a zeroed tensor of ``zeros_like_rows`` that the sublayer added its result into."""
+        y = self.take_result(y)
+        if self._pending_tanh is not None:
+            self.flush()
+        self._pending_tanh = (residual, y, alpha, weight, bias)
+
     def group_rmsnorm_gate(self, x, gate, gate_col, weight, group_size, eps, gate_first, out_dtype, gate_act="sigmoid"):
         """Float32 rows ``x [N, C]`` normed by their root mean square in groups of ``group_size`` channels, with a gate read
         from columns ``gate_col ..`` of ``gate``: ``gate_first`` multiplies by ``silu(gate)`` before the norm, otherwise by
@@ -1315,10 +1431,12 @@ class CudaKernels:
 
     # ------------------------------------------------------------------ heads normed and partly rotated on their way to the cache
     def qk_norm_rope_store(self, z, num_heads, num_kv_heads, head_dim, v_head_dim, q_weight, k_weight, eps, cos, sin, rot_dims, interleaved,
-                           slot_mapping, k_pool, v_pool, page_size, write_kv=True):
+                           slot_mapping, k_pool, v_pool, page_size, write_kv=True, v_turn=None, out_dtype=None):
         """From rows ``z = [query heads | key heads | value heads]``: per query and key head an optional RMS norm with a weight,
         then the rotation of its first ``rot_dims`` entries (pairs ``(i, i + rot_dims/2)``, or neighbours when ``interleaved``);
-        returns the query heads ``[N, heads * head_dim]`` and puts keys and values into the tokens' cache slots."""
+        returns the query heads ``[N, heads * head_dim]`` and puts keys and values into the tokens' cache slots. ``v_turn = (cos, sin)`` of
+        ``[N, v_head_dim / 2]``: the values turn too, over all their entries. ``z`` may be a product's transient float32 sums
+        (``linear(transient=True)``), which are consumed and cleared."""
         self._need(z, "z", None, 2)
         N = z.shape[0]
         if z.shape[1] < (num_heads + num_kv_heads) * head_dim + num_kv_heads * v_head_dim:
@@ -1333,17 +1451,25 @@ class CudaKernels:
                 self._need(t, name, torch.float32, 1)
                 if t.shape[0] != head_dim:
                     raise KernelError(f"qk_norm_rope_store: {name} needs one entry per element of a head")
+        if v_turn is not None:
+            for t in v_turn:
+                self._need(t, "v_turn", torch.float32, 2)
+                if v_head_dim % 2 or tuple(t.shape) != (N, v_head_dim // 2):
+                    raise KernelError("qk_norm_rope_store: the values' tables must be [tokens, v_head_dim / 2] with v_head_dim even")
+        out_dtype = out_dtype or z.dtype
+        clear = self._is_transient(z)
         if write_kv:
             self._need(slot_mapping, "slot_mapping", torch.int32, 1)
             for name, pool, d in (("k_pool", k_pool, head_dim), ("v_pool", v_pool, v_head_dim)):
-                self._need(pool, name, z.dtype, 4)
+                self._need(pool, name, out_dtype, 4)
                 if tuple(pool.shape[1:]) != (num_kv_heads, page_size, d):
                     raise KernelError(f"qk_norm_rope_store: {name} is {list(pool.shape)}, expected [pages, {num_kv_heads}, {page_size}, {d}]")
-        q = torch.empty((N, num_heads * head_dim), dtype=z.dtype, device=z.device)
+        q = torch.empty((N, num_heads * head_dim), dtype=out_dtype, device=z.device)
         self._check(self.lib.llmie_qk_norm_rope_store(_ptr(z), z.shape[1], _ptr(q), _ptr(q_weight), _ptr(k_weight), ctypes.c_float(eps), _ptr(cos if rot_dims else None),
-                                                      _ptr(sin if rot_dims else None), int(rot_dims), int(bool(interleaved)), _ptr(slot_mapping if write_kv else None),
+                                                      _ptr(sin if rot_dims else None), int(rot_dims), int(bool(interleaved)), _ptr(v_turn[0] if v_turn is not None else None),
+                                                      _ptr(v_turn[1] if v_turn is not None else None), _ptr(slot_mapping if write_kv else None),
                                                       _ptr(k_pool if write_kv else None), _ptr(v_pool if write_kv else None), N, num_heads, num_kv_heads, head_dim,
-                                                      v_head_dim, page_size, int(bool(write_kv)), self._dt(z, "z"), self._stream()), "qk_norm_rope_store")
+                                                      v_head_dim, page_size, int(bool(write_kv)), int(clear), self._dt(z, "z"), _DT[out_dtype], self._stream()), "qk_norm_rope_store")
         return q
 
     # ------------------------------------------------------------------ mixers with a state of fixed size

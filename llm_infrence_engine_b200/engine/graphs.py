@@ -128,6 +128,9 @@ class DecodeGraphs:
     def _capture_context(self, ctx: StepContext, rows: torch.Tensor) -> _Captured:
         """Warm up, then capture ``forward`` on a context whose tensors are views of a static buffer."""
         r = self.runner
+        # the warm-up runs the step on the requests' own states of fixed size, which the replay must find as they were before it
+        slots = torch.tensor(ctx.seq_slot_list, dtype=torch.long, device=r.device)
+        held = [b.state.index_select(0, slots) for b in r.all_states]
         side = torch.cuda.Stream()
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):
@@ -135,6 +138,8 @@ class DecodeGraphs:
             r.forward(ctx, rows)  # once outside the capture: whatever this shape allocates or sets up for the first time
         torch.cuda.current_stream().wait_stream(side)
         torch.cuda.synchronize()
+        for b, rows_before in zip(r.all_states, held):
+            b.state.index_copy_(0, slots, rows_before)
         ctx._tables.clear()
         before = r.K.launches
         graph, logits = self._record(lambda: r.forward(ctx, rows))

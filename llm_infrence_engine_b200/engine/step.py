@@ -107,7 +107,8 @@ class ModelRunner:
         self.bindings: List[object] = []
         self.kv_bytes_per_token = 0
         specs = spec.cache_specs()
-        self.state_bindings: List[StateBinding] = []   # every fixed-size state of the model, wherever it is bound
+        self.all_states: List[StateBinding] = []       # every fixed-size state of the model
+        self.state_bindings: List[StateBinding] = []   # ... those that start from zero
 
         def bind(entry, cs, group):
             """The binding of one spec; a tuple of specs (a mixer that asks for several things) gives a tuple of bindings."""
@@ -121,7 +122,9 @@ class ModelRunner:
                 return PagedKVBinding(group, k, v)
             if isinstance(cs, FixedStateSpec):
                 b = StateBinding(torch.zeros((max_seqs + 1,) + tuple(cs.shape), dtype=torch.float32, device=self.device))
-                self.state_bindings.append(b)
+                self.all_states.append(b)
+                if cs.zeroed:
+                    self.state_bindings.append(b)
                 return b
             if cs is None:
                 return None
@@ -397,7 +400,10 @@ class ModelRunner:
         else:
             for b in self.state_bindings:
                 self.K.zero_fresh_state(b.state, ctx.seq_slots, ctx.seq_starts_dev, ctx.positions)
-        residual = spec.embedding.forward(ctx)
+        if spec.embedding.cache_spec() is not None:
+            residual = spec.embedding.forward(ctx, self.bindings[-1])
+        else:
+            residual = spec.embedding.forward(ctx)
         if spec.streams is not None:   # several residual streams: the layers work on [N, streams, hidden]
             residual = spec.streams.expand(ctx, residual)
         for call in spec.schedule:

@@ -59,6 +59,9 @@ class ModelSpec:
                     raise ValueError(f"cache entry {call.cache} is read but no call writes it")
                 if self.layers[call.layer].cache_spec() != specs[call.cache]:
                     raise ValueError(f"layer {call.layer} reads cache entry {call.cache} of another shape")
+        own = self.embedding.cache_spec()
+        if own is not None:   # what the embedding keeps per request lies behind the layers' entries
+            specs.append(own)
         return specs
 
     def vocab_size(self) -> int:

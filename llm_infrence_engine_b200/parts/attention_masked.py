@@ -6,13 +6,13 @@ from typing import Dict, Optional
 import torch
 
 from ..cache.spec import FixedStateSpec, PagedKVSpec
-from .base import INIT_EYE, INIT_NORM, INIT_PROJ, INIT_SMALL, INIT_TAPS, MATRIX, VECTOR, Mixer, ParamSpec, PositionEncoding, Source
+from .base import INIT_EYE, INIT_NORM, INIT_PROJ, INIT_RATE, INIT_SMALL, INIT_TAPS, MATRIX, VECTOR, Mixer, ParamSpec, PositionEncoding, Source
 
 
 class MaskedAttention(Mixer):
     """``o(softmax(cap(scale * q k^T) + mask) v)`` over a paged cache, ``num_heads`` query heads sharing ``num_kv_heads``
-    key/value heads (query head ``h`` reads key/value head ``h // (num_heads // num_kv_heads)``), no biases. Options, each off
-    unless asked for:
+    key/value heads (query head ``h`` reads key/value head ``h // (num_heads // num_kv_heads)``). Options, each off unless asked
+    for:
 
     * ``conv_taps``: a short causal convolution per channel on q, k and v right after their projection (no bias, no
       activation); a request's last ``conv_taps - 1`` projected rows are part of its state;
@@ -27,7 +27,12 @@ class MaskedAttention(Mixer):
       ``score'_h = sum_g talk[h, g] score_g`` with ``talk [heads, heads]`` (``{prefix}.talk``);
     * ``sink``: a learned number per head (``{prefix}.sink``) whose exponential joins the softmax's denominator once: it has no key and
       no value and is neither scaled nor capped nor mixed;
-    * ``head_gate``: head h's result is multiplied by ``sigmoid(W_g x)_h`` (``{prefix}.g``, one row per head, read from the mixer's input).
+    * ``head_gate``: head h's result is multiplied by ``sigmoid(W_g x)_h`` (``{prefix}.g``, one row per head, read from the mixer's input);
+    * ``bias``: q, k, v and the output projection have biases (``{prefix}.q.b`` and so on);
+    * ``value_position``: a rotary encoding over all ``v_head_dim`` entries of a value: the value of position j turns by j's angles and is
+      cached so; every head's result at position i turns back by i's angles, so that the result knows distances (pairs as for q and k);
+    * ``log_distance``: ``r1_h ln(1 + r2_h (i - j))`` is taken off head h's scaled score (``{prefix}.r1``, ``{prefix}.r2``);
+    * ``scoring = "sigmoid"``: no softmax; a visible key's weight is ``sigmoid(score + pb_h)`` (``{prefix}.pb``), not normalised over keys.
 
     The three projections are one matrix; norm, rotation and the cache write are one kernel; the mask is never a tensor.
     Pages that neither window nor chunk can reach any more go back to the pool as a request moves on.
@@ -38,7 +43,8 @@ class MaskedAttention(Mixer):
     def __init__(self, hidden: int, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int, scale: float, prefix: str,
                  position: Optional[PositionEncoding] = None, interleaved: bool = False, window: Optional[int] = None, keep_first: int = 0,
                  chunk: Optional[int] = None, softcap: Optional[float] = None, conv_taps: int = 0, qk_norm: bool = False, eps: float = 1e-6,
-                 talking_heads: bool = False, sink: bool = False, head_gate: bool = False):
+                 talking_heads: bool = False, sink: bool = False, head_gate: bool = False, bias: bool = False,
+                 value_position: Optional[PositionEncoding] = None, log_distance: bool = False, scoring: str = "softmax"):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads cannot share {num_kv_heads} key/value heads")
         if keep_first and not window:
@@ -55,6 +61,20 @@ class MaskedAttention(Mixer):
         self.conv_taps, self.qk_norm, self.eps = int(conv_taps), bool(qk_norm), float(eps)
         self.channels = (num_heads + num_kv_heads) * head_dim + num_kv_heads * v_head_dim
         self.talking_heads, self.has_sink, self.head_gate = bool(talking_heads), bool(sink), bool(head_gate)
+        if scoring not in ("softmax", "sigmoid"):
+            raise ValueError(f"scoring '{scoring}' is not 'softmax' or 'sigmoid'")
+        if scoring == "sigmoid" and sink:
+            raise ValueError("weights without a softmax have no denominator that a sink could join")
+        if value_position is not None and value_position.dims != v_head_dim:
+            raise ValueError(f"values of {v_head_dim} entries turn as a whole, not in {value_position.dims} of them")
+        if conv_taps and (bias or value_position is not None):
+            raise ValueError("biases and turned values are not built together with short convolutions")
+        self.has_bias, self.value_position, self.log_distance, self.scoring = bool(bias), value_position, bool(log_distance), scoring
+        self.b_qkv: Optional[torch.Tensor] = None
+        self.b_o: Optional[torch.Tensor] = None
+        self.r1: Optional[torch.Tensor] = None
+        self.r2: Optional[torch.Tensor] = None
+        self.pb: Optional[torch.Tensor] = None
         self.talk: Optional[torch.Tensor] = None
         self.sink: Optional[torch.Tensor] = None
         self.w_qkv: Optional[torch.Tensor] = None
@@ -73,6 +93,16 @@ class MaskedAttention(Mixer):
             joined += (Source(f"{p}.g", (self.num_heads, h), INIT_PROJ),)
         out = {"w_qkv": ParamSpec(joined, MATRIX),
                "w_o": ParamSpec((Source(f"{p}.o", (h, self.num_heads * self.v_head_dim), INIT_PROJ),), MATRIX)}
+        if self.has_bias:   # (biases are kept in the type of the products they are added to)
+            if self.head_gate:
+                raise ValueError("biases are not built together with a gate per head")
+            out["b_qkv"] = ParamSpec(tuple(Source(f"{p}.{n}.b", (r,), INIT_SMALL) for n, r in self._rows()), MATRIX)
+            out["b_o"] = ParamSpec((Source(f"{p}.o.b", (h,), INIT_SMALL),), MATRIX)
+        if self.log_distance:
+            out["r1"] = ParamSpec((Source(f"{p}.r1", (self.num_heads,), INIT_RATE),), VECTOR)
+            out["r2"] = ParamSpec((Source(f"{p}.r2", (self.num_heads,), INIT_RATE),), VECTOR)
+        if self.scoring == "sigmoid":
+            out["pb"] = ParamSpec((Source(f"{p}.pb", (self.num_heads,), INIT_SMALL),), VECTOR)
         if self.talking_heads:
             out["talk"] = ParamSpec((Source(f"{p}.talk", (self.num_heads, self.num_heads), INIT_EYE),), VECTOR)
         if self.has_sink:
@@ -89,6 +119,8 @@ class MaskedAttention(Mixer):
         pad = -self.w_qkv.shape[0] % 8   # (rows of the product that start on a 16-byte boundary)
         if pad:
             self.w_qkv = torch.cat([self.w_qkv, self.w_qkv.new_zeros((pad, self.w_qkv.shape[1]))]).contiguous()
+            if self.b_qkv is not None:
+                self.b_qkv = torch.cat([self.b_qkv, self.b_qkv.new_zeros(pad)]).contiguous()
 
     def cache_spec(self):
         pages = PagedKVSpec(self.num_kv_heads, self.head_dim, self.window, self.v_head_dim, self.keep_first, self.chunk)
@@ -99,7 +131,11 @@ class MaskedAttention(Mixer):
     def forward(self, ctx, h, cache, residual):
         K = ctx.K
         kv, conv_state = cache if self.conv_taps else (cache, None)
-        z = K.linear(h, self.w_qkv, out_dtype=ctx.dtype)
+        # where nothing else reads the projections, a small batch leaves its float32 sums to the kernel that turns and stores them
+        more = {"transient": True} if not (self.head_gate or self.conv_taps) else {}
+        if self.has_bias:
+            more["bias"] = self.b_qkv
+        z = K.linear(h, self.w_qkv, out_dtype=ctx.dtype, **more)
         gate = z if self.head_gate else None   # (its columns lie behind the heads, from ``channels`` on)
         if self.conv_taps:
             z = K.causal_conv(z, 0, self.channels, self.conv_w, None, conv_state.state, ctx)
@@ -108,10 +144,22 @@ class MaskedAttention(Mixer):
         if self.position is not None:
             cos, sin = ctx.position_tables(self.position)
             dims = self.position.dims
+        v_turn = ctx.position_tables(self.value_position) if self.value_position is not None else None
         q = K.qk_norm_rope_store(z, self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim, self.q_norm, self.k_norm, self.eps, cos, sin,
-                                 dims, self.interleaved, ctx.slot_mapping[kv.group], kv.k, kv.v, ctx.page_size, write_kv=kv.write)
+                                 dims, self.interleaved, ctx.slot_mapping[kv.group], kv.k, kv.v, ctx.page_size, write_kv=kv.write,
+                                 out_dtype=ctx.dtype, **({"v_turn": v_turn} if v_turn is not None else {}))
+        more = {}
+        if v_turn is not None:
+            more["turn"] = (*v_turn, self.interleaved)
+        if self.log_distance:
+            more["log_distance"] = (self.r1, self.r2)
+        if self.scoring == "sigmoid":
+            more["sigmoid_bias"] = self.pb
         attn = K.attention_ext(q, 0, self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim, kv.k, kv.v, ctx.block_tables[kv.group],
                                ctx.token_seq, ctx.positions, ctx.page_size, self.scale, self.window or 0, ctx.max_context, batch=ctx,
                                keep_first=self.keep_first, chunk=self.chunk or 0, softcap=self.softcap, sink=self.sink, gate=gate,
-                               gate_col=self.channels, gate_per_head=True, talk=self.talk)
-        K.linear(attn, self.w_o, add_to=residual)
+                               gate_col=self.channels, gate_per_head=True, talk=self.talk, **more)
+        if self.has_bias:
+            K.linear(attn, self.w_o, add_to=residual, bias=self.b_o)
+        else:
+            K.linear(attn, self.w_o, add_to=residual)

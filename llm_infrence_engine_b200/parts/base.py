@@ -39,6 +39,7 @@ INIT_EYE = "eye"            # identity + N(0, 0.05): how the residual streams mi
 INIT_LOG_RATE = "log_rate"  # ln U(0.5, 4): the logarithm of a decay rate
 INIT_STEP_BIAS = "step_bias"  # softplus^-1 of a step size drawn log-uniformly from 0.01 to 0.3
 INIT_TAPS = "taps"          # N(0, 0.3): the few taps of a short convolution
+INIT_RATE = "rate"          # U(0.2, 1.5): a rate that must be positive
 INIT_PROJ = "projection"    # N(0, 1 / sqrt(columns)): a matrix whose product keeps its input's scale
 
 ANY = -1  # a dimension of a Source's shape that the checkpoint decides (the part reads it off the tensor it is given)

@@ -5,6 +5,7 @@ from typing import Dict, Optional
 
 import torch
 
+from ..cache.spec import FixedStateSpec
 from .base import MATRIX, ParamSpec, Part, Source
 
 
@@ -21,7 +22,11 @@ class TokenEmbedding(Part):
     def params(self) -> Dict[str, ParamSpec]:
         return {"table": ParamSpec((Source(self.name, (self.vocab, self.hidden)),), MATRIX)}
 
-    def forward(self, ctx) -> torch.Tensor:
+    def cache_spec(self):
+        """What the embedding keeps per request (as a mixer's ``cache_spec``); nothing here."""
+        return None
+
+    def forward(self, ctx, cache=None) -> torch.Tensor:
         if self.scale == 1.0:
             return ctx.K.embed(ctx.token_ids, self.table)
         return ctx.K.embed(ctx.token_ids, self.table, self.scale)
@@ -31,16 +36,44 @@ class TokenEmbedding(Part):
         ctx.K.embed_add(ctx.token_ids, self.table, residual, self.scale)
 
 
+class BigramEmbedding(TokenEmbedding):
+    """``x = table[token] * scale + bigram[(previous * mul_prev + token * mul_cur) mod buckets]``; a request's first token, which has no
+    previous one, takes the bigram table's last row, number ``buckets``. A request's last token is its state: a portion may
+    start anywhere, and a decoded token may be known to the device alone."""
+
+    def __init__(self, vocab: int, hidden: int, name: str, bigram_name: str, buckets: int, mul_prev: int, mul_cur: int, scale: float = 1.0):
+        super().__init__(vocab, hidden, name, scale)
+        if buckets < 1:
+            raise ValueError(f"a bigram table needs at least one bucket, got {buckets}")
+        self.bigram_name, self.buckets, self.mul_prev, self.mul_cur = bigram_name, int(buckets), int(mul_prev), int(mul_cur)
+        self.bigram: Optional[torch.Tensor] = None
+
+    def params(self) -> Dict[str, ParamSpec]:
+        return {**super().params(), "bigram": ParamSpec((Source(self.bigram_name, (self.buckets + 1, self.hidden)),), MATRIX)}
+
+    def cache_spec(self):
+        return FixedStateSpec((1,), zeroed=False)
+
+    def forward(self, ctx, cache=None) -> torch.Tensor:
+        return ctx.K.embed_bigram(ctx.token_ids, self.table, self.bigram, self.buckets, self.mul_prev, self.mul_cur, ctx.positions, ctx.token_seq,
+                                  ctx.seq_starts_dev, ctx.num_seqs, cache.state.view(torch.int32), self.scale)
+
+    def add_into(self, ctx, residual: torch.Tensor) -> None:
+        raise ValueError("a bigram embedding is not fed in again on the way")
+
+
 class OutputHead(Part):
     """``logits = h W^T`` without bias, in 32-bit. ``tied_to`` makes ``W`` the embedding's own table
-    (src/miniserve/model.py:204-206); a tensor of the head's name in the checkpoint is then not needed. ``softcap`` bounds the
-    logits: ``softcap * tanh(logits / softcap)``."""
+    (src/miniserve/model.py:204-206); a tensor of the head's name in the checkpoint is then not needed. The logits are multiplied by
+    ``scale``; ``softcap`` then bounds them: ``softcap * tanh(logits / softcap)``."""
 
     graph_safe = True
 
-    def __init__(self, vocab: int, hidden: int, name: str, tied_to: Optional[TokenEmbedding] = None, softcap: Optional[float] = None):
+    def __init__(self, vocab: int, hidden: int, name: str, tied_to: Optional[TokenEmbedding] = None, softcap: Optional[float] = None,
+                 scale: float = 1.0):
         self.vocab, self.hidden, self.name, self.tied_to = vocab, hidden, name, tied_to
         self.softcap = float(softcap) if softcap else None
+        self.scale = float(scale)
         self.weight: Optional[torch.Tensor] = None
 
     def params(self) -> Dict[str, ParamSpec]:
@@ -61,4 +94,6 @@ class OutputHead(Part):
 
     def forward(self, ctx, h: torch.Tensor) -> torch.Tensor:
         logits = ctx.K.linear(h, self.matrix(), out_dtype=torch.float32)
+        if self.scale != 1.0:
+            return ctx.K.softcap(logits, self.softcap, self.scale)
         return ctx.K.softcap(logits, self.softcap) if self.softcap else logits

@@ -41,10 +41,11 @@ class GatedMLP(FeedForward):
 
 class DenseMLP(FeedForward):
     """``down(act(up(x)))`` without biases; ``act`` is the tanh form of GELU,
-    ``0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))``, computed in 32-bit on the product's sums."""
+    ``0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))``, or the exact one (``gelu_erf``), ``0.5 z (1 + erf(z / sqrt(2)))``, computed in
+    32-bit on the product's sums."""
 
     graph_safe = True
-    ACTIVATIONS = ("gelu_tanh",)
+    ACTIVATIONS = ("gelu_tanh", "gelu_erf")
 
     def __init__(self, hidden: int, intermediate: int, up_name: str, down_name: str, activation: str = "gelu_tanh"):
         if activation not in self.ACTIVATIONS:

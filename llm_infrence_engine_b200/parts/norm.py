@@ -1,11 +1,11 @@
-"""Normalisation of rows of the 32-bit residual stream: root mean square, and layer norm with a weight."""
+"""Normalisation of rows of the 32-bit residual stream: root mean square, layer norm with a weight, and Dynamic Tanh in a norm's place."""
 from __future__ import annotations
 
 from typing import Dict, Optional
 
 import torch
 
-from .base import INIT_NORM, INIT_SMALL, VECTOR, Norm, ParamSpec, Source
+from .base import INIT_NORM, INIT_ONES, INIT_SMALL, VECTOR, Norm, ParamSpec, Source
 
 
 class RMSNorm(Norm):
@@ -82,3 +82,36 @@ class LayerNorm(Norm):
         if self.bias is not None:
             raise ValueError("a layer norm with a bias does not close a sublayer here")
         ctx.K.post_norm_add(residual, y, self.weight, self.eps)
+
+
+class DynamicTanh(Norm):
+    """``y = tanh(alpha x) * weight + bias``, element by element, with one number ``alpha``: it stands where a norm would and computes no
+    mean or variance. In 32-bit up to the one rounding of the result. Tensors: the weight's name, ``<name>.b`` and ``<name>.alpha``
+    (a scalar).
+
+    It closes a sublayer too: ``add_normed(ctx, residual, y)`` is ``residual += tanh(alpha y) * weight + bias``, put off until the next
+    Dynamic Tanh of the stream, whose kernel does both in one pass.
+    """
+
+    graph_safe = True
+
+    def __init__(self, dim: int, weight_name: str):
+        self.dim, self.weight_name = dim, weight_name
+        self.weight: Optional[torch.Tensor] = None
+        self.bias: Optional[torch.Tensor] = None
+        self.alpha: Optional[torch.Tensor] = None
+
+    def params(self) -> Dict[str, ParamSpec]:
+        n = self.weight_name
+        return {"weight": ParamSpec((Source(n, (self.dim,), INIT_NORM),), VECTOR),
+                "bias": ParamSpec((Source(f"{n}.b", (self.dim,), INIT_SMALL),), VECTOR),
+                "alpha": ParamSpec((Source(f"{n}.alpha", (), INIT_ONES),), VECTOR)}
+
+    def norm(self, ctx, residual):
+        return ctx.K.dynamic_tanh(residual, self.alpha, self.weight, self.bias, ctx.dtype)
+
+    def norm_rows(self, ctx, residual, rows):
+        return ctx.K.dynamic_tanh(residual, self.alpha, self.weight, self.bias, ctx.dtype, rows)
+
+    def add_normed(self, ctx, residual, y) -> None:
+        ctx.K.post_tanh_add(residual, y, self.alpha, self.weight, self.bias)

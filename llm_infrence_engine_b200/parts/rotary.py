@@ -41,6 +41,35 @@ class RotaryEncoding(PositionEncoding):
         return ctx.K.rope_tables(ctx.positions, self.inv_freq(ctx.device))
 
 
+class LinearRotary(PositionEncoding):
+    """Rotation angles ``position * base^(-2i/dims) / factor`` for ``i < dims / 2``: every frequency slowed down by one factor (1: plain
+    rotary positions). The frequencies are made once, in 64-bit, and rounded to 32-bit; the angles are 32-bit products. Which
+    entries of a head form a pair is the mixer's business, not the table's.
+    """
+
+    graph_safe = True
+
+    def __init__(self, dims: int, base: float, factor: float = 1.0):
+        if dims <= 0 or dims % 2:
+            raise ValueError(f"the rotated dimensions must be even and positive, got {dims}")
+        self.dims, self.base, self.factor = int(dims), float(base), float(factor)
+        self._inv_freq = {}
+
+    def key(self) -> tuple:
+        return ("linear-rotary", self.dims, self.base, self.factor)
+
+    def inv_freq(self, device) -> torch.Tensor:
+        dev = str(device)
+        if dev not in self._inv_freq:
+            f = [self.base ** (-2.0 * i / self.dims) / self.factor for i in range(self.dims // 2)]
+            self._inv_freq[dev] = torch.tensor(f, dtype=torch.float64).to(torch.float32).to(device)
+        return self._inv_freq[dev]
+
+    def tables(self, ctx):
+        """(cos, sin), each ``[N, dims / 2]`` in 32-bit."""
+        return ctx.K.rope_tables(ctx.positions, self.inv_freq(ctx.device))
+
+
 class RampedRotary(PositionEncoding):
     """Rotation angles ``position * f_i`` for ``i < dims / 2`` whose frequencies are stretched by wavelength (the scheme known
     as YaRN): with ``f_i = base^(-2i/dims)``, ``d(t) = dims ln(original / (2 pi t)) / (2 ln base)``, ``lo = max(floor(d(fast)), 0)``,

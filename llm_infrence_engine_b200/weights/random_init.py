@@ -15,7 +15,7 @@ from typing import Any, Dict, Mapping
 import torch
 
 from ..models.registry import build_model_spec
-from ..parts.base import (INIT_EYE, INIT_LOG_RATE, INIT_NORM, INIT_NORMAL, INIT_ONES, INIT_PROJ, INIT_SHARE, INIT_SMALL, INIT_STEP_BIAS,
+from ..parts.base import (INIT_EYE, INIT_LOG_RATE, INIT_NORM, INIT_NORMAL, INIT_ONES, INIT_PROJ, INIT_RATE, INIT_SHARE, INIT_SMALL, INIT_STEP_BIAS,
                           INIT_TAPS)
 from .safetensors_io import write_safetensors_stream
 
@@ -55,6 +55,8 @@ def _draw(s, gen: torch.Generator, std: float) -> torch.Tensor:
         return step + torch.log(-torch.expm1(-step))
     if s.init == INIT_TAPS:
         return torch.randn(shape, generator=gen) * 0.3
+    if s.init == INIT_RATE:
+        return 0.2 + 1.3 * torch.rand(shape, generator=gen)
     if s.init == INIT_PROJ:
         return torch.randn(shape, generator=gen) / math.sqrt(shape[-1])
     raise ValueError(f"tensor '{s.name}' asks for unknown initialisation '{s.init}'")

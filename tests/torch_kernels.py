@@ -23,6 +23,21 @@ class TorchKernels:
     def embed(self, token_ids, table, scale=1.0):
         return table[token_ids.long()].float() * scale
 
+    def embed_bigram(self, token_ids, table, bigram, buckets, mul_prev, mul_cur, positions, token_seq, seq_starts, num_seqs, last, scale=1.0):
+        out = table[token_ids.long()].float() * scale
+        for r in range(num_seqs):
+            a, b = int(seq_starts[r]), int(seq_starts[r + 1])
+            slot = int(token_seq[a])
+            for n in range(a, b):
+                if int(positions[n]) == 0:
+                    row = buckets
+                else:
+                    previous = int(last[slot]) if n == a else int(token_ids[n - 1])
+                    row = (previous * mul_prev + int(token_ids[n]) * mul_cur) % buckets
+                out[n] += bigram[row].float()
+            last[slot] = token_ids[b - 1]
+        return out
+
     def embed_add(self, token_ids, table, residual, scale=1.0):
         residual += table[token_ids.long()].float() * scale
 
@@ -55,7 +70,13 @@ class TorchKernels:
         h = x * torch.rsqrt(x.pow(2).mean(-1, keepdim=True) + eps)
         return (weight.float() * h.to(out_dtype).float()).to(out_dtype)
 
-    def linear(self, x, w, out_dtype=None, add_to=None, transient=False):
+    def linear(self, x, w, out_dtype=None, add_to=None, transient=False, bias=None):
+        if bias is not None:
+            y = x.float() @ w.float().T + bias.float()
+            if add_to is None:
+                return y.to(out_dtype or x.dtype)
+            add_to += y
+            return None
         y = x.float() @ w.float().T
         if add_to is not None:
             add_to += y
@@ -159,6 +180,8 @@ class TorchKernels:
     # ------------------------------------------------------------------ feed-forward with one product going in
     def linear_act(self, x, w, activation, out_dtype=None):
         z = x.float() @ w.float().T
+        if activation == "gelu_erf":
+            return (0.5 * z * (1.0 + torch.erf(z / math.sqrt(2.0)))).to(out_dtype or x.dtype)
         if activation != "gelu_tanh":
             raise ValueError(activation)
         y = 0.5 * z * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
@@ -173,7 +196,8 @@ class TorchKernels:
 
     def attention_ext(self, q, q_col, num_heads, num_kv_heads, head_dim, v_head_dim, k_pool, v_pool, block_table, token_seq, positions,
                       page_size, scale, window, max_context, temp=(0.0, 0), rel=None, rel_rows=None, sink=None, gate=None, gate_col=0,
-                      gate_per_head=False, batch=None, num_splits=None, keep_first=0, chunk=0, softcap=0.0, talk=None):
+                      gate_per_head=False, batch=None, num_splits=None, keep_first=0, chunk=0, softcap=0.0, talk=None,
+                      sigmoid_bias=None, log_distance=None, turn=None):
         N = q.shape[0]
         rep = num_heads // num_kv_heads
         qs = q[:, q_col:q_col + num_heads * head_dim].float().view(N, num_heads, head_dim)
@@ -207,6 +231,11 @@ class TorchKernels:
                     dist = p - keys
                     row = torch.where(dist < rel_rows.shape[0], rel_rows.long()[dist.clamp(max=rel_rows.shape[0] - 1)], rel.shape[0] - 1)
                     s = s + rel[row, h].float()
+                if log_distance is not None:
+                    s = s - log_distance[0][h] * torch.log1p(log_distance[1][h] * (p - keys).float())
+                if sigmoid_bias is not None:
+                    out[t, h] = torch.sigmoid(s + sigmoid_bias[h]) @ v[:, h // rep]
+                    continue
                 if sink is not None:
                     top = max(float(s.max()), float(sink[h]))
                     e = torch.exp(s - top)
@@ -214,6 +243,8 @@ class TorchKernels:
                 else:
                     pr = torch.softmax(s, dim=0)
                 out[t, h] = pr @ v[:, h // rep]
+        if turn is not None:
+            out = self._turn(out, turn[0], -turn[1], v_head_dim, turn[2])
         if gate is not None:
             if gate_per_head:
                 out = out * torch.sigmoid(gate[:, gate_col:gate_col + num_heads].float())[:, :, None]
@@ -253,7 +284,17 @@ class TorchKernels:
     def weighted_pair(self, a, b, coef_a, coef_b, add_to):
         add_to += coef_a * a.float() + coef_b * b.float()
 
-    def softcap(self, x, cap):
+    def dynamic_tanh(self, residual, alpha, weight, bias, out_dtype, rows=None):
+        x = residual if rows is None else residual[rows.long()]
+        return (torch.tanh(alpha.float() * x) * weight.float() + bias.float()).to(out_dtype)
+
+    def post_tanh_add(self, residual, y, alpha, weight, bias):
+        residual += torch.tanh(alpha.float() * y.float()) * weight.float() + bias.float()
+
+    def softcap(self, x, cap, scale=1.0):
+        if cap is None:
+            return scale * x
+        x = scale * x
         return cap * torch.tanh(x / cap)
 
     def dual_rmsnorm_mix(self, a, b, weight_a, weight_b, eps, coef, add_to):
@@ -266,8 +307,20 @@ class TorchKernels:
         g, u = gu[:, :i].float().clamp(max=limit), gu[:, i:].float().clamp(-limit, limit)
         return (g * torch.sigmoid(alpha * g) * (u + shift)).to(out_dtype or gu.dtype)
 
+    @staticmethod
+    def _turn(x, cos, sin, dims, interleaved):
+        """x [N, heads, D]: the first ``dims`` entries of every head turn, pairs half of them apart or neighbours."""
+        if not dims:
+            return x
+        c, s = cos[:, None, :], sin[:, None, :]
+        out = x.clone()
+        first, second = (slice(0, dims, 2), slice(1, dims, 2)) if interleaved else (slice(0, dims // 2), slice(dims // 2, dims))
+        a, b = x[..., first], x[..., second]
+        out[..., first], out[..., second] = a * c - b * s, b * c + a * s
+        return out
+
     def qk_norm_rope_store(self, z, num_heads, num_kv_heads, head_dim, v_head_dim, q_weight, k_weight, eps, cos, sin, rot_dims, interleaved,
-                           slot_mapping, k_pool, v_pool, page_size, write_kv=True):
+                           slot_mapping, k_pool, v_pool, page_size, write_kv=True, v_turn=None, out_dtype=None):
         N = z.shape[0]
         nq, nk = num_heads * head_dim, num_kv_heads * head_dim
         zf = z.float()
@@ -277,26 +330,14 @@ class TorchKernels:
             q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps) * q_weight.float()
             k = k * torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps) * k_weight.float()
 
-        def turn(x):
-            if not rot_dims:
-                return x
-            c, s = cos[:, None, :], sin[:, None, :]
-            out = x.clone()
-            if interleaved:
-                a, b = x[..., 0:rot_dims:2], x[..., 1:rot_dims:2]
-                out[..., 0:rot_dims:2], out[..., 1:rot_dims:2] = a * c - b * s, b * c + a * s
-            else:
-                h = rot_dims // 2
-                a, b = x[..., :h], x[..., h:rot_dims]
-                out[..., :h], out[..., h:rot_dims] = a * c - b * s, b * c + a * s
-            return out
-
-        q, k = turn(q), turn(k)
+        q, k = self._turn(q, cos, sin, rot_dims, interleaved), self._turn(k, cos, sin, rot_dims, interleaved)
+        if v_turn is not None:
+            v = self._turn(v, *v_turn, v_head_dim, interleaved)
         if write_kv:
             page, off = (slot_mapping // page_size).long(), (slot_mapping % page_size).long()
             k_pool[page, :, off] = k.to(k_pool.dtype)
             v_pool[page, :, off] = v.to(v_pool.dtype)
-        return q.reshape(N, nq).to(z.dtype)
+        return q.reshape(N, nq).to(out_dtype or z.dtype)
 
     # ------------------------------------------------------------------ mixers with a state of fixed size
     @staticmethod
