@@ -80,7 +80,7 @@ def write_safetensors(path: str | Path, tensors: Dict[str, torch.Tensor]) -> Non
         t = t.detach().cpu().contiguous()
         if t.dtype not in _NAMES:
             raise ValueError(f"tensor '{name}' has dtype {t.dtype}, which cannot be written")
-        raw = t.view(torch.uint8).numpy().tobytes() if t.numel() else b""
+        raw = t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b""
         header[name] = {"dtype": _NAMES[t.dtype], "shape": list(t.shape), "data_offsets": [offset, offset + len(raw)]}
         offset += len(raw)
         blobs.append(raw)
@@ -116,4 +116,4 @@ def write_safetensors_stream(path: str | Path, metas, produce) -> None:
             if t.dtype != dtype or tuple(t.shape) != tuple(shape):
                 raise ValueError(f"tensor '{name}' came as {t.dtype} {list(t.shape)}, announced as {dtype} {list(shape)}")
             if t.numel():
-                f.write(memoryview(t.view(torch.uint8).numpy().reshape(-1)))
+                f.write(memoryview(t.reshape(-1).view(torch.uint8).numpy().reshape(-1)))

@@ -109,7 +109,9 @@ def sigmoid_attention(m: dict, W: Dict[str, torch.Tensor], p: str, h):
     T, H, G = h.shape[0], int(m["heads"]), int(m["kv_heads"])
     q, k, v = projections(m, W, p, h, bias=False)
     dist = torch.arange(T)[:, None] - torch.arange(T)[None, :]
-    seen = (dist >= 0) & (dist < int(m["mask"]["size"]))
+    seen = dist >= 0
+    if m.get("mask"):
+        seen = seen & (dist < int(m["mask"]["size"]))
     d = dist.clamp(min=0).to(h.dtype)
     heads = []
     for n in range(H):

@@ -427,3 +427,19 @@ def test_random_weights_and_the_command_line(tmp_path):
     for t in tokens:
         assert t == int(plain_logits(cfg, tensors, seq)[-1].argmax())
         seq.append(t)
+
+
+@pytest.mark.parametrize("graphs", [False, True])
+def test_a_prompt_in_equal_portions_under_graphs(cases, graphs):
+    """A prompt under a small token budget gives step after step of one shape, which is captured while the request is in the middle of
+    its prompt: the capture's warm-up runs the step on the request's states, and must leave them as they were."""
+    from llm_infrence_engine_b200.engine import Engine
+
+    folder, cfg, tensors, prompts, want = cases[("B", "float32")]
+    eng = Engine(folder, dtype="float32", max_len=256, max_seqs=2, block_size=16, num_blocks=40, max_num_batched_tokens=16, cuda_graphs=graphs)
+    for p in (prompts["a"], prompts["e"]):
+        r = eng.generate([p], max_new_tokens=4)[0]
+        seq = list(p) + r.token_ids
+        assert r.token_ids == plain_logits(cfg, tensors, seq)[len(p) - 1:-1].argmax(-1).tolist()
+    if graphs:
+        assert eng.runner.graphs.shape_replays > 3
