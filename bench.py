@@ -20,7 +20,7 @@ batch of 8 requests and a context of 8192 tokens. A "step" is one decode step of
 ``roofline``  bytes a decode step must read (every weight once + the live requests' cache) / its time.
 ``points``    decode tokens per second at batch 1 and 64, same method as ``value``.
 
-``--workload serving | luvutar | zepalorn | mufotar | memilorn`` measure other things (a stream of requests through the engine; the other architectures
+``--workload serving | luvutar | zepalorn | mufotar | memilorn | sinorax`` measure other things (a stream of requests through the engine; the other architectures
 beside Qwen2 of equal size, Mufotar beside Zepalorn, with ``--kernels`` also kernel by kernel) and print lines of their own; the default line is
 unchanged by them.
 
@@ -1315,6 +1315,172 @@ def memilorn_workload(a) -> int:
     return 0
 
 
+# ---------------------------------------------------------------------------------------------------------------------
+# ``--workload sinorax``: the Sinorax decoder at layer sizes of real models, beside the Qwen2 decoder (the closest of the engine's other
+# models: nothing but grouped attention, full and windowed, and dense feed-forwards) of equal width, heads, layers, windows and weights.
+
+SINORAX_SIZES = {
+    # name: (width, heads, kv heads, head_dim, window, ff, gated ff of equal weights, layers, vocab)
+    "0.5b-like": (896, 14, 2, 64, 1024, 7296, 4864, 8, 32768),
+    "3b-like": (2048, 16, 4, 128, 1024, 8256, 5504, 8, 32768),
+}
+SINORAX_NAMES = ("width", "heads", "kv_heads", "head_dim", "window", "ff", "qwen2_ff", "layers", "vocab")
+
+
+def sinorax_config(size: str) -> dict:
+    """The first half of the layers full attention, the second half windowed (the order in which Qwen2 has them)."""
+    W, H, G, d, win, ff, _, layers, vocab = SINORAX_SIZES[size]
+    heads = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5}
+    mlp = {"kind": "dense", "ff": ff}
+    full = {"type": "attention", "mixer": {**heads, "rot": {"dims": d, "base": 1000000.0, "scaling": {"factor": 2.0}}}, "mlp": mlp}
+    windowed = {"type": "attention_2", "mixer": {**heads, "mask": {"size": win}}, "mlp": mlp}
+    return {"architecture": "Sinorax", "vocab": vocab, "width": W, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 8191, "mul_cur": 127}}, "logit_scale": 0.25, "logit_softcap": 30.0,
+            "layers": [full if i < layers // 2 else windowed for i in range(layers)]}
+
+
+def qwen2_beside_sinorax(size: str) -> dict:
+    W, H, G, d, win, _, ff, layers, vocab = SINORAX_SIZES[size]
+    return {"architectures": ["Qwen2ForCausalLM"], "model_type": "qwen2", "vocab_size": vocab, "hidden_size": W, "head_dim": d,
+            "intermediate_size": ff, "num_hidden_layers": layers, "num_attention_heads": H, "num_key_value_heads": G, "rms_norm_eps": 1e-6,
+            "rope_theta": 1000000.0, "tie_word_embeddings": False, "max_position_embeddings": 32768, "use_sliding_window": True, "sliding_window": win,
+            "max_window_layers": layers // 2, "hidden_act": "silu"}
+
+
+def sinorax_kernel_points(torch, pk, size: str) -> dict:
+    """Sinorax's kernels one by one, each beside the Qwen2 kernel that does the like job at the same size: microseconds, and the fraction
+    of its roofline (bytes that must move / copy peak, or flops / bf16 peak)."""
+    from types import SimpleNamespace
+
+    from llm_infrence_engine_b200.csrc import get_kernels
+
+    K = get_kernels()
+    W, H, G, d, win, ff, gated, _, vocab = SINORAX_SIZES[size]
+    bf, dev = torch.bfloat16, "cuda"
+    hbm, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    out = {}
+
+    def entry(us, bytes_=None, flops=None):
+        e = {"us": round(us, 2)}
+        if bytes_ is not None:
+            e["frac_of_copy_peak"] = round(bytes_ / (us * 1e-6) / hbm, 4)
+        if flops is not None:
+            e["frac_of_bf16_peak"] = round(flops / (us * 1e-6) / tf, 4)
+        return e
+
+    r = lambda *n: torch.randn(*n, device=dev)
+    for what, batch, ctx, T in (("decode", 8, 4096, 1), ("decode_b64", 64, 4096, 1), ("prefill", 1, 2048, 2048)):
+        per = -(-ctx // BLOCK)
+        table = torch.zeros((batch + 1, per), dtype=torch.int32, device=dev)
+        table[:batch] = (torch.randperm(batch * per, device=dev).to(torch.int32) + 1).view(batch, per)
+        N = batch * T
+        seq = torch.arange(batch, dtype=torch.int32, device=dev).repeat_interleave(T)
+        pos = (torch.arange(T, dtype=torch.int32, device=dev) + (ctx - T)).repeat(batch)
+        starts = torch.arange(0, N + 1, T, dtype=torch.int32, device=dev)
+        b = SimpleNamespace(seq_lens=[T] * batch, seq_starts_dev=starts, num_seqs=batch, max_seq_len=T, _tables={})
+        kp, vp = r(batch * per + 1, G, BLOCK, d).to(bf), r(batch * per + 1, G, BLOCK, d).to(bf)
+        qkv = r(N, (H + 2 * G) * d).to(bf)
+        q = qkv[:, :H * d].contiguous()
+        cos, sin = r(N, d // 2), r(N, d // 2)
+        pb, r1, r2 = torch.full((H,), -4.0, device=dev), torch.ones(H, device=dev), torch.ones(H, device=dev)
+        if T == 1:
+            moved, fl = batch * ctx * 2 * G * d * 2, None
+            moved_w, fl_w = batch * win * 2 * G * d * 2, None
+        else:
+            moved, fl = None, 4.0 * H * d * (T * (T + 1) / 2) * batch
+            moved_w, fl_w = None, 4.0 * H * d * sum(min(p + 1, win) for p in range(ctx - T, ctx)) * batch
+
+        def qwen2(window):
+            b._tables.clear()
+            K.paged_attention(qkv, kp, vp, table, seq, pos, H, G, d, BLOCK, d ** -0.5, window, ctx, batch=b)
+
+        def sinorax(window, **kw):
+            b._tables.clear()
+            K.attention_ext(q, 0, H, G, d, d, kp, vp, table, seq, pos, BLOCK, d ** -0.5, window, ctx, batch=b, **kw)
+
+        out[f"attention_{what}_qwen2"] = entry(_time_graph(lambda: qwen2(0), torch), moved, fl)
+        out[f"attention_{what}_sinorax_turned_values"] = entry(_time_graph(lambda: sinorax(0, turn=(cos, sin, False)), torch), moved, fl)
+        out[f"attention_{what}_qwen2_window"] = entry(_time_graph(lambda: qwen2(win), torch), moved_w, fl_w)
+        out[f"attention_{what}_sinorax_sigmoid_window"] = entry(_time_graph(lambda: sinorax(win, sigmoid_bias=pb, log_distance=(r1, r2)), torch), moved_w, fl_w)
+        # the projections with bias, rotation and cache write
+        slots = torch.randperm(batch * per * BLOCK, device=dev)[:N].to(torch.int32)
+        h, w, bias = r(N, W).to(bf), r((H + 2 * G) * d, W).to(bf) * 0.02, r((H + 2 * G) * d)
+        bias_bf = bias.to(bf)
+        fl = 2.0 * N * W * (H + 2 * G) * d if T > 1 else None
+        moved = None if T > 1 else (H + 2 * G) * d * W * 2
+        out[f"qkv_{what}_qwen2"] = entry(_time_graph(lambda: K.qkv_rope(h, w, bias, cos, sin, slots, kp, vp, H, G, d, BLOCK), torch), moved, fl)
+        out[f"qkv_{what}_sinorax"] = entry(_time_graph(lambda: K.qk_norm_rope_store(K.linear(h, w, out_dtype=bf, transient=True, bias=bias_bf), H, G, d, d, None, None, 0.0, cos, sin, d,
+                                                                                    False, slots, kp, vp, BLOCK, v_turn=(cos, sin), out_dtype=bf), torch), moved, fl)
+        del kp, vp
+        wo, bo = r(W, H * d).to(bf) * 0.02, r(W).to(bf)
+        y = torch.zeros(N, W, device=dev)
+
+        def add(bias_):
+            K.linear(q, wo, add_to=y, bias=bias_)
+            K._pending_add = None
+
+        fl, moved = (2.0 * N * W * H * d, None) if T > 1 else (None, W * H * d * 2)
+        out[f"o_{what}_qwen2"] = entry(_time_graph(lambda: add(None), torch), moved, fl)
+        out[f"o_{what}_sinorax_with_bias"] = entry(_time_graph(lambda: add(bo), torch), moved, fl)
+        # the feed-forward going in, at equal weights
+        wgu, wup = r(2 * gated, W).to(bf) * 0.02, r(ff, W).to(bf) * 0.02
+        fl, moved = (2.0 * N * W * 2 * gated, None) if T > 1 else (None, 2 * gated * W * 2)
+        out[f"ff_in_{what}_qwen2"] = entry(_time_graph(lambda: K.gate_up_act(h, wgu, bf), torch), moved, fl)
+        fl, moved = (2.0 * N * W * ff, None) if T > 1 else (None, ff * W * 2)
+        out[f"ff_in_{what}_sinorax"] = entry(_time_graph(lambda: K.linear_act(h, wup, "gelu_erf", bf), torch), moved, fl)
+        # norms: the stream takes a sublayer's result and is normed for the next one
+        res, delta, one = r(N, W), r(N, W).to(bf), torch.ones(W, device=dev)
+        alpha = torch.tensor(0.5, device=dev)
+
+        def both():
+            K.post_tanh_add(res, delta, alpha, one, one)
+            return K.dynamic_tanh(res, alpha, one, one, bf)
+
+        moved = N * W * (4 + 4 + 2 + 2)
+        out[f"norm_{what}_qwen2"] = entry(_time_graph(lambda: K.add_rmsnorm(res, delta, one, 1e-6, bf), torch), moved)
+        out[f"norm_{what}_sinorax"] = entry(_time_graph(both, torch), moved)
+        ids = torch.randint(0, vocab, (N,), device=dev, dtype=torch.int32)
+        table_e, table_b, last = r(vocab, W).to(bf), r(65522, W).to(bf), torch.zeros(batch + 1, 1, dtype=torch.int32, device=dev)
+        out[f"embedding_{what}_qwen2"] = entry(_time_graph(lambda: K.embed(ids, table_e), torch), N * W * (2 + 4))
+        out[f"embedding_{what}_sinorax"] = entry(_time_graph(lambda: K.embed_bigram(ids, table_e, table_b, 65521, 8191, 127, pos, seq, starts, batch, last), torch), N * W * (2 + 2 + 4))
+        if T == 1:
+            logits = r(N, vocab)
+            out[f"soft_cap_{what}_sinorax"] = entry(_time_graph(lambda: K.softcap(logits, 30.0, 0.25), torch), N * vocab * 8)
+    K.check_device_errors()
+    return out
+
+
+def sinorax_workload(a) -> int:
+    import torch
+
+    from llm_infrence_engine_b200.weights import write_random_model
+
+    pk = peaks()
+    sampler = ClockSampler()
+    sampler.start()
+    sizes = {}
+    steps = min(a.steps, 256)
+    for size in SINORAX_SIZES:
+        row = {}
+        for name, config in (("sinorax", sinorax_config(size)), ("qwen2", qwen2_beside_sinorax(size))):
+            with tempfile.TemporaryDirectory() as tmp:
+                folder = write_random_model(config, Path(tmp) / "model", seed=0, store_dtype="bfloat16")
+                pt = model_points(folder, SINORAX_SIZES[size][-1], a.batch, a.context or 4096, a.prefill_tokens, steps, max(a.warmup, 3), torch)
+            pt["decode_frac_of_copy_peak"] = round(pt["decode_bytes"] / (pt["decode_ms"] * 1e-3) / 1e9 / pk["hbm_gbs"], 4)
+            row[name] = pt
+        sizes[size] = row
+    line = {"metric": f"Sinorax beside Qwen2 of equal size: decode (batch {a.batch}, context {a.context or 4096}) and prefill ({a.prefill_tokens} tokens), bf16, random weights",
+            "unit": "ms and tokens/s per size", "n_gpus": 1, "impl": "ours", "dtype": "bf16", "steps": steps, "warmup": max(a.warmup, 3),
+            "data": "synthetic: random weights (seed 0), uniform random token ids, synthetic cache contents",
+            "config": {"sizes": {k: dict(zip(SINORAX_NAMES, v)) for k, v in SINORAX_SIZES.items()}, "block_size": BLOCK, "peaks": pk["source"],
+                       "l2": "weights + cache per step larger than L2, no flush"},
+            "clocks": sampler.stop(), "sizes": sizes}
+    if a.kernels:
+        line["kernels"] = {size: sinorax_kernel_points(torch, pk, size) for size in SINORAX_SIZES}
+    print(json.dumps(line))
+    return 0
+
+
 def luvutar_workload(a) -> int:
     import torch
 
@@ -1362,12 +1528,13 @@ def main() -> int:
     ap.add_argument("--skip-e2e", action="store_true")
     ap.add_argument("--no-graphs", action="store_true", help="launch every kernel of a decode step from the host instead of replaying a CUDA graph")
     ap.add_argument("--only", default="all", choices=["all", "decode", "prefill"], help="measure one part only (for profiling); the JSON line then lacks the rest")
-    ap.add_argument("--workload", default="steps", choices=["steps", "serving", "luvutar", "zepalorn", "mufotar", "memilorn"],
+    ap.add_argument("--workload", default="steps", choices=["steps", "serving", "luvutar", "zepalorn", "mufotar", "memilorn", "sinorax"],
                     help="serving: continuous batching of --requests requests (prompts U[128,2048], outputs U[64,512]) through Engine; "
                          "luvutar, zepalorn: that decoder at two layer sizes beside the Qwen2 decoder of equal size (decode and prefill); "
                          "mufotar: that decoder at two layer sizes beside the Zepalorn decoder of equal size; "
-                         "memilorn: that decoder at two layer sizes beside the Mufotar decoder of equal size")
-    ap.add_argument("--kernels", action="store_true", help="luvutar, zepalorn, mufotar, memilorn: also time its kernels one by one beside their counterparts")
+                         "memilorn: that decoder at two layer sizes beside the Mufotar decoder of equal size; "
+                         "sinorax: that decoder at two layer sizes beside the Qwen2 decoder of equal size")
+    ap.add_argument("--kernels", action="store_true", help="luvutar, zepalorn, mufotar, memilorn, sinorax: also time its kernels one by one beside their counterparts")
     ap.add_argument("--requests", type=int, default=64)
     ap.add_argument("--token-budget", type=int, default=2048, help="serving: tokens per step (max_num_batched_tokens)")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="length of the timed prompt")
@@ -1383,6 +1550,8 @@ def main() -> int:
         return zepalorn_workload(a)
     if a.workload == "mufotar":
         return mufotar_workload(a)
+    if a.workload == "sinorax":
+        return sinorax_workload(a)
     if a.workload == "memilorn":
         return memilorn_workload(a)
     PREFILL_TOKENS = a.prefill_tokens
