@@ -367,12 +367,10 @@ struct RowTerms {
             b = -1.4426950408889634f * ex.sig_bias[head];
         }
     }
-    __device__ __forceinline__ static float lg2(float v) { float y; asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(v)); return y; }
-    __device__ __forceinline__ static float ex2(float v) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(v)); return y; }
-    __device__ __forceinline__ float penalty(float dist) const { return r1 * 0.6931471805599453f * lg2(fmaf(r2, dist, 1.0f)); }
+    __device__ __forceinline__ float penalty(float dist) const { return r1 * 0.6931471805599453f * hw_log2(fmaf(r2, dist, 1.0f)); }
     // (dist < 0, a key the row does not see, may give anything: the caller masks it)
     __device__ __forceinline__ float sigmoid(float s, float dist) const {
-        return __fdividef(1.0f, 1.0f + ex2(fmaf(r1, lg2(fmaf(r2, dist, 1.0f)), fmaf(a, s, b))));
+        return __fdividef(1.0f, 1.0f + hw_exp2(fmaf(r1, hw_log2(fmaf(r2, dist, 1.0f)), fmaf(a, s, b))));
     }
 };
 

@@ -54,6 +54,27 @@ struct Params {
     bf16* k_pool_w;         // the pools again, to write into
     bf16* v_pool_w;
     int acc_stride;
+    // Decode steps: sigmoid weights (sig_bias [nq], log_r1 / log_r2 [nq] or null; see attend_chunk) and results that are turned back
+    // (turn_cos / turn_sin [tokens][D / 2], pairs D / 2 apart; or null)
+    const float* sig_bias = nullptr;
+    const float* log_r1 = nullptr;
+    const float* log_r2 = nullptr;
+    const float* turn_cos = nullptr;
+    const float* turn_sin = nullptr;
+};
+
+// A lane's two rows' terms of sigmoid weights: the weight of a key at distance d is 1 / (1 + 2^x), x = b - scale_log2 s + r1 log2(1 + r2 d).
+// There is no maximum and no sum then: m stays 0, and the outputs are divided by one in the end.
+struct SigRows {
+    float b[2] = {0.f, 0.f}, r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
+    __device__ __forceinline__ void of(int i, int head, const Params& p) {
+        b[i] = -LOG2E * p.sig_bias[head];
+        if (p.log_r1) { r1[i] = p.log_r1[head]; r2[i] = p.log_r2[head]; }
+    }
+    // (a key behind the row's position may give anything: the caller masks it)
+    __device__ __forceinline__ float weight(int i, float s, int dist, float scale_log2) const {
+        return __fdividef(1.0f, 1.0f + hw_exp2(fmaf(r1[i], hw_log2(fmaf(r2[i], (float)dist, 1.0f)), fmaf(-scale_log2, s, b[i]))));
+    }
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
@@ -151,10 +172,10 @@ __device__ __forceinline__ void load_rows_warp(const Params& p, const int* table
 }
 
 // One chunk of BN keys for one warp's 16 rows: S = Q K^T, masked online softmax, O += P V.
-template <int D, int BN, bool MASKED = true>
+template <int D, int BN, bool MASKED = true, bool SIG = false>
 __device__ __forceinline__ void attend_chunk(const uint32_t (&qa)[D / 16][4], const bf16* ks, const bf16* vs, float (&o)[D / 8][4],
                                              float (&m)[2], float (&l)[2], int key0, const int (&row_pos)[2], const bool (&row_ok)[2],
-                                             int window, float scale_log2, int lane) {
+                                             int window, float scale_log2, int lane, const SigRows* sig = nullptr) {
     float s[BN / 8][4];
 #pragma unroll
     for (int i = 0; i < BN / 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
@@ -170,6 +191,22 @@ __device__ __forceinline__ void attend_chunk(const uint32_t (&qa)[D / 16][4], co
             mma_bf16(s[2 * nt + 1], qa[kk], b[2], b[3]);
         }
     }
+    uint32_t pa[BN / 16][4];
+    if constexpr (SIG) {
+#pragma unroll
+        for (int nt = 0; nt < BN / 8; ++nt) {
+            float w[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int r = e >> 1;
+                const int key = key0 + nt * 8 + ((lane & 3) << 1) + (e & 1);
+                const bool ok = !MASKED || (row_ok[r] && key <= row_pos[r] && (window <= 0 || key > row_pos[r] - window));
+                w[e] = ok ? sig->weight(r, s[nt][e], row_pos[r] - key, scale_log2) : 0.f;
+            }
+            pa[nt >> 1][(nt & 1) * 2] = pack_bf16(w[0], w[1]);
+            pa[nt >> 1][(nt & 1) * 2 + 1] = pack_bf16(w[2], w[3]);
+        }
+    } else {
     // mask and running maximum, in units of log2: x = s * scale * log2(e)
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -200,7 +237,6 @@ __device__ __forceinline__ void attend_chunk(const uint32_t (&qa)[D / 16][4], co
         o[dt][0] *= corr[0]; o[dt][1] *= corr[0];
         o[dt][2] *= corr[1]; o[dt][3] *= corr[1];
     }
-    uint32_t pa[BN / 16][4];
 #pragma unroll
     for (int nt = 0; nt < BN / 8; ++nt) {
         const float p0 = fast_exp2(s[nt][0] - use[0]), p1 = fast_exp2(s[nt][1] - use[0]);
@@ -209,6 +245,7 @@ __device__ __forceinline__ void attend_chunk(const uint32_t (&qa)[D / 16][4], co
         l[1] += p2 + p3;
         pa[nt >> 1][(nt & 1) * 2] = pack_bf16(p0, p1);
         pa[nt >> 1][(nt & 1) * 2 + 1] = pack_bf16(p2, p3);
+    }
     }
 #pragma unroll
     for (int kk = 0; kk < BN / 16; ++kk) {
@@ -238,10 +275,10 @@ __device__ __forceinline__ uint32_t transpose_8x8(uint32_t a) {
     return d;
 }
 
-template <int D, int BN, bool MASKED>
+template <int D, int BN, bool MASKED, bool SIG = false>
 __device__ __forceinline__ void attend_chunk_t8(const uint32_t (&qb)[D / 16][2], const bf16* ks, const bf16* vs, float (&ot)[D / 16][4],
                                                 float (&m)[2], float (&l)[2], int key0, int pos, int nrows, int window, float scale_log2,
-                                                int lane) {
+                                                int lane, const SigRows* sig = nullptr) {
     float st[BN / 16][4];
 #pragma unroll
     for (int kt = 0; kt < BN / 16; ++kt) {
@@ -256,6 +293,21 @@ __device__ __forceinline__ void attend_chunk_t8(const uint32_t (&qb)[D / 16][2],
             mma_bf16(st[kt], a, qb[kk][0], qb[kk][1]);
         }
     }
+    uint32_t pb[BN / 16][2];
+    if constexpr (SIG) {
+#pragma unroll
+        for (int kt = 0; kt < BN / 16; ++kt) {
+            float w[4];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int key = key0 + kt * 16 + (lane >> 2) + ((e >> 1) << 3);
+                const bool ok = !MASKED || (((lane & 3) << 1) + (e & 1) < nrows && key <= pos && (window <= 0 || key > pos - window));
+                w[e] = ok ? sig->weight(e & 1, st[kt][e], pos - key, scale_log2) : 0.f;
+            }
+            pb[kt][0] = transpose_8x8(pack_bf16(w[0], w[1]));
+            pb[kt][1] = transpose_8x8(pack_bf16(w[2], w[3]));
+        }
+    } else {
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int kt = 0; kt < BN / 16; ++kt) {
@@ -285,7 +337,6 @@ __device__ __forceinline__ void attend_chunk_t8(const uint32_t (&qb)[D / 16][2],
         ot[dt][0] *= corr[0]; ot[dt][1] *= corr[1];
         ot[dt][2] *= corr[0]; ot[dt][3] *= corr[1];
     }
-    uint32_t pb[BN / 16][2];
 #pragma unroll
     for (int kt = 0; kt < BN / 16; ++kt) {
         const float p0 = fast_exp2(st[kt][0] - use[0]), p1 = fast_exp2(st[kt][1] - use[1]);
@@ -294,6 +345,7 @@ __device__ __forceinline__ void attend_chunk_t8(const uint32_t (&qb)[D / 16][2],
         l[1] += p1 + p3;
         pb[kt][0] = transpose_8x8(pack_bf16(p0, p1));  // keys 0-7 of the tile: [key][row] -> [row][key]
         pb[kt][1] = transpose_8x8(pack_bf16(p2, p3));  // keys 8-15
+    }
     }
 #pragma unroll
     for (int dt = 0; dt < D / 16; ++dt) {
@@ -311,7 +363,7 @@ __device__ __forceinline__ void attend_chunk_t8(const uint32_t (&qb)[D / 16][2],
 
 // ---------------------------------------------------------------------------------------------- decode
 // T8: every tile has at most 8 rows and one token (a decode step of a model with up to 8 heads per group): the transposed form.
-template <int D, int BN, int STAGES, int DW, bool T8>
+template <int D, int BN, int STAGES, int DW, bool T8, bool SIG>
 __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p) {
     extern __shared__ __align__(128) unsigned char smem_raw[];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -459,6 +511,14 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
         for (int i = 0; i < D / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     }
     float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    SigRows sig;
+    if constexpr (SIG) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+            const int row = T8 ? ((lane & 3) << 1) + j : (lane >> 2) + 8 * j;
+            sig.of(j, kvh * G + (row < nrows ? row % G : 0), p);
+        }
+    }
 
 #pragma unroll
     for (int s = 0; s < STAGES; ++s) {
@@ -497,11 +557,11 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
         // rows beyond the tile then collect numbers nobody reads
         const bool interior = key0 + BN - 1 <= pos0 && (p.window <= 0 || key0 > hi - 1 - p.window);
         if constexpr (T8) {
-            if (interior) attend_chunk_t8<D, BN, false>(qb, cur, cur + TILE, o, m, l, key0, pos0, nrows, p.window, p.scale_log2, lane);
-            else attend_chunk_t8<D, BN, true>(qb, cur, cur + TILE, o, m, l, key0, pos0, nrows, p.window, p.scale_log2, lane);
+            if (interior) attend_chunk_t8<D, BN, false, SIG>(qb, cur, cur + TILE, o, m, l, key0, pos0, nrows, p.window, p.scale_log2, lane, &sig);
+            else attend_chunk_t8<D, BN, true, SIG>(qb, cur, cur + TILE, o, m, l, key0, pos0, nrows, p.window, p.scale_log2, lane, &sig);
         } else {
-            if (interior) attend_chunk<D, BN, false>(qa, cur, cur + TILE, o, m, l, key0, row_pos, row_ok, p.window, p.scale_log2, lane);
-            else attend_chunk<D, BN, true>(qa, cur, cur + TILE, o, m, l, key0, row_pos, row_ok, p.window, p.scale_log2, lane);
+            if (interior) attend_chunk<D, BN, false, SIG>(qa, cur, cur + TILE, o, m, l, key0, row_pos, row_ok, p.window, p.scale_log2, lane, &sig);
+            else attend_chunk<D, BN, true, SIG>(qa, cur, cur + TILE, o, m, l, key0, row_pos, row_ok, p.window, p.scale_log2, lane, &sig);
         }
         __syncwarp();  // every lane is done with the slot
         const int nxt = it + STAGES;
@@ -523,6 +583,10 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
             l[r] += __shfl_xor_sync(0xffffffffu, l[r], 1);
             l[r] += __shfl_xor_sync(0xffffffffu, l[r], 2);
         }
+    }
+    if constexpr (SIG) {   // nothing is relative to a maximum, and the outputs are divided by one
+        m[0] = m[1] = 0.f;
+        l[0] = l[1] = (warp == 0 && split == 0) ? 1.f : 0.f;
     }
     __syncthreads();  // every warp is done with its ring; the space is reused for the merge
     constexpr int MR = T8 ? 8 : 16;                     // rows that are merged
@@ -582,6 +646,17 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
         }
     }
     __syncthreads();
+    if (p.turn_cos) {
+        // turned back here, slice by slice (the turn is linear and the same for all slices of a row)
+        for (int i = tid; i < nrows * (D / 2); i += DW * 32) {
+            const int r = i / (D / 2), k = i % (D / 2);
+            const size_t at = (size_t)(n0 + r / G) * (D / 2) + k;
+            const float a = fo[r * D + k], b = fo[r * D + D / 2 + k], c = p.turn_cos[at], sn = p.turn_sin[at];
+            fo[r * D + k] = fmaf(b, sn, a * c);
+            fo[r * D + D / 2 + k] = fmaf(-a, sn, b * c);
+        }
+        __syncthreads();
+    }
     if (p.cluster && p.num_splits > 1) {
         // The slices of this tile are the blocks of one cluster: block 0 reads every block's (max, sum, output) out of
         // its shared memory and writes the rows. Nothing goes through global memory and nobody waits on a counter.
@@ -747,7 +822,7 @@ __global__ void attn_plan_kernel(const int* __restrict__ starts, int num_seqs, i
     for (; t < max_tiles; ++t) { tile_info[2 * t] = 0; tile_info[2 * t + 1] = 0; }
 }
 
-template <int D, bool T8, int DW>
+template <int D, bool T8, int DW, bool SIG = false>
 int launch_decode(const Params& p, dim3 grid, cudaStream_t s) {
     constexpr int BN = D == 64 ? 32 : 16, STAGES = 3;  // DW warps, each with its own ring of 4 KB + 4 KB chunks
     constexpr size_t ring = (size_t)DW * STAGES * 2 * BN * D * sizeof(bf16);
@@ -755,7 +830,7 @@ int launch_decode(const Params& p, dim3 grid, cudaStream_t s) {
     constexpr size_t smem = ring > merge ? ring : merge;
     static bool set = false;
     if (!set) {
-        cudaError_t e = cudaFuncSetAttribute(attn_mma_decode_kernel<D, BN, STAGES, DW, T8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         set = true;
     }
@@ -774,9 +849,9 @@ int launch_decode(const Params& p, dim3 grid, cudaStream_t s) {
         attr[1].val.programmaticStreamSerializationAllowed = 1;
         cfg.attrs = attr;
         cfg.numAttrs = llmie_pdl_flag ? 2 : 1;
-        return (int)cudaLaunchKernelEx(&cfg, attn_mma_decode_kernel<D, BN, STAGES, DW, T8>, p);
+        return (int)cudaLaunchKernelEx(&cfg, attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG>, p);
     }
-    return launch_kernel(attn_mma_decode_kernel<D, BN, STAGES, DW, T8>, grid, dim3(DW * 32), smem, s, p);
+    return launch_kernel(attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG>, grid, dim3(DW * 32), smem, s, p);
 }
 
 template <int D>
@@ -789,6 +864,10 @@ int launch(const Params& p, int num_tiles, int decode_mode, cudaStream_t s) {
         // blocks than multiprocessors and nothing is cut into slices, the caller may ask for blocks of four warps (96 KB:
         // two per multiprocessor), which then run in fewer, fuller rounds (96 requests of 8,192 keys: 94 us in two rounds of
         // eight-warp blocks, the second half empty; 74.5 us at once).
+        if (p.sig_bias) {
+            if (decode_mode == 2 && p.num_splits == 1) return t8 ? launch_decode<D, true, 4, true>(p, grid, s) : launch_decode<D, false, 4, true>(p, grid, s);
+            return t8 ? launch_decode<D, true, 8, true>(p, grid, s) : launch_decode<D, false, 8, true>(p, grid, s);
+        }
         if (decode_mode == 2 && p.num_splits == 1) return t8 ? launch_decode<D, true, 4>(p, grid, s) : launch_decode<D, false, 4>(p, grid, s);
         return t8 ? launch_decode<D, true, 8>(p, grid, s) : launch_decode<D, false, 8>(p, grid, s);
     } else {
@@ -815,14 +894,19 @@ LLMIE_API int llmie_attn_plan(const int* seq_starts, int num_seqs, int tokens_pe
 
 // decode_mode 1 or 2: every tile has at most 16 rows (tokens * group); 2 asks for blocks of four warps instead of eight when
 // nothing is cut into slices. 0: at most 64 rows.
+// turn_cos / turn_sin (or null), sig_bias (or null), log_r1 / log_r2 (or null): decode modes only.
 // scratch_o / scratch_ml / counters are needed for num_splits > 1 (counters zeroed once; the kernel leaves them zero), unless
 // `cluster` is set (decode mode, at most 8 slices): the slices then form one thread-block cluster and merge in shared memory.
 static int run_mma(const bf16* q, int q_stride, const bf16* k_pool, const bf16* v_pool, const int* block_table,
                    int max_blocks, const int* token_seq, const int* positions, const int* tile_info, int num_tiles,
                    bf16* out, float* scratch_o, float* scratch_ml, int* counters, int nq, int nkv, int d,
                    int page_size, float scale, int window, int num_splits, int decode_mode, int cluster, const float* qkv_acc,
-                   int acc_stride, const float* bias, const float* cos_t, const float* sin_t, const int* slots, cudaStream_t s) {
+                   int acc_stride, const float* bias, const float* cos_t, const float* sin_t, const int* slots, const float* turn_cos, const float* turn_sin,
+                   const float* sig_bias, const float* log_r1, const float* log_r2, cudaStream_t s) {
     if (num_tiles <= 0) return 0;
+    if ((turn_cos == nullptr) != (turn_sin == nullptr) || (log_r1 == nullptr) != (log_r2 == nullptr) || (log_r1 && !sig_bias) ||
+        ((turn_cos || sig_bias) && !decode_mode))
+        return LLMIE_ERR_BAD_ARGUMENT;
     if (qkv_acc && (!decode_mode || tile_info || nq / (nkv > 0 ? nkv : 1) > 8 || !cos_t || !sin_t || acc_stride < (nq + 2 * nkv) * d ||
                     (acc_stride & 1) || ((uintptr_t)qkv_acc & 7) || ((uintptr_t)bias & 7) || ((uintptr_t)cos_t & 7) || ((uintptr_t)sin_t & 7)))
         return LLMIE_ERR_BAD_ARGUMENT;
@@ -839,6 +923,7 @@ static int run_mma(const bf16* q, int q_stride, const bf16* k_pool, const bf16* 
     p.page_shift = (page_size & (page_size - 1)) == 0 ? __builtin_ctz((unsigned)page_size) : -1;
     p.num_splits = num_splits; p.scale_log2 = scale * LOG2E; p.cluster = cluster;
     p.qkv_acc = qkv_acc; p.acc_stride = acc_stride; p.bias = bias; p.cos_t = cos_t; p.sin_t = sin_t; p.slots = slots;
+    p.turn_cos = turn_cos; p.turn_sin = turn_sin; p.sig_bias = sig_bias; p.log_r1 = log_r1; p.log_r2 = log_r2;
     p.k_pool_w = const_cast<bf16*>(k_pool); p.v_pool_w = const_cast<bf16*>(v_pool);
     return d == 64 ? launch<64>(p, num_tiles, decode_mode, s) : launch<128>(p, num_tiles, decode_mode, s);
 }
@@ -846,10 +931,11 @@ static int run_mma(const bf16* q, int q_stride, const bf16* k_pool, const bf16* 
 LLMIE_API int llmie_paged_attention_mma(const bf16* q, int q_stride, const bf16* k_pool, const bf16* v_pool, const int* block_table,
                                         int max_blocks, const int* token_seq, const int* positions, const int* tile_info, int num_tiles,
                                         bf16* out, float* scratch_o, float* scratch_ml, int* counters, int nq, int nkv, int d,
-                                        int page_size, float scale, int window, int num_splits, int decode_mode, int cluster, cudaStream_t s) {
+                                        int page_size, float scale, int window, int num_splits, int decode_mode, int cluster, const float* turn_cos,
+                                        const float* turn_sin, const float* sig_bias, const float* log_r1, const float* log_r2, cudaStream_t s) {
     return run_mma(q, q_stride, k_pool, v_pool, block_table, max_blocks, token_seq, positions, tile_info, num_tiles, out, scratch_o, scratch_ml,
                    counters, nq, nkv, d, page_size, scale, window, num_splits, decode_mode, cluster, nullptr, 0, nullptr, nullptr, nullptr,
-                   nullptr, s);
+                   nullptr, turn_cos, turn_sin, sig_bias, log_r1, log_r2, s);
 }
 
 // Decode steps (every tile one token, at most 8 query heads per key/value head): the same attention, with the queries, keys and
@@ -863,5 +949,6 @@ LLMIE_API int llmie_paged_attention_mma_acc(const float* qkv_acc, int acc_stride
                                             int num_splits, int cluster, int four_warps, cudaStream_t s) {
     if (!qkv_acc) return LLMIE_ERR_BAD_ARGUMENT;
     return run_mma(nullptr, 8, k_pool, v_pool, block_table, max_blocks, token_seq, positions, nullptr, num_tokens, out, scratch_o, scratch_ml,
-                   counters, nq, nkv, d, page_size, scale, window, num_splits, four_warps ? 2 : 1, cluster, qkv_acc, acc_stride, bias, cos_t, sin_t, slots, s);
+                   counters, nq, nkv, d, page_size, scale, window, num_splits, four_warps ? 2 : 1, cluster, qkv_acc, acc_stride, bias, cos_t, sin_t, slots,
+                   nullptr, nullptr, nullptr, nullptr, nullptr, s);
 }

@@ -25,6 +25,11 @@
 //              guarded by mbarriers
 //   warp 5     one lane issues the MMAs and commits them to the barriers the other warps wait on
 //
+// Two more things a mixer may ask for. Sigmoid weights (SIG): a visible key's weight is sigmoid(scale s - r1 ln(1 + r2 distance) + bias) with
+// three numbers per query head; there is no maximum, no reference and no sum, P is the weights themselves. Values that were turned
+// by their positions when they were cached: a row's outputs are turned back by the row's own position before they leave the
+// block (a slice's partial outputs too: the turn is linear and the same for all slices of a row).
+//
 // A launch follows a plan made once per step on the device (attn_tc_plan_kernel): which pieces of work there are (a tile,
 // or one slice of a long tile's keys, whose partial result the last slice merges), long pieces first.
 //
@@ -72,6 +77,11 @@ struct TcParams {
     int box_rows;           // rows per TMA box: min(page_size, BN)
     int num_tiles;
     float scale_log2;       // softmax scale * log2(e)
+    const float* turn_cos;  // [tokens][D / 2], with turn_sin: outputs are turned back (pairs D / 2 apart); or null
+    const float* turn_sin;
+    const float* sig_bias;  // SIG: [nq]
+    const float* log_r1;    // SIG: [nq] or null, with log_r2
+    const float* log_r2;
 };
 
 __device__ __forceinline__ float fast_exp2(float x) {
@@ -131,7 +141,7 @@ __device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
     asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(bar)) : "memory");
 }
 
-template <int D>
+template <int D, bool SIG>
 __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k,
                                                                                           const __grid_constant__ CUtensorMap tmap_v, const TcParams p) {
     constexpr int ATOMS = Sizes<D>::ATOMS, STAGES = Sizes<D>::STAGES, Q_BYTES = Sizes<D>::Q_BYTES, K_BYTES = Sizes<D>::K_BYTES;
@@ -340,7 +350,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
         const bool row_ok = row < nrows;
         const int tok = row_ok ? row / G : 0;
         const int pos = pos0 + tok;
-        {
+        if (chunks > 0) {   // (an empty slice puts its zeros where the tile would lie, without another wait)
             // this thread's query row into the swizzled tile (zeros for rows beyond the tile)
             const uint4* src = reinterpret_cast<const uint4*>(p.q + (size_t)(n0 + tok) * p.q_stride + (size_t)(kvh * G + (row_ok ? row % G : 0)) * D);
 #pragma unroll
@@ -355,6 +365,15 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
         // m: the row's running maximum (log2 units); ref: what P is taken relative to (-inf until the row has seen a key);
         // l: the row's sum of P relative to ref
         float m = -INFINITY, ref = -INFINITY, l = 0.f;
+        // (SIG) the row's weight of a key at distance d is 1 / (1 + 2^x), x = sig_b - scale_log2 s + sig_r1 log2(1 + sig_r2 d)
+        float sig_b = 0.f, sig_r1 = 0.f, sig_r2 = 0.f;
+        if constexpr (SIG) {
+            const int head = kvh * G + (row_ok ? row % G : 0);
+            sig_b = -LOG2E * p.sig_bias[head];
+            if (p.log_r1) { sig_r1 = p.log_r1[head]; sig_r2 = p.log_r2[head]; }
+            ref = 0.f;
+            l = split == 0 ? 1.f : 0.f;   // (what the outputs are divided by in the end: one)
+        }
         const uint32_t lane_base = tmem + ((uint32_t)(warp * 32) << 16);
         const uint32_t o_addr = lane_base + S_BUFS * BN;
         // the scores of chunk c are waited for during chunk c - 1 (see below): only the first ones here
@@ -374,6 +393,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
             // A chunk that every row of the tile sees in full needs no mask arithmetic (rows beyond the tile have zero
             // queries and collect numbers nobody reads). The scale is positive: the maximum is taken over the raw scores.
             const bool interior = key0 >= lo && key0 + BN - 1 <= pos0 && (p.window <= 0 || key0 > hi - 1 - p.window);
+            uint32_t keep_lo = 0xffffffffu, keep_hi = 0xffffffffu;
             if (__builtin_expect(!interior, 0)) {
                 // The columns this row sees are a run [first, last] of the chunk's 64: two words of bits say which, and a
                 // column outside is replaced (not multiplied: the score may be NaN) by -inf. Written small (three
@@ -386,10 +406,41 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 const uint32_t seen_lo = (uint32_t)seen, seen_hi = (uint32_t)(seen >> 32);
 #pragma unroll
                 for (int j = 0; j < 32; ++j) {
-                    if (!((seen_lo >> j) & 1u)) s[j] = 0xff800000u;
-                    if (!((seen_hi >> j) & 1u)) s[32 + j] = 0xff800000u;
+                    if (!((seen_lo >> j) & 1u)) s[j] = SIG ? 0u : 0xff800000u;
+                    if (!((seen_hi >> j) & 1u)) s[32 + j] = SIG ? 0u : 0xff800000u;
                 }
+                keep_lo = seen_lo;
+                keep_hi = seen_hi;
             }
+            float corr = 1.f;
+            uint64_t sum2[2] = {pair_of(0.f, 0.f), pair_of(0.f, 0.f)};
+            if constexpr (SIG) {
+                // two weights per division: 1 / t0 = t1 / (t0 t1), with t bounded so that the product stays finite (a weight below
+                // 2^-60 becomes 2^-60). What log2 makes of a key behind the row's position (a number or NaN) is replaced by
+                // the bound, and its weight by zero below.
+                ok = __all_sync(0xffffffffu, mbar_wait(s_ready + (c + 1) % S_BUFS, ((c + 1) / S_BUFS) & 1, abort_flag, p.error_flag, 15));
+                if (!ok) break;
+                const uint64_t scale2 = pair_of(-p.scale_log2, -p.scale_log2), bias2 = pair_of(sig_b, sig_b), r1_2 = pair_of(sig_r1, sig_r1);
+                const float far = fmaf(sig_r2, (float)(pos - key0), 1.0f);
+                const uint64_t step2 = pair_of(-sig_r2, -sig_r2), far2 = pair_of(far, far), one2 = pair_of(1.f, 1.f);
+#pragma unroll
+                for (int j = 0; j < BN; j += 2) {
+                    float y0, y1, x0, x1, t0, t1;
+                    unpair(fma2(pair_of((float)j, (float)(j + 1)), step2, far2), y0, y1);
+                    unpair(fma2(r1_2, pair_of(hw_log2(y0), hw_log2(y1)), fma2(pair_of(__uint_as_float(s[j]), __uint_as_float(s[j + 1])), scale2, bias2)), x0, x1);
+                    unpair(add2(pair_of(fast_exp2(fminf(x0, 60.f)), fast_exp2(fminf(x1, 60.f))), one2), t0, t1);
+                    const float r = __fdividef(1.0f, t0 * t1);
+                    s[j] = __float_as_uint(r * t1);
+                    s[j + 1] = __float_as_uint(r * t0);
+                }
+                if (__builtin_expect(!interior, 0)) {
+#pragma unroll
+                    for (int j = 0; j < 32; ++j) {
+                        if (!((keep_lo >> j) & 1u)) s[j] = 0u;
+                        if (!((keep_hi >> j) & 1u)) s[32 + j] = 0u;
+                    }
+                }
+            } else {
             // four running maxima and sums each: a single chain of 64 dependent operations would cost its latency 64 times
             float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -401,7 +452,6 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
             m = fmaxf(m, mx * p.scale_log2);
             // The reference follows the maximum only when it lags too far behind: then this row of O and the row's sum are
             // scaled down. The first keys a row sees set its reference for free (everything so far was zero).
-            float corr = 1.f;
             bool rescale = false;
             if (ref == -INFINITY) {
                 ref = m;
@@ -447,14 +497,16 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 s[j] = __float_as_uint(fast_exp2(x0));
                 s[j + 1] = __float_as_uint(fast_exp2(x1));
             }
-            uint64_t sum2[2] = {pair_of(0.f, 0.f), pair_of(0.f, 0.f)};
+            }
 #pragma unroll
             for (int j = 0; j < BN; j += 8) {
                 float e[8];
 #pragma unroll
                 for (int i = 0; i < 8; ++i) e[i] = __uint_as_float(s[j + i]);
-                sum2[0] = add2(add2(sum2[0], pair_of(e[0], e[1])), pair_of(e[4], e[5]));
-                sum2[1] = add2(add2(sum2[1], pair_of(e[2], e[3])), pair_of(e[6], e[7]));
+                if constexpr (!SIG) {
+                    sum2[0] = add2(add2(sum2[0], pair_of(e[0], e[1])), pair_of(e[4], e[5]));
+                    sum2[1] = add2(add2(sum2[1], pair_of(e[2], e[3])), pair_of(e[6], e[7]));
+                }
                 uint4 packed;
                 packed.x = pack_bf16x2(e[0], e[1]); packed.y = pack_bf16x2(e[2], e[3]);
                 packed.z = pack_bf16x2(e[4], e[5]); packed.w = pack_bf16x2(e[6], e[7]);
@@ -466,10 +518,12 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
             tmem_st16(lane_base + (c % S_BUFS) * BN, s);
             tmem_st16(lane_base + (c % S_BUFS) * BN + 16, s + 16);
             asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
-            float sum4[4];
-            unpair(sum2[0], sum4[0], sum4[1]);
-            unpair(sum2[1], sum4[2], sum4[3]);
-            l = l * corr + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
+            if constexpr (!SIG) {
+                float sum4[4];
+                unpair(sum2[0], sum4[0], sum4[1]);
+                unpair(sum2[1], sum4[2], sum4[3]);
+                l = l * corr + ((sum4[0] + sum4[1]) + (sum4[2] + sum4[3]));
+            }
             if (key0 + BN > hi) {
                 // the chunk reaches behind the last key: those value rows may hold anything; they become zeros
                 unsigned char* v_c = v_s + (c % STAGES) * K_BYTES;
@@ -511,23 +565,40 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
         }
         const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll 1
-        for (int part = 0; part < D && ok; part += 64) {
+        for (int part = 0; part < D / 2 && ok; part += 32) {   // 32 entries of either half: both partners of every pair that may turn
             float o[64];
 #pragma unroll
             for (int i = 0; i < 64; ++i) o[i] = 0.f;
             if (chunks > 0) {
                 uint32_t v[64];
 #pragma unroll
-                for (int j = 0; j < 64; j += 16) tmem_ld16(o_addr + part + j, v + j);
+                for (int j = 0; j < 64; j += 16) tmem_ld16(o_addr + (j < 32 ? part + j : D / 2 + part + j - 32), v + j);
                 asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
 #pragma unroll
                 for (int i = 0; i < 64; ++i) o[i] = __uint_as_float(v[i]);
             }
+            if (p.turn_cos && row_ok) {
+                const float* tc = p.turn_cos + (size_t)(n0 + tok) * (D / 2) + part;
+                const float* ts = p.turn_sin + (size_t)(n0 + tok) * (D / 2) + part;
+#pragma unroll
+                for (int i = 0; i < 32; i += 4) {
+                    float cs[4], sn[4];
+                    load4(tc + i, cs);
+                    load4(ts + i, sn);
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        const float a = o[i + k], b = o[32 + i + k];
+                        o[i + k] = fmaf(b, sn[k], a * cs[k]);
+                        o[32 + i + k] = fmaf(-a, sn[k], b * cs[k]);
+                    }
+                }
+            }
             if (num_splits == 1) {
                 if (row_ok) {
-                    uint4* dst = reinterpret_cast<uint4*>(p.out + (size_t)(n0 + tok) * p.nq * D + (size_t)(kvh * G + row % G) * D + part);
+                    bf16* row_out = p.out + (size_t)(n0 + tok) * p.nq * D + (size_t)(kvh * G + row % G) * D + part;
 #pragma unroll
                     for (int j = 0; j < 8; ++j) {
+                        uint4* dst = reinterpret_cast<uint4*>(row_out + (j < 4 ? 0 : D / 2 - 32));
                         uint4 packed;
                         packed.x = pack_bf16x2(o[8 * j] * inv, o[8 * j + 1] * inv); packed.y = pack_bf16x2(o[8 * j + 2] * inv, o[8 * j + 3] * inv);
                         packed.z = pack_bf16x2(o[8 * j + 4] * inv, o[8 * j + 5] * inv); packed.w = pack_bf16x2(o[8 * j + 6] * inv, o[8 * j + 7] * inv);
@@ -536,7 +607,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 }
             } else {
 #pragma unroll
-                for (int i = 0; i < 64; i += 4) *reinterpret_cast<float4*>(fo + row * D + part + i) = make_float4(o[i], o[i + 1], o[i + 2], o[i + 3]);
+                for (int i = 0; i < 64; i += 4) *reinterpret_cast<float4*>(fo + row * D + (i < 32 ? part + i : D / 2 + part + i - 32)) = make_float4(o[i], o[i + 1], o[i + 2], o[i + 3]);
             }
         }
     }
@@ -682,12 +753,16 @@ LLMIE_API int llmie_attn_tc_plan(const int* tile_info, int num_tiles, const int*
 // [pages][nkv][page_size][d]. `work` is the plan that llmie_attn_tc_plan made for the step's num_tiles tiles, its positions,
 // this window and page size, with the same max_items. The slices of a tile meet in scratch_o [max_items * nkv * 128 * d]
 // and scratch_ml [max_items * nkv * 128 * 2] floats; the block that finishes a tile last (counters [tiles * nkv], zero before and
-// after) merges them.
+// after) merges them. turn_cos / turn_sin: [tokens][d / 2], 16-byte aligned, or null; sig_bias (or null), log_r1, log_r2 (or null): [nq].
 LLMIE_API int llmie_paged_attention_tc(const bf16* q, int q_stride, const bf16* k_pool, const bf16* v_pool, long long pool_pages,
                                        const int* block_table, int max_blocks, int num_tiles, const int* work, int max_items, bf16* out, float* scratch_o,
                                        float* scratch_ml, int* counters, int nq, int nkv, int d, int page_size, float scale, int window,
-                                       int* error_flag, cudaStream_t s) {
+                                       int* error_flag, const float* turn_cos, const float* turn_sin, const float* sig_bias, const float* log_r1,
+                                       const float* log_r2, cudaStream_t s) {
     if (num_tiles <= 0) return 0;
+    if ((turn_cos == nullptr) != (turn_sin == nullptr) || ((uintptr_t)turn_cos & 15) || ((uintptr_t)turn_sin & 15) || (log_r1 == nullptr) != (log_r2 == nullptr) ||
+        (log_r1 && !sig_bias))
+        return LLMIE_ERR_BAD_ARGUMENT;
     if ((d != 64 && d != 128) || nkv <= 0 || nq % nkv || nq / nkv > BM || page_size <= 0 || page_size % 8 || q_stride % 8 ||
         !(BN % page_size == 0 || page_size % BN == 0) || !error_flag || pool_pages <= 0 || ((uintptr_t)q & 15) ||
         ((uintptr_t)out & 15) || pool_pages * nkv * page_size > 0x7fffffffLL || !work || ((uintptr_t)work & 15) || max_items < num_tiles ||
@@ -698,6 +773,7 @@ LLMIE_API int llmie_paged_attention_tc(const bf16* q, int q_stride, const bf16* 
     p.out = out; p.error_flag = error_flag; p.part_o = scratch_o; p.part_ml = scratch_ml; p.counters = counters; p.max_items = max_items;
     p.q_stride = q_stride; p.max_blocks = max_blocks; p.nq = nq; p.nkv = nkv; p.page_size = page_size; p.num_tiles = num_tiles;
     p.window = window; p.box_rows = page_size < BN ? page_size : BN; p.scale_log2 = scale * LOG2E;
+    p.turn_cos = turn_cos; p.turn_sin = turn_sin; p.sig_bias = sig_bias; p.log_r1 = log_r1; p.log_r2 = log_r2;
     CUtensorMap mk, mv;
     const int rows = (int)(pool_pages * nkv * page_size);
     int rc = tensor_map(k_pool, rows, d, p.box_rows, &mk);
@@ -706,7 +782,7 @@ LLMIE_API int llmie_paged_attention_tc(const bf16* q, int q_stride, const bf16* 
     if (rc) return rc;
     const long long blocks = (long long)max_items * nkv;
     if (blocks > 0x7fffffffLL) return LLMIE_ERR_BAD_ARGUMENT;
-    static bool set[2] = {false, false};
+    static bool set[4] = {false, false, false, false};
     auto launch = [&](auto kernel, size_t smem, int which) -> int {
         if (!set[which]) {
             cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -715,5 +791,6 @@ LLMIE_API int llmie_paged_attention_tc(const bf16* q, int q_stride, const bf16* 
         }
         return launch_kernel(kernel, dim3((unsigned)blocks), dim3(THREADS), smem, s, mk, mv, p);
     };
-    return d == 64 ? launch(attn_tc_prefill_kernel<64>, Sizes<64>::SMEM, 0) : launch(attn_tc_prefill_kernel<128>, Sizes<128>::SMEM, 1);
+    if (sig_bias) return d == 64 ? launch(attn_tc_prefill_kernel<64, true>, Sizes<64>::SMEM, 2) : launch(attn_tc_prefill_kernel<128, true>, Sizes<128>::SMEM, 3);
+    return d == 64 ? launch(attn_tc_prefill_kernel<64, false>, Sizes<64>::SMEM, 0) : launch(attn_tc_prefill_kernel<128, false>, Sizes<128>::SMEM, 1);
 }

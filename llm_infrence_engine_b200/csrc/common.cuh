@@ -92,6 +92,10 @@ __device__ __forceinline__ void store4(bf16* p, const float* v) {
     *reinterpret_cast<uint2*>(p) = t;
 }
 
+// 2^v and log2(v) by the hardware's approximation unit (errors of about 1e-7 of the result), denormals flushed.
+__device__ __forceinline__ float hw_exp2(float v) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(v)); return y; }
+__device__ __forceinline__ float hw_log2(float v) { float y; asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(v)); return y; }
+
 static inline int launch_status() {
     return (int)cudaGetLastError();
 }

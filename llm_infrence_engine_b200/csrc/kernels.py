@@ -70,6 +70,9 @@ class CudaKernels:
         # more rows); measured slower at 2,048 tokens (heads of 128: 311 -> 415 us): their registers leave one block per
         # multiprocessor where tiles of 32 rows leave two, and the kernel waits on its barriers, not on the keys
         self.attention_ext_tile_rows = 32
+        # attention with no extras but sigmoid weights, a penalty by distance with them, or values that are turned back: heads of 64 or 128
+        # take the kernels of plain attention (tcgen05 for steps with prompt portions, the decode kernel for single tokens)
+        self.use_plain_attention_for_ext = True
         self.masked_attention_tensor_cores = True    # kept first tokens, chunks and soft caps on the tensor-core kernels too
         self.use_fa_attention_ext = True     # prompt portions with heads of 64 / 128: the kernel in which a warp owns 16 rows and all keys of a chunk
         self.use_mma_attention_talk = True   # heads that talk, steps with prompt portions in bfloat16: plain scores and P V on the tensor cores
@@ -629,8 +632,9 @@ class CudaKernels:
         return tiles, batch._tables[key]
 
     def _attention_tc(self, qkv, k_pool, v_pool, block_table, token_seq, positions, out, num_heads, num_kv_heads, head_dim,
-                      page_size, scale, window, span, batch, num_splits):
-        """The tcgen05 kernel for prompt portions, if it takes this case: returns ``out`` or None."""
+                      page_size, scale, window, span, batch, num_splits, turn=None, sigmoid_bias=None, log_distance=None):
+        """The tcgen05 kernel for prompt portions, if it takes this case: returns ``out`` or None. (``turn``, ``sigmoid_bias``,
+        ``log_distance``: see ``attention_ext``.)"""
         group = num_heads // num_kv_heads
         if not (self.use_tc_attention and head_dim in (64, 128) and batch.max_seq_len > 1 and group <= 128 and page_size % 8 == 0
                 and (64 % page_size == 0 or page_size % 64 == 0) and (num_splits is None or 1 <= num_splits <= 16)):
@@ -662,8 +666,15 @@ class CudaKernels:
             _ptr(qkv), qkv.shape[1], _ptr(k_pool), _ptr(v_pool), ctypes.c_longlong(k_pool.shape[0]), _ptr(block_table),
             block_table.shape[1], tiles, _ptr(work), max_items, _ptr(out),
             _ptr(scratch_o), _ptr(scratch_ml), _ptr(self._attn_counters), num_heads, num_kv_heads, head_dim, page_size,
-            ctypes.c_float(scale), int(window), _ptr(self._errors(qkv.device)), self._stream()), "paged_attention (tcgen05)")
+            ctypes.c_float(scale), int(window), _ptr(self._errors(qkv.device)), *self._turn_and_sigmoid(turn, sigmoid_bias, log_distance),
+            self._stream()), "paged_attention (tcgen05)")
         return out
+
+    @staticmethod
+    def _turn_and_sigmoid(turn, sigmoid_bias, log_distance) -> tuple:
+        cos, sin = (None, None) if turn is None else turn[:2]
+        r1, r2 = (None, None) if log_distance is None else log_distance
+        return _ptr(cos), _ptr(sin), _ptr(sigmoid_bias), _ptr(r1), _ptr(r2)
 
     def _decode_plan(self, tokens, num_kv_heads, head_dim, span, num_splits, device):
         return self._slices(tokens, num_kv_heads, head_dim, span, num_splits, True, device)
@@ -712,15 +723,17 @@ class CudaKernels:
         return num_splits, cluster, scratch_o, scratch_ml, counters
 
     def _attention_mma(self, qkv, k_pool, v_pool, block_table, token_seq, positions, out, num_heads, num_kv_heads, head_dim,
-                       page_size, scale, window, span, batch, num_splits):
+                       page_size, scale, window, span, batch, num_splits, turn=None, sigmoid_bias=None, log_distance=None):
         group = num_heads // num_kv_heads
         decode = batch.max_seq_len == 1
         N = qkv.shape[0]
         if not decode:
             done = self._attention_tc(qkv, k_pool, v_pool, block_table, token_seq, positions, out, num_heads, num_kv_heads, head_dim,
-                                      page_size, scale, window, span, batch, num_splits)
+                                      page_size, scale, window, span, batch, num_splits, turn, sigmoid_bias, log_distance)
             if done is not None:
                 return done
+            if turn is not None or sigmoid_bias is not None:
+                return None   # (the mma.sync kernel for prompt portions knows neither)
         if decode:
             tile_info = None
             num_splits, cluster, scratch_o, scratch_ml, counters = self._decode_plan(N, num_kv_heads, head_dim, span, num_splits, qkv.device)
@@ -732,7 +745,8 @@ class CudaKernels:
             _ptr(qkv), qkv.shape[1], _ptr(k_pool), _ptr(v_pool), _ptr(block_table), block_table.shape[1], _ptr(token_seq),
             _ptr(positions), _ptr(tile_info), tiles, _ptr(out), _ptr(scratch_o), _ptr(scratch_ml), _ptr(counters), num_heads,
             num_kv_heads, head_dim, page_size, ctypes.c_float(scale), int(window), num_splits,
-            2 if (decode and self._decode_four_warps) else int(decode), cluster, self._stream()),
+            2 if (decode and self._decode_four_warps) else int(decode), cluster,
+            *self._turn_and_sigmoid(turn, sigmoid_bias, log_distance), self._stream()),
             "paged_attention (tensor cores)")
         return out
 
@@ -1069,6 +1083,16 @@ class CudaKernels:
             return self._attention_talk(q, q_col, num_heads, num_kv_heads, head_dim, v_head_dim, k_pool, v_pool, block_table, token_seq, positions,
                                         page_size, scale, window, max_context, talk, sink, gate, gate_col, gate_mode, keep_first, chunk, softcap,
                                         temp, rel, out, batch)
+        if keep_first < 0 or chunk < 0 or softcap < 0 or (keep_first and not window):
+            raise KernelError("attention_ext: keep_first needs a window, and keep_first, chunk and softcap cannot be negative")
+        if (self.use_plain_attention_for_ext and self.use_mma_attention and dt == 1 and batch is not None and v_pool is not None and head_dim == v_head_dim
+                and head_dim in (64, 128) and q_col == 0 and q.shape[1] % 8 == 0 and not (keep_first or chunk or softcap or temp[1]) and rel is None
+                and sink is None and gate is None and (turn is None or not turn[2]) and (log_distance is None or sigmoid_bias is not None) and scale > 0
+                and num_heads // num_kv_heads <= (16 if batch.max_seq_len == 1 else 64) and (num_splits is None or num_splits <= 16)):
+            done = self._attention_mma(q, k_pool, v_pool, block_table, token_seq, positions, out, num_heads, num_kv_heads, head_dim, page_size, scale,
+                                       int(window), min(max_context, window) if window else max_context, batch, num_splits, turn, sigmoid_bias, log_distance)
+            if done is not None:
+                return done
         max_rows = 0
         tensor_cores = dt == 1 and self.use_mma_attention_ext and batch is not None and (q_col * esize) % 16 == 0 and q.shape[1] % 8 == 0
         masked = bool(keep_first or chunk or softcap)
@@ -1076,8 +1100,6 @@ class CudaKernels:
             tensor_cores = False   # (the tensor-core kernels know sigmoid weights under a causal mask and a window)
         if masked and not self.masked_attention_tensor_cores:
             tensor_cores = False
-        if keep_first < 0 or chunk < 0 or softcap < 0 or (keep_first and not window):
-            raise KernelError("attention_ext: keep_first needs a window, and keep_first, chunk and softcap cannot be negative")
         if (tensor_cores and self.use_fa_attention_ext and batch.max_seq_len > 1
                 and self.lib.llmie_attention_ext_fa_fits(head_dim, v_head_dim, int(v_pool is not None), num_heads // num_kv_heads)):
             # steps with prompt portions, heads of 64 or 128: tiles of 64 rows, a warp to 16 rows and all of a chunk's keys

@@ -201,37 +201,42 @@ def paged(N_ctx, page, nkv, dk, dv, dtype, seed=0):
     return k_pool, v_pool, table, k, v
 
 
-WAYS = ("generic", "portion", "portion, split-part kernel", "single tokens", "two equal runs", "single tokens, five runs")
+WAYS = ("generic", "portion", "portion, warp-to-rows kernel", "portion, split-part kernel", "single tokens", "single tokens, split-part kernel", "two equal runs",
+        "single tokens, five runs", "single tokens, five runs, split-part kernel")
 
 
 def run_attention(K, how, q, q_col, common, seq, pos, page, scale, window, ctx_len, **kw):
     """``attention_ext`` by one of the ways its kernels are reached."""
     N = q.shape[0]
     batch, more = None, {}
-    if how.startswith("portion") or how == "two equal runs":
-        batch = SimpleNamespace(seq_lens=[N], seq_starts_dev=torch.tensor([0, N], dtype=torch.int32).cuda(), max_seq_len=N, _tables={})
+    if how.startswith("portion") or how == "two equal runs":     # a portion holds neighbouring positions: one per run of them
+        starts = [0] + [i for i in range(1, N) if int(pos[i]) != int(pos[i - 1]) + 1] + [N]
+        lens = [b - a for a, b in zip(starts, starts[1:])]
+        batch = SimpleNamespace(seq_lens=lens, seq_starts_dev=torch.tensor(starts, dtype=torch.int32).cuda(), max_seq_len=max(lens), _tables={})
     if how.startswith("single"):
         batch = SimpleNamespace(seq_lens=[1] * N, seq_starts_dev=torch.arange(N + 1, dtype=torch.int32).cuda(), max_seq_len=1, _tables={})
     if how == "two equal runs":
         more = {"num_splits": 2}
-    if how.endswith("five runs"):
+    if "five runs" in how:
         more = {"num_splits": 5}
-    K.use_fa_attention_ext = how != "portion, split-part kernel"
+    K.use_fa_attention_ext = not how.endswith("split-part kernel")
+    K.use_plain_attention_for_ext = not how.endswith("kernel")
     try:
         return K.attention_ext(q.cuda(), q_col, *common, seq.cuda(), pos.cuda(), page, scale, window, ctx_len, batch=batch, **kw, **more)
     finally:
-        K.use_fa_attention_ext = True
+        K.use_fa_attention_ext = K.use_plain_attention_for_ext = True
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("nq,nkv,dk,dv", [(4, 2, 16, 8), (6, 1, 64, 64), (4, 2, 96, 96), (3, 3, 24, 40), (4, 4, 128, 128), (16, 4, 128, 64), (2, 1, 64, 128),
+@pytest.mark.parametrize("nq,nkv,dk,dv", [(4, 2, 16, 8), (6, 1, 64, 64), (4, 2, 96, 96), (3, 3, 24, 40), (4, 4, 128, 128), (16, 4, 128, 64), (2, 1, 64, 128), (14, 2, 64, 64), (16, 1, 128, 128), (12, 1, 64, 64), (40, 2, 128, 128),
                                           (5, 1, 48, 256), (3, 3, 10, 6)])
 def test_attention_sigmoid_penalty_and_turned_values(K, dtype, nq, nkv, dk, dv):
     """Positions spread over a request of 1,300 tokens, as a prompt portion and as single tokens; every kernel that takes the sizes."""
     ctx_len, page = 1300, 16
     k_pool, v_pool, table, _, _ = paged(ctx_len, page, nkv, dk, dv, dtype, 3)
-    pos = torch.tensor([0, 1, 5, 15, 16, 17, 100, 199, 200, 201, 1023, 1024, 1025, 1299] + list(range(1180, 1299, 4)), dtype=torch.int32).sort().values
+    pos = torch.tensor([0, 1, 5, 15, 16, 17, 100, 199, 200, 201, 1023, 1024, 1025] + list(range(1180, 1213)) + [1299], dtype=torch.int32)
     N = pos.shape[0]
+    col = 0 if dk in (64, 128) else 8      # (the kernels of plain attention take rows that begin with the queries)
     q = rnd(N, nq * dk + 8, seed=5, scale=0.5).to(TD[dtype])
     seq = torch.ones(N, dtype=torch.int32)
     pb, r1, r2 = rnd(nq, seed=6) - 2.0, rnd(nq, seed=7).abs() + 0.2, rnd(nq, seed=8).abs() + 0.1
@@ -251,10 +256,10 @@ def test_attention_sigmoid_penalty_and_turned_values(K, dtype, nq, nkv, dk, dv):
     }
     dev = lambda v: tuple(dev(t) for t in v) if isinstance(v, tuple) else (v.cuda() if torch.is_tensor(v) else v)
     for what, (window, kw) in variants.items():
-        want = TorchKernels().attention_ext(q, 8, nq, nkv, dk, dv, k_pool, v_pool, table, seq, pos, page, 0.3, window, ctx_len, **kw)
+        want = TorchKernels().attention_ext(q, col, nq, nkv, dk, dv, k_pool, v_pool, table, seq, pos, page, 0.3, window, ctx_len, **kw)
         top = float(want.float().abs().max())
         for how in WAYS:
-            got = run_attention(K, how, q, 8, (nq, nkv, dk, dv, k_pool.cuda(), v_pool.cuda(), table.cuda()), seq, pos, page, 0.3, window, ctx_len,
+            got = run_attention(K, how, q, col, (nq, nkv, dk, dv, k_pool.cuda(), v_pool.cuda(), table.cuda()), seq, pos, page, 0.3, window, ctx_len,
                                 **{k: dev(v) for k, v in kw.items()})
             # (softmax results are of size 1; sums of sigmoid weights over a thousand keys have a size of their own)
             close(got, want, dtype, f"attention_ext {what} ({how})", scale=8.0 * max(1.0, dk / 64) ** 0.5 * max(1.0, top / 4) if dtype == "float32" else None)
