@@ -96,6 +96,38 @@ __device__ __forceinline__ void store4(bf16* p, const float* v) {
 __device__ __forceinline__ float hw_exp2(float v) { float y; asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(v)); return y; }
 __device__ __forceinline__ float hw_log2(float v) { float y; asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(v)); return y; }
 
+// z times the normal distribution's share below z (the exact GELU) for results that are rounded to bfloat16: the share beyond |z| is
+// t (a1 + t (a2 + ... + t a5)) e^(-z^2 / 2) / 2 with t = 1 / (1 + p |z| / sqrt 2), Abramowitz and Stegun, Handbook of Mathematical
+// Functions, 7.1.26 (an error of at most 1.5e-7 in erf).
+__device__ __forceinline__ float gelu_erf_fast(float z) {
+    const float a = fabsf(z);
+    const float t = __fdividef(1.0f, fmaf(0.3275911f * 0.7071067811865476f, a, 1.0f));
+    float h = fmaf(t, 0.5f * 1.061405429f, 0.5f * -1.453152027f);
+    h = fmaf(h, t, 0.5f * 1.421413741f);
+    h = fmaf(h, t, 0.5f * -0.284496736f);
+    h = fmaf(h, t, 0.5f * 0.254829592f);
+    h = h * t * hw_exp2(-0.7213475204444817f * z * z);
+    return fmaf(-a, h, fmaxf(z, 0.0f));
+}
+// The tanh form, 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), likewise (tanh(t) = 1 - 2 / (exp(2 t) + 1)).
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+    const float t = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+    return z * (1.0f - __fdividef(1.0f, __expf(2.0f * t) + 1.0f));
+}
+
+// What a feed-forward's first product ends in; a compile-time choice, so that an epilogue's elements stand in one straight run of
+// instructions (a branch per element, even a uniform one, would leave nothing to overlap their latencies with).
+enum { UNIT_SILU = 0, UNIT_CLAMPED = 1, UNIT_GELU_TANH = 2, PLAIN_GELU_ERF = 3, PLAIN_GELU_TANH = 4 };
+template <int UNIT>
+__device__ __forceinline__ float gated_unit(float g, float u, float limit, float alpha, float shift) {
+    if constexpr (UNIT == UNIT_GELU_TANH) return gelu_tanh_fast(g) * u;
+    if constexpr (UNIT == UNIT_CLAMPED) {   // min(g, limit) * sigmoid(alpha g) * (clamp(u) + shift)
+        const float c = fminf(g, limit);
+        return __fdividef(c, 1.0f + __expf(-alpha * c)) * (fminf(fmaxf(u, -limit), limit) + shift);
+    }
+    return __fdividef(g, 1.0f + __expf(-g)) * u;
+}
+
 static inline int launch_status() {
     return (int)cudaGetLastError();
 }

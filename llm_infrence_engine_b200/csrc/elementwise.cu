@@ -581,6 +581,13 @@ LLMIE_API int llmie_kv_store(const void* z, int z_stride, int k_col, int v_col, 
 // out = act(in), elementwise in 32-bit. kind 0: the tanh form of GELU, 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)));
 // kind 1: a soft cap on a scaled input, param * tanh(scale z / param); kind 2: the exact GELU, 0.5 z (1 + erf(z / sqrt 2)); kind 3: scale z.
 // With `clear_in` the input is set to zero after it was read (a float32 accumulation buffer of a split-K product).
+__device__ __forceinline__ float act_of(float z, int kind, float param, float scale) {
+    if (kind == 1) return param * tanhf(scale * z / param);
+    if (kind == 2) return 0.5f * z * (1.0f + erff(0.7071067811865476f * z));
+    if (kind == 3) return scale * z;
+    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+
 template <typename TI, typename TO>
 __global__ void act_kernel(TI* __restrict__ in, TO* __restrict__ out, long long total, int kind, int clear_in, float param, float scale) {
     pdl_trigger();
@@ -589,16 +596,33 @@ __global__ void act_kernel(TI* __restrict__ in, TO* __restrict__ out, long long 
     if (i >= total) return;
     const float z = to_f32(in[i]);
     if (clear_in) in[i] = from_f32<TI>(0.f);
-    float y;
-    if (kind == 1) y = param * tanhf(scale * z / param);
-    else if (kind == 2) y = 0.5f * z * (1.0f + erff(0.7071067811865476f * z));
-    else if (kind == 3) y = scale * z;
-    else y = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-    out[i] = from_f32<TO>(y);
+    out[i] = from_f32<TO>(act_of(z, kind, param, scale));
+}
+
+// float in, four elements (16 bytes) per thread. Results that are rounded to bfloat16 take the fast forms of the activations.
+template <typename TO>
+__global__ void __launch_bounds__(128) act_vec_kernel(float* __restrict__ in, TO* __restrict__ out, long long items, int kind, int clear_in, float param,
+                                                      float scale) {
+    pdl_trigger();
+    pdl_wait();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= items) return;
+    float z[4];
+    load4(in + i * 4, z);
+    if (clear_in) {
+        const float zero[4] = {0.f, 0.f, 0.f, 0.f};
+        store4(in + i * 4, zero);
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+        if constexpr (sizeof(TO) == 2) z[j] = kind == 2 ? gelu_erf_fast(z[j]) : (kind == 0 ? gelu_tanh_fast(z[j]) : act_of(z[j], kind, param, scale));
+        else z[j] = act_of(z[j], kind, param, scale);
+    }
+    store4(out + i * 4, z);
 }
 
 // bfloat16 in and out, 8 elements (16 bytes) per thread. The result is rounded to bfloat16 (8 bits), so the hyperbolic tangent is
-// the fast 32-bit form (tanh(a) = 1 - 2 / (exp(2a) + 1), errors of about 1e-7). ERF: the exact GELU instead.
+// the fast 32-bit form (errors of about 1e-7). ERF: the exact GELU instead.
 template <bool ERF>
 __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict__ in, bf16* __restrict__ out, long long items) {
     pdl_trigger();
@@ -615,10 +639,7 @@ __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict_
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
             const float v = z[2 * j + k];
-            if (ERF) { y[k] = 0.5f * v * (1.0f + erff(0.7071067811865476f * v)); continue; }
-            const float a = 0.7978845608028654f * (v + 0.044715f * v * v * v);
-            const float t = 1.0f - __fdividef(2.0f, __expf(2.0f * a) + 1.0f);
-            y[k] = 0.5f * v * (1.0f + t);
+            y[k] = ERF ? gelu_erf_fast(v) : gelu_tanh_fast(v);
         }
         const __nv_bfloat162 v2 = __floats2bfloat162_rn(y[0], y[1]);
         w[j] = *reinterpret_cast<const uint32_t*>(&v2);
@@ -634,6 +655,11 @@ LLMIE_API int llmie_act(void* in, void* out, long long total, int kind, int clea
         const dim3 blocks((unsigned)((total / 8 + 255) / 256));
         if (kind == 2) return launch_kernel(act_bf16x8_kernel<true>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
         return launch_kernel(act_bf16x8_kernel<false>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
+    }
+    if (in_dtype == DT_F32 && total % 4 == 0 && ((uintptr_t)in % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
+        const dim3 blocks((unsigned)((total / 4 + 127) / 128));
+        if (out_dtype == DT_F32) return launch_kernel(act_vec_kernel<float>, blocks, dim3(128), 0, s, (float*)in, (float*)out, total / 4, kind, clear_in, param, scale);
+        return launch_kernel(act_vec_kernel<bf16>, blocks, dim3(128), 0, s, (float*)in, (bf16*)out, total / 4, kind, clear_in, param, scale);
     }
     const dim3 grid((unsigned)((total + 255) / 256));
     if (in_dtype == DT_F32 && out_dtype == DT_F32) return launch_kernel(act_kernel<float, float>, grid, dim3(256), 0, s, (float*)in, (float*)out, total, kind, clear_in, param, scale);

@@ -27,7 +27,10 @@ namespace {
 
 constexpr int BM = 128, BK = 64, UMMA_K = 16;
 constexpr int A_BYTES = BM * BK * 2;
-constexpr int EPI_THREADS = 128, THREADS = 64 + EPI_THREADS;
+// The epilogue's warps: four, or eight where a plain product's activation is applied to every sum (two warps to the same 32 lanes of
+// tensor memory then, taking 16 columns in turn: one warp waits for its exponentials and divisions one after the other).
+template <bool PLAIN> constexpr int EPI_THREADS = PLAIN ? 256 : 128;
+template <bool PLAIN> constexpr int THREADS = 64 + EPI_THREADS<PLAIN>;
 
 __device__ __forceinline__ uint32_t cluster_address_of(const void* own_smem, uint32_t rank) {
     uint32_t r;
@@ -56,10 +59,13 @@ __device__ __forceinline__ void cluster_sync_all() {
     asm volatile("barrier.cluster.wait.acquire.aligned;\n" ::: "memory");
 }
 
-template <int BN, int STAGES>
-__global__ void __launch_bounds__(THREADS) gateup_silu_tc_pair_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
+// UNIT: what the epilogue computes (common.cuh). PLAIN_...: a plain product with an activation instead of a gated one. The matrix [2 I, K] is taken as two halves of output columns side
+// by side: the activation of the first half's sums goes to columns n of rows of 2 I, that of the second half's to columns I + n.
+template <int BN, int STAGES, int UNIT>
+__global__ void __launch_bounds__(THREADS<(UNIT >= PLAIN_GELU_ERF)>) gateup_silu_tc_pair_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
                                                                        bf16* __restrict__ out, int M, int I, int K, int* error_flag, float limit, float alpha, float shift) {
     constexpr int B_BYTES = BN * BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;   // this block's half of the weight rows of a K step
+    constexpr bool PLAIN = UNIT >= PLAIN_GELU_ERF;
     extern __shared__ unsigned char raw[];
     unsigned char* tiles = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
     uint64_t* full = reinterpret_cast<uint64_t*>(tiles + STAGES * STAGE_BYTES);  // used in the leader only
@@ -78,7 +84,7 @@ __global__ void __launch_bounds__(THREADS) gateup_silu_tc_pair_kernel(const __gr
 
     if (tid == 0) {
         for (int s = 0; s < STAGES; ++s) { mbar_init(full + s, 1); mbar_init(empty + s, 1); }
-        for (int s = 0; s < 2; ++s) { mbar_init(acc_full + s, 1); mbar_init(acc_free + s, 2 * (EPI_THREADS / 32)); }
+        for (int s = 0; s < 2; ++s) { mbar_init(acc_full + s, 1); mbar_init(acc_free + s, 2 * (EPI_THREADS<PLAIN> / 32)); }
         *abort_flag = 0;
         *issued = 0;
         asm volatile("fence.mbarrier_init.release.cluster;\n" ::: "memory");
@@ -155,32 +161,37 @@ __global__ void __launch_bounds__(THREADS) gateup_silu_tc_pair_kernel(const __gr
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
             const uint32_t base = tmem + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(buf * 2 * BN);
-            bf16* dst = out + (size_t)m * I + n0;
+            bf16* dst = out + (size_t)m * (PLAIN ? 2 * I : I) + n0;
 #pragma unroll 2
-            for (int c = 0; c < BN; c += 16) {
+            for (int c = PLAIN ? ((warp - 2) >> 2) * 16 : 0; c < BN; c += PLAIN ? 32 : 16) {
                 uint32_t gv[16], uv[16];
                 tmem_ld16(base + c, gv);
                 tmem_ld16(base + BN + c, uv);
                 asm volatile("tcgen05.wait::ld.sync.aligned;\n" ::: "memory");
+                if constexpr (PLAIN) {
+#pragma unroll
+                    for (int half = 0; half < 2; ++half) {
+                        uint32_t packed[8];
+#pragma unroll
+                        for (int j = 0; j < 8; ++j) {
+                            const float z0 = __uint_as_float(half ? uv[2 * j] : gv[2 * j]), z1 = __uint_as_float(half ? uv[2 * j + 1] : gv[2 * j + 1]);
+                            const __nv_bfloat162 v = UNIT == PLAIN_GELU_TANH ? __floats2bfloat162_rn(gelu_tanh_fast(z0), gelu_tanh_fast(z1))
+                                                                            : __floats2bfloat162_rn(gelu_erf_fast(z0), gelu_erf_fast(z1));
+                            packed[j] = *reinterpret_cast<const uint32_t*>(&v);
+                        }
+                        if (m < M) {
+                            bf16* d2 = dst + (half ? I : 0) + c;
+                            if (n0 + c + 8 <= I) *reinterpret_cast<uint4*>(d2) = make_uint4(packed[0], packed[1], packed[2], packed[3]);
+                            if (n0 + c + 16 <= I) *reinterpret_cast<uint4*>(d2 + 8) = make_uint4(packed[4], packed[5], packed[6], packed[7]);
+                        }
+                    }
+                    continue;
+                }
                 uint32_t packed[8];
 #pragma unroll
                 for (int j = 0; j < 8; ++j) {
-                    const float g0 = __uint_as_float(gv[2 * j]), g1 = __uint_as_float(gv[2 * j + 1]);
-                    float u0 = __uint_as_float(uv[2 * j]), u1 = __uint_as_float(uv[2 * j + 1]), a, b;
-                    if (limit < 0.f) {   // the GELU unit (tanh form, tanh(t) = 1 - 2 / (exp(2t) + 1)): 0.5 g (1 + tanh(c (g + 0.044715 g^3))) * u
-                        const float t0 = 0.7978845608028654f * (g0 + 0.044715f * g0 * g0 * g0), t1 = 0.7978845608028654f * (g1 + 0.044715f * g1 * g1 * g1);
-                        a = g0 * (1.0f - __fdividef(1.0f, __expf(2.0f * t0) + 1.0f)) * u0;
-                        b = g1 * (1.0f - __fdividef(1.0f, __expf(2.0f * t1) + 1.0f)) * u1;
-                    } else if (limit > 0.f) {   // the clamped unit: min(g, limit) * sigmoid(alpha g) * (clamp(u) + shift)
-                        const float c0 = fminf(g0, limit), c1 = fminf(g1, limit);
-                        u0 = fminf(fmaxf(u0, -limit), limit) + shift;
-                        u1 = fminf(fmaxf(u1, -limit), limit) + shift;
-                        a = __fdividef(c0, 1.0f + __expf(-alpha * c0)) * u0;
-                        b = __fdividef(c1, 1.0f + __expf(-alpha * c1)) * u1;
-                    } else {
-                        a = __fdividef(g0, 1.0f + __expf(-g0)) * u0;
-                        b = __fdividef(g1, 1.0f + __expf(-g1)) * u1;
-                    }
+                    const float a = gated_unit<UNIT>(__uint_as_float(gv[2 * j]), __uint_as_float(uv[2 * j]), limit, alpha, shift);
+                    const float b = gated_unit<UNIT>(__uint_as_float(gv[2 * j + 1]), __uint_as_float(uv[2 * j + 1]), limit, alpha, shift);
                     const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
                     packed[j] = *reinterpret_cast<const uint32_t*>(&v);
                 }
@@ -224,7 +235,7 @@ inline int best_tile_width(long long m_pairs, int I, int pairs_at_once) {
     return best;
 }
 
-template <int BN>
+template <int BN, int UNIT>
 int launch_gateup_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, int K, int num_blocks, int* error_flag, float limit, float alpha,
                   float shift, cudaStream_t s) {
     constexpr int STAGES = BN > 96 ? 6 : 7;   // 32 KB (BN = 128) to 24 KB (BN = 64) per stage
@@ -236,7 +247,7 @@ int launch_gateup_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, in
     constexpr size_t smem = (size_t)STAGES * (A_BYTES + BN * BK * 2) + 1024 + 256;
     static bool set = false;
     if (!set) {
-        cudaError_t e = cudaFuncSetAttribute(gateup_silu_tc_pair_kernel<BN, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(gateup_silu_tc_pair_kernel<BN, STAGES, UNIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         set = true;
     }
@@ -244,7 +255,7 @@ int launch_gateup_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, in
     const long long want = pairs < num_blocks / 2 ? pairs : num_blocks / 2;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3((unsigned)(2 * want));
-    cfg.blockDim = dim3(THREADS);
+    cfg.blockDim = dim3(THREADS<(UNIT >= PLAIN_GELU_ERF)>);
     cfg.dynamicSmemBytes = smem;
     cfg.stream = s;
     cudaLaunchAttribute attr[2];
@@ -256,7 +267,22 @@ int launch_gateup_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, in
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = llmie_pdl_flag ? 2 : 1;
-    return (int)cudaLaunchKernelEx(&cfg, gateup_silu_tc_pair_kernel<BN, STAGES>, mx, mw, out, M, I, K, error_flag, limit, alpha, shift);
+    return (int)cudaLaunchKernelEx(&cfg, gateup_silu_tc_pair_kernel<BN, STAGES, UNIT>, mx, mw, out, M, I, K, error_flag, limit, alpha, shift);
+}
+
+template <int UNIT>
+int dispatch_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, int K, int num_blocks, int* error_flag, float limit, float alpha,
+                 float shift, cudaStream_t s) {
+    if (M <= 0 || I <= 0) return 0;
+    if (K <= 0 || K % 8 || I % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ((uintptr_t)out & 15) || !error_flag || num_blocks < 2)
+        return LLMIE_ERR_BAD_ARGUMENT;
+    switch (best_tile_width(((M + BM - 1) / BM + 1) / 2, I, num_blocks / 2)) {
+        case 112: return launch_gateup_pair<112, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
+        case 96: return launch_gateup_pair<96, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
+        case 80: return launch_gateup_pair<80, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
+        case 64: return launch_gateup_pair<64, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
+        default: return launch_gateup_pair<128, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
+    }
 }
 
 }  // namespace
@@ -267,19 +293,20 @@ int launch_gateup_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, in
 LLMIE_API int llmie_gateup_glu_tc_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, int K, int num_blocks, int* error_flag,
                                         float limit, float alpha, float shift,
                                         cudaStream_t s) {
-    if (M <= 0 || I <= 0) return 0;
-    if (K <= 0 || K % 8 || I % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ((uintptr_t)out & 15) || !error_flag || num_blocks < 2)
-        return LLMIE_ERR_BAD_ARGUMENT;
-    switch (best_tile_width(((M + BM - 1) / BM + 1) / 2, I, num_blocks / 2)) {
-        case 112: return launch_gateup_pair<112>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-        case 96: return launch_gateup_pair<96>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-        case 80: return launch_gateup_pair<80>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-        case 64: return launch_gateup_pair<64>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-        default: return launch_gateup_pair<128>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-    }
+    if (limit > 0.f) return dispatch_pair<UNIT_CLAMPED>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
+    if (limit < 0.f) return dispatch_pair<UNIT_GELU_TANH>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
+    return dispatch_pair<UNIT_SILU>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
 }
 
 // The same with silu(gate) * up as the epilogue.
 LLMIE_API int llmie_gateup_silu_tc_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, int K, int num_blocks, int* error_flag, cudaStream_t s) {
     return llmie_gateup_glu_tc_pair(x, w, out, M, I, K, num_blocks, error_flag, 0.f, 1.f, 0.f, s);
+}
+
+// act(x w^T) for w [N, K]: the same product without a gate; N a multiple of 16. tanh_form: the tanh form of GELU instead of the exact one.
+LLMIE_API int llmie_up_gelu_tc_pair(const bf16* x, const bf16* w, bf16* out, int M, int N, int K, int num_blocks, int* error_flag, int tanh_form,
+                                 cudaStream_t s) {
+    if (N % 16) return LLMIE_ERR_BAD_ARGUMENT;
+    if (tanh_form) return dispatch_pair<PLAIN_GELU_TANH>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, s);
+    return dispatch_pair<PLAIN_GELU_ERF>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, s);
 }

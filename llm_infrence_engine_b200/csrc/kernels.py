@@ -62,6 +62,7 @@ class CudaKernels:
         self.use_fused_router = os.environ.get("LLMIE_FUSED_ROUTER", "1") != "0"   # a router's product and choice in one kernel (few rows, float32)
         self.use_tc_experts = True     # routed experts with many rows per expert: both grouped products on tcgen05 (bfloat16)
         self.use_tc_gate_up = True     # prompt portions: gate/up product with the activation as its epilogue, one tcgen05 kernel
+        self.up_act_min_rows = 512     # ... and a plain product with a GELU as its epilogue, from this many rows on (below, product and activation are faster)
         self.use_tc_qkv = True         # prompt portions, head size 64: q/k/v product with bias, rotation and cache write in one kernel ...
         self.tc_qkv_min_rows = 2048    # ... from this many rows on: below, the library product + the rotation kernel are 4 to 10 % of a step faster
         self.tc_max_rows = 128        # batches up to this many rows take the small-batch tensor-core product
@@ -121,10 +122,11 @@ class CudaKernels:
                    "llmie_dynamic_tanh"):
             getattr(self.lib, fn).restype = ctypes.c_int
         # two forms of the gate/up kernel live in source files of their own, and the library also builds without them
-        self._gate_up_cluster = self._gate_up_pair = self._gate_up_glu_pair = None
+        self._gate_up_cluster = self._gate_up_pair = self._gate_up_glu_pair = self._up_gelu_pair = None
         self.lib.llmie_gateup_glu_tc.restype = ctypes.c_int
+        self.lib.llmie_up_gelu_tc.restype = ctypes.c_int
         for attr, name in (("_gate_up_cluster", "llmie_gateup_silu_tc_cluster"), ("_gate_up_pair", "llmie_gateup_silu_tc_pair"),
-                           ("_gate_up_glu_pair", "llmie_gateup_glu_tc_pair")):
+                           ("_gate_up_glu_pair", "llmie_gateup_glu_tc_pair"), ("_up_gelu_pair", "llmie_up_gelu_tc_pair")):
             try:
                 fn = getattr(self.lib, name)
                 fn.restype = ctypes.c_int
@@ -979,6 +981,15 @@ class CudaKernels:
         if activation not in kinds:
             raise KernelError(f"linear_act: activation '{activation}' is not built")
         out_dtype = out_dtype or x.dtype
+        M, K_ = x.shape
+        if (self.use_tc_gate_up and x.dtype == torch.bfloat16 and out_dtype == torch.bfloat16 and M > self.tc_max_rows and M >= self.up_act_min_rows
+                and K_ % 8 == 0 and w.dim() == 2 and w.shape[0] % 16 == 0 and w.shape[1] == K_ and w.dtype == torch.bfloat16 and x.is_contiguous() and w.is_contiguous()):
+            # prompt portions: one tcgen05 kernel whose epilogue is the activation (the gate/up kernels without a gate)
+            out = torch.empty((M, w.shape[0]), dtype=torch.bfloat16, device=x.device)
+            fn = self._up_gelu_pair if (self.use_pair_gate_up and self._up_gelu_pair is not None and M >= self.pair_gate_up_min_rows) else self.lib.llmie_up_gelu_tc
+            self._check(fn(_ptr(x), _ptr(w), _ptr(out), M, w.shape[0], K_, self.num_sms, _ptr(self._errors(x.device)), int(activation == "gelu_tanh"),
+                           self._stream()), "linear_act (tcgen05)")
+            return out
         z = self.linear(x, w, transient=True)
         clear = self._is_transient(z)
         out = torch.empty(z.shape, dtype=out_dtype, device=z.device)

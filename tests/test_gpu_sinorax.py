@@ -140,9 +140,25 @@ def test_products_with_a_bias_exact_gelu_and_scaled_cap(K, dtype):
             close(z, want, "float32", "transient sums with a bias", scale=tol, f32=4e-6)
             z.zero_()
     K.check_device_errors()
-    for M, N in ((3, 40), (200, 264)):
+    for M, N in ((3, 40), (7, 33), (200, 264), (300, 272), (130, 16), (1100, 1040), (2048, 96)):
         x, w = rnd(M, 64, seed=5).to(T), rnd(N, 64, seed=6, scale=0.3).to(T)
-        close(K.linear_act(x.cuda(), w.cuda(), "gelu_erf", T), ref.linear_act(x, w, "gelu_erf", T), dtype, f"exact GELU {M}x{N}", f32=4e-6)
+        for act in ("gelu_erf", "gelu_tanh"):
+            want = ref.linear_act(x, w, act, T)
+            for rows in (1, 1 << 20):      # one kernel with the activation in it, where it takes the sizes; product and activation
+                before, K.up_act_min_rows = K.up_act_min_rows, rows
+                try:
+                    got = K.linear_act(x.cuda(), w.cuda(), act, T)
+                finally:
+                    K.up_act_min_rows = before
+                close(got, want, dtype, f"{act} {M}x{N} (one kernel from {rows} rows)", f32=4e-6)
+    if dtype == "bfloat16":   # the fast form of the exact GELU, value by value: a product with the identity
+        z = torch.linspace(-12, 12, 256 * 16).to(T).view(256, 16)
+        want = ref.linear_act(z.float(), torch.eye(16), "gelu_erf", torch.float32)
+        for rows in (z.repeat(4, 1), z, z[:100]):
+            got = K.linear_act(rows.contiguous().cuda(), torch.eye(16, dtype=T).cuda(), "gelu_erf", T).float().cpu()
+            w_ = want.repeat(4, 1)[:rows.shape[0]]
+            assert float(((got - w_).abs() / (w_.abs() * 2 ** -8 + 1e-6)).max()) < 1.0
+        K.check_device_errors()
     if dtype == "bfloat16":
         assert K._acc is None or float(K._acc.abs().max()) == 0.0
     x = rnd(9, 77, seed=7, scale=30.0)
