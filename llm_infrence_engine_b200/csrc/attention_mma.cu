@@ -363,7 +363,8 @@ __device__ __forceinline__ void attend_chunk_t8(const uint32_t (&qb)[D / 16][2],
 
 // ---------------------------------------------------------------------------------------------- decode
 // T8: every tile has at most 8 rows and one token (a decode step of a model with up to 8 heads per group): the transposed form.
-template <int D, int BN, int STAGES, int DW, bool T8, bool SIG>
+// SIG: sigmoid weights; TURN: results are turned back (each compiled in only where it is asked for)
+template <int D, int BN, int STAGES, int DW, bool T8, bool SIG, bool TURN>
 __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p) {
     extern __shared__ __align__(128) unsigned char smem_raw[];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -646,7 +647,7 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
         }
     }
     __syncthreads();
-    if (p.turn_cos) {
+    if constexpr (TURN) {
         // turned back here, slice by slice (the turn is linear and the same for all slices of a row)
         for (int i = tid; i < nrows * (D / 2); i += DW * 32) {
             const int r = i / (D / 2), k = i % (D / 2);
@@ -822,15 +823,15 @@ __global__ void attn_plan_kernel(const int* __restrict__ starts, int num_seqs, i
     for (; t < max_tiles; ++t) { tile_info[2 * t] = 0; tile_info[2 * t + 1] = 0; }
 }
 
-template <int D, bool T8, int DW, bool SIG = false>
-int launch_decode(const Params& p, dim3 grid, cudaStream_t s) {
+template <int D, bool T8, int DW, bool SIG, bool TURN>
+int launch_decode_as(const Params& p, dim3 grid, cudaStream_t s) {
     constexpr int BN = D == 64 ? 32 : 16, STAGES = 3;  // DW warps, each with its own ring of 4 KB + 4 KB chunks
     constexpr size_t ring = (size_t)DW * STAGES * 2 * BN * D * sizeof(bf16);
     constexpr size_t merge = (size_t)(DW * 16 * (D + 8 + 3) + 16 * (D + 2)) * sizeof(float);
     constexpr size_t smem = ring > merge ? ring : merge;
     static bool set = false;
     if (!set) {
-        cudaError_t e = cudaFuncSetAttribute(attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG, TURN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         set = true;
     }
@@ -849,9 +850,15 @@ int launch_decode(const Params& p, dim3 grid, cudaStream_t s) {
         attr[1].val.programmaticStreamSerializationAllowed = 1;
         cfg.attrs = attr;
         cfg.numAttrs = llmie_pdl_flag ? 2 : 1;
-        return (int)cudaLaunchKernelEx(&cfg, attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG>, p);
+        return (int)cudaLaunchKernelEx(&cfg, attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG, TURN>, p);
     }
-    return launch_kernel(attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG>, grid, dim3(DW * 32), smem, s, p);
+    return launch_kernel(attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG, TURN>, grid, dim3(DW * 32), smem, s, p);
+}
+
+template <int D, bool T8, int DW>
+int launch_decode(const Params& p, dim3 grid, cudaStream_t s) {
+    if (p.sig_bias) return p.turn_cos ? launch_decode_as<D, T8, DW, true, true>(p, grid, s) : launch_decode_as<D, T8, DW, true, false>(p, grid, s);
+    return p.turn_cos ? launch_decode_as<D, T8, DW, false, true>(p, grid, s) : launch_decode_as<D, T8, DW, false, false>(p, grid, s);
 }
 
 template <int D>
@@ -864,10 +871,6 @@ int launch(const Params& p, int num_tiles, int decode_mode, cudaStream_t s) {
         // blocks than multiprocessors and nothing is cut into slices, the caller may ask for blocks of four warps (96 KB:
         // two per multiprocessor), which then run in fewer, fuller rounds (96 requests of 8,192 keys: 94 us in two rounds of
         // eight-warp blocks, the second half empty; 74.5 us at once).
-        if (p.sig_bias) {
-            if (decode_mode == 2 && p.num_splits == 1) return t8 ? launch_decode<D, true, 4, true>(p, grid, s) : launch_decode<D, false, 4, true>(p, grid, s);
-            return t8 ? launch_decode<D, true, 8, true>(p, grid, s) : launch_decode<D, false, 8, true>(p, grid, s);
-        }
         if (decode_mode == 2 && p.num_splits == 1) return t8 ? launch_decode<D, true, 4>(p, grid, s) : launch_decode<D, false, 4>(p, grid, s);
         return t8 ? launch_decode<D, true, 8>(p, grid, s) : launch_decode<D, false, 8>(p, grid, s);
     } else {

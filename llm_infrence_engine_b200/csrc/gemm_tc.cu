@@ -30,7 +30,7 @@ namespace {
 
 constexpr int BM = 128, BK = 64, STAGES = 4, UMMA_K = 16;
 
-template <int TN>
+template <int TN, bool BIAS>
 __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant__ CUtensorMap tmap_x,
                                                       float* __restrict__ out, int ldo, int M, int N, int K, int kb_per_split,
                                                       int accumulate, int* error_flag, const bf16* __restrict__ bias) {
@@ -117,7 +117,8 @@ __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CU
     if (done) {
         const int n = n0 + warp * 32 + lane;
         const int rows = min(TN, M - m0);
-        const float add = (bias && n < N && blockIdx.z == 0) ? to_f32(bias[n]) : 0.f;
+        float add = 0.f;
+        if constexpr (BIAS) add = (n < N && blockIdx.z == 0) ? to_f32(bias[n]) : 0.f;
 #pragma unroll
         for (int c = 0; c < TN; c += 16) {
             uint32_t v[16];
@@ -129,8 +130,8 @@ __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CU
                     const int m = c + j;
                     if (m < rows) {
                         float* dst = out + (size_t)(m0 + m) * ldo + n;
-                        if (accumulate) atomicAdd(dst, __uint_as_float(v[j]) + add);
-                        else *dst = __uint_as_float(v[j]) + add;
+                        if (accumulate) atomicAdd(dst, BIAS ? __uint_as_float(v[j]) + add : __uint_as_float(v[j]));
+                        else *dst = BIAS ? __uint_as_float(v[j]) + add : __uint_as_float(v[j]);
                     }
                 }
             }
@@ -153,13 +154,13 @@ __global__ void __launch_bounds__(128) gemm_tc_kernel(const __grid_constant__ CU
 }
 
 // ------------------------------------------------------------------------------------------------ host side
-template <int TN>
-int launch(const CUtensorMap& mw, const CUtensorMap& mx, float* out, int ldo, int M, int N, int K, int k_splits, int accumulate,
+template <int TN, bool BIAS>
+int launch_as(const CUtensorMap& mw, const CUtensorMap& mx, float* out, int ldo, int M, int N, int K, int k_splits, int accumulate,
            int* error_flag, const bf16* bias, cudaStream_t s) {
     constexpr size_t smem = (size_t)STAGES * (BM * BK * 2 + TN * BK * 2) + 1024 + 256;
     static bool set = false;
     if (!set) {
-        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<TN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(gemm_tc_kernel<TN, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         set = true;
     }
@@ -167,7 +168,14 @@ int launch(const CUtensorMap& mw, const CUtensorMap& mx, float* out, int ldo, in
     const int per = (nkb + k_splits - 1) / k_splits;
     const int splits = (nkb + per - 1) / per;  // no empty split
     const dim3 grid((N + BM - 1) / BM, (M + TN - 1) / TN, splits);
-    return launch_kernel(gemm_tc_kernel<TN>, grid, dim3(128), smem, s, mw, mx, out, ldo, M, N, K, per, accumulate, error_flag, bias);
+    return launch_kernel(gemm_tc_kernel<TN, BIAS>, grid, dim3(128), smem, s, mw, mx, out, ldo, M, N, K, per, accumulate, error_flag, bias);
+}
+
+template <int TN>
+int launch(const CUtensorMap& mw, const CUtensorMap& mx, float* out, int ldo, int M, int N, int K, int k_splits, int accumulate,
+           int* error_flag, const bf16* bias, cudaStream_t s) {
+    if (bias) return launch_as<TN, true>(mw, mx, out, ldo, M, N, K, k_splits, accumulate, error_flag, bias, s);
+    return launch_as<TN, false>(mw, mx, out, ldo, M, N, K, k_splits, accumulate, error_flag, nullptr, s);
 }
 
 static int run(const bf16* x, const bf16* w, float* out, int ldo, int M, int N, int K, int k_splits, int accumulate, int* error_flag,
