@@ -15,6 +15,7 @@ class PagedKVSpec:
     v_head_dim: Optional[int] = None  # size of a value row; None: as the keys; 0: no value pool (values are read out of the key rows)
     keep_first: int = 0           # with a window: keys at positions below this are read for ever, whatever the window
     chunk: Optional[int] = None   # n: position p reads only keys from floor(p / n) * n on (runs of n positions from the request's start)
+    token_scalar: bool = False    # one 32-bit number per cached token rides in a pool of its own
 
 
 @dataclass(frozen=True)

@@ -995,3 +995,141 @@ class SinoraxConfig:
             raise ConfigError(f"config.json: 'logit_softcap' must be positive, got {cap}")
         return cls(_pos_int(d, "vocab", ""), _pos_int(d, "width", ""), _number(norm, "eps", "norm.") if norm and "eps" in norm else 0.0,
                    BigramConfig.from_dict(bigram, "embedding.bigram.") if bigram else None, scale, cap, tuple(layers))
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Putelix: a decoder whose config.json lists its layers one by one; the sublayers read the stream itself and their RESULTS are
+# normed. Mixer: chunked attention whose values are its keys, beside linear attention with a fixed decay per head. Feed-forwards: a
+# dense unit with squared relu, or routed experts weighted by a softmax over the chosen logits, with a gated shared expert.
+
+@dataclass(frozen=True)
+class SharedKeyAttentionConfig:
+    """The left half of ``parallel``: grouped attention without rotation whose values are the keys as projected, so ``vdim`` (where
+    given) equals ``dim``; a learned bias by distance (rows up to ``bias_max``), an optional soft cap and chunks of ``chunk`` positions."""
+
+    heads: int
+    kv_heads: int
+    dim: int
+    scale: float
+    bias_max: float
+    chunk: Optional[int] = None
+    softcap: Optional[float] = None
+
+    @classmethod
+    def from_dict(cls, m: Mapping[str, Any], where: str) -> "SharedKeyAttentionConfig":
+        heads, kv_heads = _pos_int(m, "heads", where), _pos_int(m, "kv_heads", where)
+        if heads % kv_heads:
+            raise ConfigError(f"config.json: {where}{heads} heads cannot share {kv_heads} kv_heads")
+        dim = _pos_int(m, "dim", where)
+        if m.get("vdim") is not None and _pos_int(m, "vdim", where) != dim:
+            raise ConfigError(f"config.json: {where}'vdim' {m['vdim']} differs from 'dim' {dim}, but the values are the keys")
+        mask = _opt_sub(m, "mask", where)
+        cap = _number(m, "softcap", where) if m.get("softcap") is not None else None
+        if cap is not None and not cap > 0:
+            raise ConfigError(f"config.json: {where}'softcap' must be positive, got {cap}")
+        return cls(heads, kv_heads, dim, _number(m, "scale", where), _number(m, "bias_max", where),
+                   _pos_int(mask, "size", where + "mask.") if mask else None, cap)
+
+
+@dataclass(frozen=True)
+class LinearAttentionConfig:
+    """The right half of ``parallel``: a matrix memory per head that shrinks by ``decay[head]`` at every token."""
+
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple
+
+    @classmethod
+    def from_dict(cls, m: Mapping[str, Any], where: str) -> "LinearAttentionConfig":
+        heads, dim = _pos_int(m, "heads", where), _pos_int(m, "dim", where)
+        if dim > 256:
+            raise ConfigError(f"config.json: {where}'dim' {dim} is more than the 256 entries of a memory column that are built")
+        decay = m.get("decay")
+        if isinstance(decay, (int, float)) and not isinstance(decay, bool):
+            decay = [decay] * heads
+        if not isinstance(decay, (list, tuple)) or len(decay) != heads or any(isinstance(d, bool) or not isinstance(d, (int, float)) for d in decay):
+            raise ConfigError(f"config.json: {where}'decay' must be {heads} numbers, one per head, got {decay!r}")
+        if not all(0.0 <= float(d) <= 1.0 for d in decay):
+            raise ConfigError(f"config.json: {where}'decay' must lie between 0 and 1, got {decay!r}")
+        return cls(heads, dim, _pos_int(m, "vdim", where) if "vdim" in m else dim, tuple(float(d) for d in decay))
+
+
+@dataclass(frozen=True)
+class NormedPairConfig:
+    """Mixer ``parallel`` of Putelix: the two halves, whose normed results are averaged."""
+
+    left: SharedKeyAttentionConfig
+    right: LinearAttentionConfig
+
+    @classmethod
+    def from_dict(cls, m: Mapping[str, Any], where: str) -> "NormedPairConfig":
+        return cls(SharedKeyAttentionConfig.from_dict(_sub(m, "left", where), where + "left."),
+                   LinearAttentionConfig.from_dict(_sub(m, "right", where), where + "right."))
+
+
+@dataclass(frozen=True)
+class TopSoftmaxExpertsConfig:
+    """``mlp.kind = "moe"``: ``experts`` gated units of width ``ff`` of which a token uses the ``top`` with the largest logits, weighted by
+    the softmax over those alone; ``shared_ff`` (or None): the width of a unit that every token uses, behind a gate of its own."""
+
+    experts: int
+    top: int
+    ff: int
+    shared_ff: Optional[int]
+
+    @classmethod
+    def from_dict(cls, mlp: Mapping[str, Any], where: str) -> "TopSoftmaxExpertsConfig":
+        r = _sub(mlp, "router", where)
+        shared = _opt_sub(mlp, "shared", where)
+        c = cls(_pos_int(r, "experts", where + "router."), _pos_int(r, "top", where + "router."),
+                _pos_int(_sub(mlp, "expert", where), "ff", where + "expert."), _pos_int(shared, "ff", where + "shared.") if shared else None)
+        if c.top > c.experts:
+            raise ConfigError(f"config.json: {where}router.top {c.top} is more than the {c.experts} experts")
+        if c.experts > 511:
+            raise ConfigError(f"config.json: {where}router: at most 511 experts are built")
+        return c
+
+
+@dataclass(frozen=True)
+class PutelixLayerConfig:
+    mixer: NormedPairConfig
+    mlp: Any                   # None: the layer is a mixer alone; the width of a dense unit; or a TopSoftmaxExpertsConfig
+
+
+@dataclass(frozen=True)
+class PutelixConfig:
+    """The whole of a Putelix config.json: vocabulary, width, norm epsilon, the rows of the position table (None: the checkpoint
+    decides) and the list of layers."""
+
+    architecture = "Putelix"
+
+    vocab: int
+    width: int
+    eps: float
+    max_positions: Optional[int]
+    layers: tuple
+
+    @classmethod
+    def from_dict(cls, d: Mapping[str, Any]) -> "PutelixConfig":
+        if not isinstance(d.get("layers"), (list, tuple)) or not d["layers"]:
+            raise ConfigError("config.json: 'layers' must be a list with at least one layer")
+        layers = []
+        for i, layer in enumerate(d["layers"]):
+            where = f"layers[{i}]."
+            if not isinstance(layer, Mapping):
+                raise ConfigError(f"config.json: layers[{i}] must be an object")
+            if layer.get("type") != "parallel":
+                raise ConfigError(f"config.json: {where}type {layer.get('type')!r} is not 'parallel'")
+            mixer = NormedPairConfig.from_dict(_sub(layer, "mixer", where), where + "mixer.")
+            mlp = layer.get("mlp")
+            if mlp is not None:
+                if not isinstance(mlp, Mapping) or mlp.get("kind", "dense") not in ("dense", "moe"):
+                    raise ConfigError(f"config.json: {where}mlp must be null or an object of kind 'dense' or 'moe'")
+                mlp = _pos_int(mlp, "ff", where + "mlp.") if mlp.get("kind", "dense") == "dense" else TopSoftmaxExpertsConfig.from_dict(mlp, where + "mlp.")
+            layers.append(PutelixLayerConfig(mixer, mlp))
+        cfg = cls(_pos_int(d, "vocab", ""), _pos_int(d, "width", ""), _number(_sub(d, "norm", ""), "eps", "norm."),
+                  _pos_int(d, "max_positions", "") if d.get("max_positions") is not None else None, tuple(layers))
+        if not cfg.eps > 0:
+            raise ConfigError(f"norm.eps must be positive, got {cfg.eps}")
+        return cfg

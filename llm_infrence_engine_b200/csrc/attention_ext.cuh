@@ -13,6 +13,8 @@
 //     window has passed them (at their true positions);
 //   * chunks: with `chunk` > 0 a position sees only keys of its own run of `chunk` positions, counted from the request's start;
 //   * a soft cap: score <- cap * tanh(score / cap), applied to the scaled score;
+//   * a number per cached token that multiplies its keys' scores (before the cap): keys that are cached as they were before a norm
+//     over the whole key projection carry that norm's reciprocal root mean square so, and can be the values too;
 //   * a penalty by the logarithm of the distance: r1[head] * ln(1 + r2[head] * (p - j)) is taken off the scaled score;
 //   * weights without a softmax: with `sig_bias` a visible key's weight is sigmoid(score + sig_bias[head]), and nothing is divided
 //     by a sum over the keys (no maximum, no sink);
@@ -49,6 +51,7 @@ struct Extras {
     const float* turn_cos = nullptr;   // [N, dv / 2], with turn_sin: results are turned back
     const float* turn_sin = nullptr;
     int turn_neighbours = 0;  // 1: pairs (2 m, 2 m + 1)
+    const float* key_scale = nullptr;  // [pages][page_size]: a number per cached token, on its scores
 };
 
 // Where the pair of result entry `dim` lies: its number m, and the other entry.
@@ -188,6 +191,11 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attn_ext_kernel(
 #pragma unroll
                     for (int g = 0; g < GC; ++g) s[g] = fmaf(qs[g * dkp + c], kf, s[g]);
                 }
+            }
+            if (ex.key_scale) {
+                const float f = ex.key_scale[(size_t)blk * page_size + key % page_size];
+#pragma unroll
+                for (int g = 0; g < GC; ++g) s[g] *= f;
             }
             if (ex.softcap > 0.f) {
 #pragma unroll
@@ -351,7 +359,7 @@ __global__ void attn_ext_combine_kernel(const float* __restrict__ part_acc, cons
 enum { PLAIN = 0, MASKS = 1, SIGMOID = 2 };
 inline int kind_of(const Extras& ex) {
     if (ex.sig_bias) return SIGMOID;
-    return (ex.keep_first > 0 || ex.chunk > 0 || ex.softcap > 0.f || ex.log_r1) ? MASKS : PLAIN;
+    return (ex.keep_first > 0 || ex.chunk > 0 || ex.softcap > 0.f || ex.log_r1 || ex.key_scale) ? MASKS : PLAIN;
 }
 
 // A row's terms of its scores in the tensor-core kernels, whose weights are rounded to 8 bits: the fast exponential, logarithm and
@@ -373,6 +381,11 @@ struct RowTerms {
         return __fdividef(1.0f, 1.0f + hw_exp2(fmaf(r1, hw_log2(fmaf(r2, dist, 1.0f)), fmaf(a, s, b))));
     }
 };
+
+// cap * tanh(v / cap) there, by tanh(t) = 1 - 2 / (exp(2 t) + 1); two_log2e_over_cap = 2 log2(e) / cap
+__device__ __forceinline__ float cap_fast(float v, float cap, float two_log2e_over_cap) {
+    return fmaf(-2.0f * cap, __fdividef(1.0f, hw_exp2(v * two_log2e_over_cap) + 1.0f), cap);
+}
 
 // True if the extras contradict each other or lack a pointer.
 inline bool bad_extras(const Extras& ex, int dv) {

@@ -7,7 +7,7 @@ LLMIE_API int llmie_paged_attention_ext_f32(const float* q, int q_stride, const 
                                            int slice_keys, float temp_coef, int temp_every, const float* rel, const int* rows_of,
                                            int n_rows_of, int rel_rows, const float* sink, const float* gate, int gate_stride, int gate_mode,
                                            int keep_first, int chunk, float softcap, const float* sig_bias, const float* log_r1,
-                                           const float* log_r2, const float* turn_cos, const float* turn_sin, int turn_neighbours, cudaStream_t s) {
+                                           const float* log_r2, const float* turn_cos, const float* turn_sin, int turn_neighbours, const float* key_scale, cudaStream_t s) {
     attn_ext::Extras ex;
     ex.temp_coef = temp_coef; ex.temp_every = temp_every;
     ex.rel = rel; ex.rows_of = rows_of; ex.n_rows_of = n_rows_of; ex.rel_rows = rel_rows;
@@ -15,6 +15,7 @@ LLMIE_API int llmie_paged_attention_ext_f32(const float* q, int q_stride, const 
     ex.keep_first = keep_first; ex.chunk = chunk; ex.softcap = softcap;
     ex.sig_bias = sig_bias; ex.log_r1 = log_r1; ex.log_r2 = log_r2;
     ex.turn_cos = turn_cos; ex.turn_sin = turn_sin; ex.turn_neighbours = turn_neighbours;
+    ex.key_scale = key_scale;
     return attn_ext::paged_attention_ext<float>(q, q_stride, k_pool, v_pool, block_table, max_blocks, token_seq, positions, out, scratch, N,
                                             nq, nkv, dk, dv, page_size, scale, window, num_splits, slice_keys, ex, s);
 }

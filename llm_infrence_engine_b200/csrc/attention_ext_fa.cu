@@ -4,6 +4,7 @@
 // queries held in registers for the whole tile, keys by ldmatrix from shared memory), scales, biases and masks them, takes
 // maxima and sums inside its quads (four lanes share a row), and feeds the rounded weights straight from the score registers
 // into the P V products. The only barriers are the two per chunk around the cp.async ring of keys and values (two stages).
+// Values may be the keys themselves (`v_pool == nullptr`, sizes alike): a chunk is then fetched once and read in both products.
 // Key slices (grid.z) and the finishing of rows (sink, division, gate) are those of attention_ext_mma.cu.
 #include "attention_ext.cuh"
 
@@ -21,6 +22,7 @@ struct Params {
     bf16* out; float* part_acc; float* part_ml;
     int nq, nkv, dk, dv, page_size; float scale; int window, num_splits, gh, head_chunks;
     int bias_in_smem;
+    unsigned key_scale_at;   // with ex.key_scale: byte offset in shared memory of the chunks' numbers per key, [2][KEYS] floats
     Extras ex;
 };
 
@@ -40,6 +42,10 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src, int src_b
     const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(d), "l"(src), "r"(src_bytes));
 }
+__device__ __forceinline__ void cp_async4(void* dst, const void* src, int src_bytes) {
+    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;\n" ::"r"(d), "l"(src), "r"(src_bytes));
+}
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;\n" ::); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
 __device__ __forceinline__ uint32_t pack2(float a, float b) {
@@ -57,8 +63,10 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
     constexpr int dk = 16 * KD, dv = 16 * NV, ks = dk + 8, vs = dv + 8;
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);            // [ROWS][ks]: only until the queries are in registers
     bf16* Ks = Qs + ROWS * ks;                               // [2][KEYS][ks]
-    bf16* Vs = Ks + 2 * KEYS * ks;                           // [2][KEYS][vs]
+    bf16* Vs = P.v_pool ? Ks + 2 * KEYS * ks : Ks;           // [2][KEYS][vs], or the keys themselves
     float* bias_val = reinterpret_cast<float*>(Vs + 2 * KEYS * vs);   // [rel_rows][gh]
+    float* key_scale_s = reinterpret_cast<float*>(smem_raw + P.key_scale_at);   // (only with ex.key_scale)
+    const float cap_k = MASKS && P.ex.softcap > 0.f ? 2.8853900817779268f / P.ex.softcap : 0.f;   // 2 log2(e) / cap
     unsigned short* bias_row = reinterpret_cast<unsigned short*>(bias_val + (P.bias_in_smem ? P.ex.rel_rows * P.gh : 0));
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, gid = lane >> 2, tig = lane & 3;
@@ -131,13 +139,19 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
     auto load_chunk = [&](int c, int stage) {
         const int key = (c < npre ? c * KEYS : start + (c - npre) * KEYS) + my_key;
         const bool ok = c < npre ? key < kept : (key < end && key >= lo);
-        size_t row = 0;
-        if (ok) row = ((size_t)table[key / P.page_size] * P.nkv + kvh) * P.page_size + key % P.page_size;
+        size_t row = 0, slot = 0;
+        if (ok) {
+            const size_t page = table[key / P.page_size];
+            row = (page * P.nkv + kvh) * P.page_size + key % P.page_size;
+            slot = page * P.page_size + key % P.page_size;
+        }
         const int bytes = ok ? 16 : 0;
+        if (MASKS && P.ex.key_scale && odd == 0) cp_async4(key_scale_s + stage * KEYS + my_key, P.ex.key_scale + slot, ok ? 4 : 0);
         bf16* kd = Ks + (stage * KEYS + my_key) * ks;
         const bf16* ksrc = P.k_pool + row * dk;
 #pragma unroll
         for (int sgm = odd; sgm < segs; sgm += 2) cp_async16(kd + sgm * 8, ksrc + sgm * 8, bytes);
+        if (!P.v_pool) return;
         bf16* vd = Vs + (stage * KEYS + my_key) * vs;
         const bf16* vsrc = P.v_pool + row * dv;
 #pragma unroll
@@ -209,6 +223,13 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
             }
         } else {
         float mx[2] = {-INFINITY, -INFINITY};
+        if (MASKS && P.ex.key_scale) {   // (before the scale and the cap: both halves of a pair of keys of my tiles)
+#pragma unroll
+            for (int t = 0; t < 8; ++t) {
+                const float2 kf = *reinterpret_cast<const float2*>(key_scale_s + stage * KEYS + t * 8 + 2 * tig);
+                s[t][0] *= kf.x; s[t][1] *= kf.y; s[t][2] *= kf.x; s[t][3] *= kf.y;
+            }
+        }
         if (interior) {
 #pragma unroll
             for (int t = 0; t < 8; ++t)
@@ -216,7 +237,7 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
                 for (int e = 0; e < 4; ++e) {
                     const int i = e >> 1;
                     float v = s[t][e] * row_factor[i];
-                    if (MASKS && P.ex.softcap > 0.f) v = P.ex.softcap * tanhf(v / P.ex.softcap);
+                    if (MASKS && P.ex.softcap > 0.f) v = attn_ext::cap_fast(v, P.ex.softcap, cap_k);
                     if (P.ex.rel) {
                         const int dist = row_pos[i] - (base + t * 8 + 2 * tig + (e & 1));
                         if (P.bias_in_smem) {
@@ -243,7 +264,7 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
                     float v = -INFINITY;
                     if (seen) {
                         v = s[t][e] * row_factor[i];
-                        if (MASKS && P.ex.softcap > 0.f) v = P.ex.softcap * tanhf(v / P.ex.softcap);
+                        if (MASKS && P.ex.softcap > 0.f) v = attn_ext::cap_fast(v, P.ex.softcap, cap_k);
                         if (P.ex.rel) {
                             const int dist = p - key;
                             if (P.bias_in_smem) {
@@ -370,7 +391,9 @@ __global__ void __launch_bounds__(THREADS) attn_ext_fa_kernel(const Params P) {
     }
 }
 
-size_t smem_bytes(int dk, int dv) { return 2 * ((size_t)ROWS * (dk + 8) + 2 * KEYS * (dk + 8) + 2 * KEYS * (dv + 8)); }
+size_t smem_bytes(int dk, int dv, bool own_values) {
+    return 2 * ((size_t)ROWS * (dk + 8) + 2 * KEYS * (dk + 8) + (own_values ? 2 * KEYS * (dv + 8) : 0));
+}
 size_t bias_bytes(int rel_rows, int gh, int n_rows_of) { return sizeof(float) * (size_t)rel_rows * gh + 2 * (size_t)((n_rows_of + 1) & ~1); }
 
 template <int KD, int NV, int KIND>
@@ -394,10 +417,10 @@ int launch(const Params& P, dim3 grid, size_t smem, cudaStream_t s) {
 
 }  // namespace
 
-// 64 (the rows of a tile) if the kernel takes these sizes: bfloat16, a value pool of its own, heads of 64 or 128 entries for keys
-// and for values (either combination), groups of up to 64 heads; else 0.
+// 64 (the rows of a tile) if the kernel takes these sizes: bfloat16, heads of 64 or 128 entries for keys and for values (either
+// combination with a value pool of its own, the same size where the values are the keys); else 0.
 LLMIE_API int llmie_attention_ext_fa_fits(int dk, int dv, int own_values, int group) {
-    return (own_values && (dk == 64 || dk == 128) && (dv == 64 || dv == 128) && group >= 1) ? ROWS : 0;
+    return ((own_values || dk == dv) && (dk == 64 || dk == 128) && (dv == 64 || dv == 128) && group >= 1) ? ROWS : 0;
 }
 
 // tile_info: [tiles][2] = (first token, tokens) with at most 64 / min(group, 64) tokens of one request per tile.
@@ -407,7 +430,7 @@ LLMIE_API int llmie_paged_attention_ext_fa(const bf16* q, int q_stride, const bf
                                            int window, int num_splits, float temp_coef, int temp_every, const float* rel, const int* rows_of,
                                            int n_rows_of, int rel_rows, const float* sink, const bf16* gate, int gate_stride, int gate_mode,
                                            int keep_first, int chunk, float softcap, const float* sig_bias, const float* log_r1,
-                                           const float* log_r2, const float* turn_cos, const float* turn_sin, int turn_neighbours, cudaStream_t s) {
+                                           const float* log_r2, const float* turn_cos, const float* turn_sin, int turn_neighbours, const float* key_scale, cudaStream_t s) {
     if (N <= 0 || tiles <= 0) return 0;
     if (nkv <= 0 || nq % nkv || !llmie_attention_ext_fa_fits(dk, dv, v_pool != nullptr, nq / nkv) || !tile_info || page_size <= 0 ||
         num_splits < 1 || (num_splits > 1 && !scratch) || q_stride % 8 || ((uintptr_t)q % 16) || ((uintptr_t)k_pool % 16) ||
@@ -426,13 +449,19 @@ LLMIE_API int llmie_paged_attention_ext_fa(const bf16* q, int q_stride, const bf
     P.ex.keep_first = keep_first; P.ex.chunk = chunk; P.ex.softcap = softcap;
     P.ex.sig_bias = sig_bias; P.ex.log_r1 = log_r1; P.ex.log_r2 = log_r2;
     P.ex.turn_cos = turn_cos; P.ex.turn_sin = turn_sin; P.ex.turn_neighbours = turn_neighbours;
-    if (attn_ext::bad_extras(P.ex, dv) || (sig_bias && (rel || keep_first || chunk || softcap != 0.f))) return LLMIE_ERR_BAD_ARGUMENT;
+    P.ex.key_scale = key_scale;
+    if (attn_ext::bad_extras(P.ex, dv) || (sig_bias && (rel || keep_first || chunk || softcap != 0.f || key_scale))) return LLMIE_ERR_BAD_ARGUMENT;
     if ((long long)nkv * P.head_chunks > 65535 || num_splits > 65535) return LLMIE_ERR_BAD_ARGUMENT;
-    size_t smem = smem_bytes(dk, dv);
+    size_t smem = smem_bytes(dk, dv, v_pool != nullptr);
     P.bias_in_smem = 0;
     if (rel && rel_rows <= 65535 && bias_bytes(rel_rows, P.gh, n_rows_of) <= 24 * 1024) {
         P.bias_in_smem = 1;
         smem += bias_bytes(rel_rows, P.gh, n_rows_of);
+    }
+    P.key_scale_at = 0;
+    if (key_scale) {
+        P.key_scale_at = (unsigned)((smem + 7) / 8 * 8);
+        smem = P.key_scale_at + sizeof(float) * KEYS * 2;
     }
     const dim3 grid(tiles, nkv * P.head_chunks, num_splits);
     int rc;

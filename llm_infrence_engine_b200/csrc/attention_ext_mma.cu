@@ -27,7 +27,7 @@ LLMIE_API int llmie_paged_attention_ext_mma(const bf16* q, int q_stride, const b
                                             float scale, int window, int num_splits, float temp_coef, int temp_every, const float* rel,
                                             const int* rows_of, int n_rows_of, int rel_rows, const float* sink, const bf16* gate,
                                             int gate_stride, int gate_mode, int keep_first, int chunk, float softcap, const float* sig_bias, const float* log_r1,
-                                            const float* log_r2, const float* turn_cos, const float* turn_sin, int turn_neighbours, cudaStream_t s) {
+                                            const float* log_r2, const float* turn_cos, const float* turn_sin, int turn_neighbours, const float* key_scale, cudaStream_t s) {
     if (N <= 0 || tiles <= 0) return 0;
     const int fits = llmie_attention_ext_mma_fits(dk, dv, v_pool != nullptr);
     if (nkv <= 0 || nq % nkv || !fits || tile_rows > fits || (tile_rows != 32 && tile_rows != 64 && tile_rows != 128) || page_size <= 0 ||
@@ -47,7 +47,8 @@ LLMIE_API int llmie_paged_attention_ext_mma(const bf16* q, int q_stride, const b
     P.ex.keep_first = keep_first; P.ex.chunk = chunk; P.ex.softcap = softcap;
     P.ex.sig_bias = sig_bias; P.ex.log_r1 = log_r1; P.ex.log_r2 = log_r2;
     P.ex.turn_cos = turn_cos; P.ex.turn_sin = turn_sin; P.ex.turn_neighbours = turn_neighbours;
-    if (attn_ext::bad_extras(P.ex, dv) || (sig_bias && (rel || keep_first || chunk || softcap != 0.f))) return LLMIE_ERR_BAD_ARGUMENT;
+    P.ex.key_scale = key_scale;
+    if (attn_ext::bad_extras(P.ex, dv) || (sig_bias && (rel || keep_first || chunk || softcap != 0.f || key_scale))) return LLMIE_ERR_BAD_ARGUMENT;
     if ((long long)nkv * P.head_chunks > 65535 || num_splits > 65535) return LLMIE_ERR_BAD_ARGUMENT;
     const dim3 grid(tiles, nkv * P.head_chunks, num_splits);
     const int R = tile_rows / ROWS;
@@ -65,6 +66,13 @@ LLMIE_API int llmie_paged_attention_ext_mma(const bf16* q, int q_stride, const b
     if (rel && rel_rows <= 65535 && bias_bytes(rel_rows, P.gh, n_rows_of) <= 32 * 1024 && smem + bias_bytes(rel_rows, P.gh, n_rows_of) <= 227 * 1024) {
         P.bias_in_smem = 1;
         smem += bias_bytes(rel_rows, P.gh, n_rows_of);
+    }
+    P.key_scale_at = 0;
+    if (key_scale) {
+        P.key_scale_at = (unsigned)smem;   // (a multiple of 8: whole rows of 16 bytes, floats, an even number of 16-bit row numbers)
+        if (P.key_scale_at % 8) P.key_scale_at += 8 - P.key_scale_at % 8;
+        smem = P.key_scale_at + sizeof(float) * KEYS * (deep ? DEEP : 2);
+        if (smem > 227 * 1024) return LLMIE_ERR_BAD_ARGUMENT;
     }
     const int kind = attn_ext::kind_of(P.ex);
     int rc = kind == attn_ext::SIGMOID ? launch_sigmoid(P, grid, smem, s, R, deep)

@@ -27,6 +27,7 @@ struct Params {
     bf16* out; float* part_acc; float* part_ml;
     int nq, nkv, dk, dv, page_size; float scale; int window, num_splits, gh, head_chunks;
     int bias_in_smem;   // the distance table's rows (as 16-bit numbers) and this block's heads' columns of it are copied to shared memory
+    unsigned key_scale_at;   // with ex.key_scale: byte offset in shared memory of the chunks' numbers per key, [stages][KEYS] floats
     Extras ex;
 };
 
@@ -49,6 +50,10 @@ __device__ __forceinline__ void mma_bf16(float* c, uint32_t a0, uint32_t a1, uin
 __device__ __forceinline__ void cp_async16(void* dst, const void* src, int src_bytes) {
     const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(d), "l"(src), "r"(src_bytes));
+}
+__device__ __forceinline__ void cp_async4(void* dst, const void* src, int src_bytes) {
+    const uint32_t d = (uint32_t)__cvta_generic_to_shared(dst);
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;\n" ::"r"(d), "l"(src), "r"(src_bytes));
 }
 __device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;\n" ::); }
 template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
@@ -74,6 +79,8 @@ __global__ void __launch_bounds__(THREADS) attn_ext_mma_kernel(const Params P) {
     float* red_sum = red_max + 2 * R * 4 * 16;                  // [2 R][4][16]
     float* bias_val = red_sum + 2 * R * 4 * 16;                 // [rel_rows][gh]: the distance table's columns of this block's heads
     unsigned short* bias_row = reinterpret_cast<unsigned short*>(bias_val + (P.bias_in_smem ? P.ex.rel_rows * P.gh : 0));   // [n_rows_of]
+    float* key_scale_s = reinterpret_cast<float*>(smem_raw + P.key_scale_at);   // (only with ex.key_scale)
+    const float cap_k = MASKS && P.ex.softcap > 0.f ? 2.8853900817779268f / P.ex.softcap : 0.f;   // 2 log2(e) / cap
     constexpr int PS = KEYS + 8;
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -147,9 +154,14 @@ __global__ void __launch_bounds__(THREADS) attn_ext_mma_kernel(const Params P) {
     auto load_chunk = [&](int c, int stage) {
         const int key = (c < npre ? c * KEYS : start + (c - npre) * KEYS) + my_key;
         const bool ok = c < npre ? key < kept : (key < end && key >= lo);
-        size_t row = 0;
-        if (ok) row = ((size_t)table[key / P.page_size] * P.nkv + kvh) * P.page_size + key % P.page_size;
+        size_t row = 0, slot = 0;
+        if (ok) {
+            const size_t page = table[key / P.page_size];
+            row = (page * P.nkv + kvh) * P.page_size + key % P.page_size;
+            slot = page * P.page_size + key % P.page_size;
+        }
         const int bytes = ok ? 16 : 0;
+        if (MASKS && P.ex.key_scale && quarter == 0) cp_async4(key_scale_s + stage * KEYS + my_key, P.ex.key_scale + slot, ok ? 4 : 0);
         bf16* kd = Ks + (stage * KEYS + my_key) * ks;
         const bf16* ksrc = P.k_pool + row * dk;
         for (int sgm = quarter; sgm < segs; sgm += 4) cp_async16(kd + sgm * 8, ksrc + sgm * 8, bytes);
@@ -269,7 +281,9 @@ __global__ void __launch_bounds__(THREADS) attn_ext_mma_kernel(const Params P) {
             if (r >= r_live) break;
             float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-            for (int t = 0; t < 2; ++t)
+            for (int t = 0; t < 2; ++t) {
+                float2 kf = make_float2(1.f, 1.f);
+                if (MASKS && P.ex.key_scale) kf = *reinterpret_cast<const float2*>(key_scale_s + stage * KEYS + part * 16 + t * 8 + 2 * tig);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int i = e >> 1;
@@ -279,7 +293,8 @@ __global__ void __launch_bounds__(THREADS) attn_ext_mma_kernel(const Params P) {
                     float v = -INFINITY;
                     if (seen) {
                         v = (s[r][t][e] + s2[r][t][e]) * row_factor[r][i];
-                        if (MASKS && P.ex.softcap > 0.f) v = P.ex.softcap * tanhf(v / P.ex.softcap);
+                        if (MASKS) v *= (e & 1) ? kf.y : kf.x;
+                        if (MASKS && P.ex.softcap > 0.f) v = attn_ext::cap_fast(v, P.ex.softcap, cap_k);
                         if (P.ex.rel) {
                             const int dist = p - key;
                             if (P.bias_in_smem) {
@@ -295,6 +310,7 @@ __global__ void __launch_bounds__(THREADS) attn_ext_mma_kernel(const Params P) {
                     s[r][t][e] = v;
                     mx[i] = fmaxf(mx[i], v);
                 }
+            }
 #pragma unroll
             for (int i = 0; i < 2; ++i) {
                 mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], 1));

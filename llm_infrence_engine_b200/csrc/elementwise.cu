@@ -50,6 +50,31 @@ LLMIE_API int llmie_embed(const int* ids, const void* table, float* out, int N, 
     return launch_kernel(embed_kernel<bf16>, dim3(N), dim3(threads), 0, s, ids, (const bf16*)table, out, H, scale);
 }
 
+// x[n, :] = table[ids[n], :] * scale + pos_table[positions[n], :], widened to float before the sum
+template <typename T>
+__global__ void embed_positions_kernel(const int* __restrict__ ids, const T* __restrict__ table, const int* __restrict__ positions,
+                                       const T* __restrict__ pos_table, float* __restrict__ out, int H, float scale, int max_positions) {
+    pdl_trigger();
+    pdl_wait();
+    const int n = blockIdx.x;
+    const T* row = table + (size_t)ids[n] * H;
+    const T* pos = pos_table + (size_t)min(positions[n], max_positions - 1) * H;
+    float* o = out + (size_t)n * H;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) o[i] = fmaf(to_f32(row[i]), scale, to_f32(pos[i]));
+}
+
+LLMIE_API int llmie_embed_positions(const int* ids, const void* table, const int* positions, const void* pos_table, float* out, int N, int H,
+                                    int max_positions, int dtype, float scale, cudaStream_t s) {
+    if (N <= 0) return 0;
+    if (H <= 0 || max_positions <= 0) return LLMIE_ERR_BAD_ARGUMENT;
+    const int threads = H >= 1024 ? 256 : 128;
+    if (dtype == DT_F32)
+        return launch_kernel(embed_positions_kernel<float>, dim3(N), dim3(threads), 0, s, ids, (const float*)table, positions, (const float*)pos_table, out, H,
+                             scale, max_positions);
+    return launch_kernel(embed_positions_kernel<bf16>, dim3(N), dim3(threads), 0, s, ids, (const bf16*)table, positions, (const bf16*)pos_table, out, H, scale,
+                         max_positions);
+}
+
 // ------------------------------------------------------------------------------------------------
 // x[n, :] = table[ids[n], :] * scale + bigram[row(n), :], widened to float, with
 //   row(n) = (previous token * mul_prev + token * mul_cur) mod buckets, or `buckets` (the last row) for a request's first token.
@@ -405,8 +430,10 @@ LLMIE_API int llmie_rope_kv_write(void* in, void* out, const float* bias, const 
 // grid = (column blocks, rows); VEC = 4 moves four columns per thread.
 // `also_zero` (with `zero_n4` groups of four floats): another float32 accumulation buffer that this kernel clears on its way,
 // one that an earlier kernel of the step read but could not clear itself because several of its blocks read it.
+// `row_scale` (one number per row, or null) multiplies the row's results.
 template <typename TI, typename TO, int VEC>
-__global__ void silu_mul_kernel(TI* __restrict__ gu, TO* __restrict__ out, int I, int clear_in, float* __restrict__ also_zero, int zero_n4) {
+__global__ void silu_mul_kernel(TI* __restrict__ gu, TO* __restrict__ out, int I, int clear_in, float* __restrict__ also_zero, int zero_n4,
+                                const float* __restrict__ row_scale) {
     pdl_trigger();
     pdl_wait();
     if (also_zero) {
@@ -414,6 +441,7 @@ __global__ void silu_mul_kernel(TI* __restrict__ gu, TO* __restrict__ out, int I
         for (int i = (blockIdx.y * gridDim.x + blockIdx.x) * blockDim.x + threadIdx.x; i < zero_n4; i += threads)
             reinterpret_cast<float4*>(also_zero)[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    const float rs = row_scale ? row_scale[blockIdx.y] : 1.f;
     constexpr int PER = VEC == 4 ? 2 : 1;  // vectors per thread: two loads of gate and two of up are in flight together
     const int i0 = (blockIdx.x * blockDim.x + threadIdx.x) * VEC * PER;
     TI* row = gu + (size_t)blockIdx.y * 2 * I;
@@ -435,7 +463,7 @@ __global__ void silu_mul_kernel(TI* __restrict__ gu, TO* __restrict__ out, int I
         }
         float y[VEC];
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) y[j] = g[v][j] / (1.0f + expf(-g[v][j])) * u[v][j];
+        for (int j = 0; j < VEC; ++j) y[j] = g[v][j] / (1.0f + expf(-g[v][j])) * u[v][j] * rs;
         TO* o = out + (size_t)blockIdx.y * I + i;
         if constexpr (VEC == 4) store4(o, y); else *o = from_f32<TO>(y[0]);
     }
@@ -481,35 +509,36 @@ __global__ void __launch_bounds__(256) silu_mul_bf16x8_kernel(const bf16* __rest
 }
 
 template <typename TI, typename TO>
-static int launch_silu_mul(TI* gu, TO* out, int N, int I, int clear_in, float* also_zero, int zero_n4, cudaStream_t s) {
+static int launch_silu_mul(TI* gu, TO* out, int N, int I, int clear_in, float* also_zero, int zero_n4, const float* row_scale, cudaStream_t s) {
     if (N > 65535) {  // rows ride in grid.y; more rows than that go in slabs
         for (int n0 = 0; n0 < N; n0 += 65535) {
             const int rc = launch_silu_mul<TI, TO>(gu + (size_t)n0 * 2 * I, out + (size_t)n0 * I, min(65535, N - n0), I, clear_in,
-                                                   n0 == 0 ? also_zero : nullptr, zero_n4, s);
+                                                   n0 == 0 ? also_zero : nullptr, zero_n4, row_scale ? row_scale + n0 : nullptr, s);
             if (rc) return rc;
         }
         return 0;
     }
     const bool vec = I % 4 == 0 && ((uintptr_t)gu % 16 == 0) && ((uintptr_t)out % 16 == 0);
-    if (vec) return launch_kernel(silu_mul_kernel<TI, TO, 4>, dim3(((I + 7) / 8 + 127) / 128, N), dim3(128), 0, s, gu, out, I, clear_in, also_zero, zero_n4);
-    return launch_kernel(silu_mul_kernel<TI, TO, 1>, dim3((I + 127) / 128, N), dim3(128), 0, s, gu, out, I, clear_in, also_zero, zero_n4);
+    if (vec) return launch_kernel(silu_mul_kernel<TI, TO, 4>, dim3(((I + 7) / 8 + 127) / 128, N), dim3(128), 0, s, gu, out, I, clear_in, also_zero, zero_n4, row_scale);
+    return launch_kernel(silu_mul_kernel<TI, TO, 1>, dim3((I + 127) / 128, N), dim3(128), 0, s, gu, out, I, clear_in, also_zero, zero_n4, row_scale);
 }
 
 // also_zero / zero_floats: a float32 buffer (16-byte aligned, a multiple of 4 floats) that is cleared as well, or null.
+// row_scale: [N] floats, or null.
 LLMIE_API int llmie_silu_mul(void* gu, void* out, int N, int I, int clear_in, int in_dtype, int out_dtype, float* also_zero,
-                             long long zero_floats, cudaStream_t s) {
+                             long long zero_floats, const float* row_scale, cudaStream_t s) {
     if (N <= 0) return 0;
     if (also_zero && (((uintptr_t)also_zero & 15) || (zero_floats & 3) || zero_floats > (1ll << 32))) return LLMIE_ERR_BAD_ARGUMENT;
     const int n4 = also_zero ? (int)(zero_floats / 4) : 0;
-    if (in_dtype == DT_F32 && out_dtype == DT_F32) return launch_silu_mul<float, float>((float*)gu, (float*)out, N, I, clear_in, also_zero, n4, s);
+    if (in_dtype == DT_F32 && out_dtype == DT_F32) return launch_silu_mul<float, float>((float*)gu, (float*)out, N, I, clear_in, also_zero, n4, row_scale, s);
     if (in_dtype == DT_BF16 && out_dtype == DT_BF16) {
-        if (!clear_in && !also_zero && I % 8 == 0 && ((uintptr_t)gu % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
+        if (!clear_in && !also_zero && !row_scale && I % 8 == 0 && ((uintptr_t)gu % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
             const long long items = (long long)N * (I / 8);
             return launch_kernel(silu_mul_bf16x8_kernel, dim3((unsigned)(((items + 1) / 2 + 255) / 256)), dim3(256), 0, s, (const bf16*)gu, (bf16*)out, I, items);
         }
-        return launch_silu_mul<bf16, bf16>((bf16*)gu, (bf16*)out, N, I, clear_in, also_zero, n4, s);
+        return launch_silu_mul<bf16, bf16>((bf16*)gu, (bf16*)out, N, I, clear_in, also_zero, n4, row_scale, s);
     }
-    if (in_dtype == DT_F32 && out_dtype == DT_BF16) return launch_silu_mul<float, bf16>((float*)gu, (bf16*)out, N, I, clear_in, also_zero, n4, s);
+    if (in_dtype == DT_F32 && out_dtype == DT_BF16) return launch_silu_mul<float, bf16>((float*)gu, (bf16*)out, N, I, clear_in, also_zero, n4, row_scale, s);
     return LLMIE_ERR_BAD_ARGUMENT;
 }
 
@@ -579,12 +608,14 @@ LLMIE_API int llmie_kv_store(const void* z, int z_stride, int k_col, int v_col, 
 
 // ------------------------------------------------------------------------------------------------
 // out = act(in), elementwise in 32-bit. kind 0: the tanh form of GELU, 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)));
-// kind 1: a soft cap on a scaled input, param * tanh(scale z / param); kind 2: the exact GELU, 0.5 z (1 + erf(z / sqrt 2)); kind 3: scale z.
+// kind 1: a soft cap on a scaled input, param * tanh(scale z / param); kind 2: the exact GELU, 0.5 z (1 + erf(z / sqrt 2)); kind 3: scale z;
+// kind 4: the square of the positive part, max(z, 0)^2.
 // With `clear_in` the input is set to zero after it was read (a float32 accumulation buffer of a split-K product).
 __device__ __forceinline__ float act_of(float z, int kind, float param, float scale) {
     if (kind == 1) return param * tanhf(scale * z / param);
     if (kind == 2) return 0.5f * z * (1.0f + erff(0.7071067811865476f * z));
     if (kind == 3) return scale * z;
+    if (kind == 4) { const float r = fmaxf(z, 0.f); return r * r; }
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
@@ -622,8 +653,8 @@ __global__ void __launch_bounds__(128) act_vec_kernel(float* __restrict__ in, TO
 }
 
 // bfloat16 in and out, 8 elements (16 bytes) per thread. The result is rounded to bfloat16 (8 bits), so the hyperbolic tangent is
-// the fast 32-bit form (errors of about 1e-7). ERF: the exact GELU instead.
-template <bool ERF>
+// the fast 32-bit form (errors of about 1e-7). KIND: as in act_of, 0, 2 or 4.
+template <int KIND>
 __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict__ in, bf16* __restrict__ out, long long items) {
     pdl_trigger();
     pdl_wait();
@@ -639,7 +670,7 @@ __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict_
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
             const float v = z[2 * j + k];
-            y[k] = ERF ? gelu_erf_fast(v) : gelu_tanh_fast(v);
+            y[k] = KIND == 4 ? fmaxf(v, 0.f) * fmaxf(v, 0.f) : (KIND == 2 ? gelu_erf_fast(v) : gelu_tanh_fast(v));
         }
         const __nv_bfloat162 v2 = __floats2bfloat162_rn(y[0], y[1]);
         w[j] = *reinterpret_cast<const uint32_t*>(&v2);
@@ -650,11 +681,12 @@ __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict_
 LLMIE_API int llmie_act(void* in, void* out, long long total, int kind, int clear_in, float param, float scale, int in_dtype,
                         int out_dtype, cudaStream_t s) {
     if (total <= 0) return 0;
-    if (kind < 0 || kind > 3 || (kind == 1 && !(param > 0.f))) return LLMIE_ERR_BAD_ARGUMENT;
-    if ((kind == 0 || kind == 2) && in_dtype == DT_BF16 && out_dtype == DT_BF16 && !clear_in && total % 8 == 0 && ((uintptr_t)in % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
+    if (kind < 0 || kind > 4 || (kind == 1 && !(param > 0.f))) return LLMIE_ERR_BAD_ARGUMENT;
+    if ((kind == 0 || kind == 2 || kind == 4) && in_dtype == DT_BF16 && out_dtype == DT_BF16 && !clear_in && total % 8 == 0 && ((uintptr_t)in % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
         const dim3 blocks((unsigned)((total / 8 + 255) / 256));
-        if (kind == 2) return launch_kernel(act_bf16x8_kernel<true>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
-        return launch_kernel(act_bf16x8_kernel<false>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
+        if (kind == 2) return launch_kernel(act_bf16x8_kernel<2>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
+        if (kind == 4) return launch_kernel(act_bf16x8_kernel<4>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
+        return launch_kernel(act_bf16x8_kernel<0>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
     }
     if (in_dtype == DT_F32 && total % 4 == 0 && ((uintptr_t)in % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
         const dim3 blocks((unsigned)((total / 4 + 127) / 128));

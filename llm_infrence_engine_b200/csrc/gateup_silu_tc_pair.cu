@@ -63,7 +63,8 @@ __device__ __forceinline__ void cluster_sync_all() {
 // by side: the activation of the first half's sums goes to columns n of rows of 2 I, that of the second half's to columns I + n.
 template <int BN, int STAGES, int UNIT>
 __global__ void __launch_bounds__(THREADS<(UNIT >= PLAIN_GELU_ERF)>) gateup_silu_tc_pair_kernel(const __grid_constant__ CUtensorMap tmap_x, const __grid_constant__ CUtensorMap tmap_w,
-                                                                       bf16* __restrict__ out, int M, int I, int K, int* error_flag, float limit, float alpha, float shift) {
+                                                                       bf16* __restrict__ out, int M, int I, int K, int* error_flag, float limit, float alpha, float shift,
+                                                                       const float* __restrict__ row_scale) {
     constexpr int B_BYTES = BN * BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;   // this block's half of the weight rows of a K step
     constexpr bool PLAIN = UNIT >= PLAIN_GELU_ERF;
     extern __shared__ unsigned char raw[];
@@ -161,6 +162,7 @@ __global__ void __launch_bounds__(THREADS<(UNIT >= PLAIN_GELU_ERF)>) gateup_silu
             if (!ok) break;
             asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
             const uint32_t base = tmem + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(buf * 2 * BN);
+            const float rs = (!PLAIN && row_scale && m < M) ? row_scale[m] : 1.f;
             bf16* dst = out + (size_t)m * (PLAIN ? 2 * I : I) + n0;
 #pragma unroll 2
             for (int c = PLAIN ? ((warp - 2) >> 2) * 16 : 0; c < BN; c += PLAIN ? 32 : 16) {
@@ -175,8 +177,7 @@ __global__ void __launch_bounds__(THREADS<(UNIT >= PLAIN_GELU_ERF)>) gateup_silu
 #pragma unroll
                         for (int j = 0; j < 8; ++j) {
                             const float z0 = __uint_as_float(half ? uv[2 * j] : gv[2 * j]), z1 = __uint_as_float(half ? uv[2 * j + 1] : gv[2 * j + 1]);
-                            const __nv_bfloat162 v = UNIT == PLAIN_GELU_TANH ? __floats2bfloat162_rn(gelu_tanh_fast(z0), gelu_tanh_fast(z1))
-                                                                            : __floats2bfloat162_rn(gelu_erf_fast(z0), gelu_erf_fast(z1));
+                            const __nv_bfloat162 v = __floats2bfloat162_rn(plain_unit<UNIT>(z0), plain_unit<UNIT>(z1));
                             packed[j] = *reinterpret_cast<const uint32_t*>(&v);
                         }
                         if (m < M) {
@@ -192,7 +193,7 @@ __global__ void __launch_bounds__(THREADS<(UNIT >= PLAIN_GELU_ERF)>) gateup_silu
                 for (int j = 0; j < 8; ++j) {
                     const float a = gated_unit<UNIT>(__uint_as_float(gv[2 * j]), __uint_as_float(uv[2 * j]), limit, alpha, shift);
                     const float b = gated_unit<UNIT>(__uint_as_float(gv[2 * j + 1]), __uint_as_float(uv[2 * j + 1]), limit, alpha, shift);
-                    const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+                    const __nv_bfloat162 v = __floats2bfloat162_rn(a * rs, b * rs);
                     packed[j] = *reinterpret_cast<const uint32_t*>(&v);
                 }
                 if (m < M) {
@@ -237,7 +238,7 @@ inline int best_tile_width(long long m_pairs, int I, int pairs_at_once) {
 
 template <int BN, int UNIT>
 int launch_gateup_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, int K, int num_blocks, int* error_flag, float limit, float alpha,
-                  float shift, cudaStream_t s) {
+                  float shift, const float* row_scale, cudaStream_t s) {
     constexpr int STAGES = BN > 96 ? 6 : 7;   // 32 KB (BN = 128) to 24 KB (BN = 64) per stage
     CUtensorMap mx, mw;
     int rc = tensor_map(x, M, K, BM, &mx);
@@ -267,21 +268,21 @@ int launch_gateup_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, in
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.attrs = attr;
     cfg.numAttrs = llmie_pdl_flag ? 2 : 1;
-    return (int)cudaLaunchKernelEx(&cfg, gateup_silu_tc_pair_kernel<BN, STAGES, UNIT>, mx, mw, out, M, I, K, error_flag, limit, alpha, shift);
+    return (int)cudaLaunchKernelEx(&cfg, gateup_silu_tc_pair_kernel<BN, STAGES, UNIT>, mx, mw, out, M, I, K, error_flag, limit, alpha, shift, row_scale);
 }
 
 template <int UNIT>
 int dispatch_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, int K, int num_blocks, int* error_flag, float limit, float alpha,
-                 float shift, cudaStream_t s) {
+                 float shift, const float* row_scale, cudaStream_t s) {
     if (M <= 0 || I <= 0) return 0;
     if (K <= 0 || K % 8 || I % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ((uintptr_t)out & 15) || !error_flag || num_blocks < 2)
         return LLMIE_ERR_BAD_ARGUMENT;
     switch (best_tile_width(((M + BM - 1) / BM + 1) / 2, I, num_blocks / 2)) {
-        case 112: return launch_gateup_pair<112, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-        case 96: return launch_gateup_pair<96, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-        case 80: return launch_gateup_pair<80, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-        case 64: return launch_gateup_pair<64, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-        default: return launch_gateup_pair<128, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
+        case 112: return launch_gateup_pair<112, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, row_scale, s);
+        case 96: return launch_gateup_pair<96, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, row_scale, s);
+        case 80: return launch_gateup_pair<80, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, row_scale, s);
+        case 64: return launch_gateup_pair<64, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, row_scale, s);
+        default: return launch_gateup_pair<128, UNIT>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, row_scale, s);
     }
 }
 
@@ -291,22 +292,24 @@ int dispatch_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, int K, 
 // limit > 0: the epilogue is min(g, limit) * sigmoid(alpha g) * (clamp(u, -limit, limit) + shift); limit == 0: silu(g) * u;
 // limit < 0: gelu_tanh(g) * u.
 LLMIE_API int llmie_gateup_glu_tc_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, int K, int num_blocks, int* error_flag,
-                                        float limit, float alpha, float shift,
+                                        float limit, float alpha, float shift, const float* row_scale,
                                         cudaStream_t s) {
-    if (limit > 0.f) return dispatch_pair<UNIT_CLAMPED>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-    if (limit < 0.f) return dispatch_pair<UNIT_GELU_TANH>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
-    return dispatch_pair<UNIT_SILU>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, s);
+    // row_scale: [M] floats that multiply the rows' results, or null
+    if (limit > 0.f) return dispatch_pair<UNIT_CLAMPED>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, row_scale, s);
+    if (limit < 0.f) return dispatch_pair<UNIT_GELU_TANH>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, row_scale, s);
+    return dispatch_pair<UNIT_SILU>(x, w, out, M, I, K, num_blocks, error_flag, limit, alpha, shift, row_scale, s);
 }
 
 // The same with silu(gate) * up as the epilogue.
 LLMIE_API int llmie_gateup_silu_tc_pair(const bf16* x, const bf16* w, bf16* out, int M, int I, int K, int num_blocks, int* error_flag, cudaStream_t s) {
-    return llmie_gateup_glu_tc_pair(x, w, out, M, I, K, num_blocks, error_flag, 0.f, 1.f, 0.f, s);
+    return llmie_gateup_glu_tc_pair(x, w, out, M, I, K, num_blocks, error_flag, 0.f, 1.f, 0.f, nullptr, s);
 }
 
-// act(x w^T) for w [N, K]: the same product without a gate; N a multiple of 16. tanh_form: the tanh form of GELU instead of the exact one.
-LLMIE_API int llmie_up_gelu_tc_pair(const bf16* x, const bf16* w, bf16* out, int M, int N, int K, int num_blocks, int* error_flag, int tanh_form,
+// act(x w^T) for w [N, K]: the same product without a gate; N a multiple of 16. form 0: the exact GELU, 1: its tanh form, 2: max(z, 0)^2.
+LLMIE_API int llmie_up_gelu_tc_pair(const bf16* x, const bf16* w, bf16* out, int M, int N, int K, int num_blocks, int* error_flag, int form,
                                  cudaStream_t s) {
     if (N % 16) return LLMIE_ERR_BAD_ARGUMENT;
-    if (tanh_form) return dispatch_pair<PLAIN_GELU_TANH>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, s);
-    return dispatch_pair<PLAIN_GELU_ERF>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, s);
+    if (form == 2) return dispatch_pair<PLAIN_RELU2>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, nullptr, s);
+    if (form == 1) return dispatch_pair<PLAIN_GELU_TANH>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, nullptr, s);
+    return dispatch_pair<PLAIN_GELU_ERF>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, nullptr, s);
 }

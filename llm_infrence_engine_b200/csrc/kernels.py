@@ -92,6 +92,11 @@ class CudaKernels:
         self._pending_post: Optional[tuple] = None
         # ... and one that a Dynamic Tanh closes waits here: (stream, result, alpha, weight, bias)
         self._pending_tanh: Optional[tuple] = None
+        # ... one that an RMS norm closes waits here: (stream, (a, b, weight of a, weight of b, factor), the norm's weight, eps): the result
+        # is a, or (b not None) factor * (a / rms(a) * weight of a + b / rms(b) * weight of b)
+        self._pending_rms: Optional[tuple] = None
+        # two results side by side that are to be normed and summed into a zeroed tensor: (tensor, a, b, weight of a, weight of b, eps, factor)
+        self._pending_mix: Optional[tuple] = None
         self._state_lists: dict = {}   # the addresses of a runner's state tensors on the device (zero_fresh_states)
         self._fresh: list = []   # zeroed tensors of ``zeros_like_rows`` that nothing has been added into yet
         # ``zeros_like_rows`` hands out views of one float32 buffer that is zero between uses: the stream kernels that read a
@@ -119,7 +124,7 @@ class CudaKernels:
                    "llmie_moe_tile_rows", "llmie_moe_router", "llmie_moe_gather", "llmie_moe_grouped_tc", "llmie_moe_grouped_tc_rows",
                    "llmie_embed_add", "llmie_mlstm_prepare", "llmie_mlstm_scan", "llmie_mlstm_finish", "llmie_paged_attention_talk",
                    "llmie_attention_talk_slice", "llmie_attention_talk_mma_fits", "llmie_paged_attention_talk_mma", "llmie_embed_bigram",
-                   "llmie_dynamic_tanh"):
+                   "llmie_dynamic_tanh", "llmie_embed_positions", "llmie_post_rms", "llmie_qk_rows_norm_store", "llmie_linear_attention_scan"):
             getattr(self.lib, fn).restype = ctypes.c_int
         # two forms of the gate/up kernel live in source files of their own, and the library also builds without them
         self._gate_up_cluster = self._gate_up_pair = self._gate_up_glu_pair = self._up_gelu_pair = None
@@ -152,6 +157,8 @@ class CudaKernels:
         self._pending_streams = None
         self._pending_post = None
         self._pending_tanh = None
+        self._pending_rms = None
+        self._pending_mix = None
         self._fresh = []
         self._dirty_qkv = None
         for t in [self._acc, self._acc_qkv, *self._zero_bufs, *self._retired_acc]:
@@ -199,6 +206,20 @@ class CudaKernels:
         out = torch.empty((N, H), dtype=torch.float32, device=table.device)
         self._check(self.lib.llmie_embed(_ptr(token_ids), _ptr(table), _ptr(out), N, H, self._dt(table, "table"), ctypes.c_float(scale),
                                         self._stream()), "embed")
+        return out
+
+    def embed_positions(self, token_ids, table, positions, position_table, scale: float = 1.0):
+        """``table[token] * scale + position_table[position]`` in 32-bit."""
+        self._need(token_ids, "token_ids", torch.int32, 1)
+        self._need(positions, "positions", torch.int32, 1)
+        self._need(table, "table", None, 2)
+        self._need(position_table, "position_table", table.dtype, 2)
+        N, H = token_ids.shape[0], table.shape[1]
+        if position_table.shape[1] != H or positions.shape[0] != N:
+            raise KernelError("embed_positions: the position table must be as wide as the embedding, with a position per token")
+        out = torch.empty((N, H), dtype=torch.float32, device=table.device)
+        self._check(self.lib.llmie_embed_positions(_ptr(token_ids), _ptr(table), _ptr(positions), _ptr(position_table), _ptr(out), N, H,
+                                                   position_table.shape[0], self._dt(table, "table"), ctypes.c_float(scale), self._stream()), "embed_positions")
         return out
 
     def embed_bigram(self, token_ids, table, bigram, buckets: int, mul_prev: int, mul_cur: int, positions, token_seq, seq_starts, num_seqs: int, last,
@@ -322,6 +343,10 @@ class CudaKernels:
             N, S, H = xs.shape
             self._check(self.lib.llmie_streams_update(_ptr(xs), _ptr(y), self._dt(y, "y"), int(self._clears(y)), _ptr(mix), _ptr(coef_out), N, S, H,
                                                       self._stream()), "streams_update")
+        if self._pending_mix is not None:
+            y, a, b, wa, wb, eps, coef = self._pending_mix
+            self._pending_mix = None
+            self._dual_mix_now(y, a, b, wa, wb, eps, coef)
         if self._pending_post is not None:
             x, y, w_post, eps, plain = self._pending_post
             self._pending_post = None
@@ -330,6 +355,13 @@ class CudaKernels:
             x, y, alpha, weight, bias = self._pending_tanh
             self._pending_tanh = None
             self._dynamic_tanh(x, (y, alpha, weight, bias), None, None, None, "post_tanh_add")
+        self._flush_rms()
+
+    def _flush_rms(self) -> None:
+        if self._pending_rms is not None:
+            x, parts, w_post, eps = self._pending_rms
+            self._pending_rms = None
+            self._post_rms(x, parts, w_post, eps, None, None, None, "post_rms_add")
 
     def _take_pending(self, residual, out_dtype):
         """The put-off addend for ``residual`` if there is one that the norm kernel can add on its way (same dtype as its output)."""
@@ -350,6 +382,11 @@ class CudaKernels:
         return self._norm(residual, delta, weight, eps, None, out_dtype, "add_rmsnorm")
 
     def rmsnorm_rows(self, residual, delta, weight, eps, rows, out_dtype):
+        if delta is None and self._rms_waits_for(residual) and self._pending_rms[3] == eps:
+            _, parts, w_post, _ = self._pending_rms
+            self._pending_rms = None
+            self._need(weight, "weight", torch.float32, 1)
+            return self._post_rms(residual, parts, w_post, eps, weight, rows, out_dtype, "rmsnorm_rows")
         self.flush()
         return self._norm(residual, delta, weight, eps, rows, out_dtype, "rmsnorm_rows")
 
@@ -414,8 +451,8 @@ class CudaKernels:
             return self.linear_tc(x, w, out=self._transient(M, N, w.device), accumulate=True, bias=bias)
         if small and out_dtype == torch.float32:
             return self.linear_tc(x, w, bias=bias)
-        if bf16 and out_dtype == torch.float32 and self.use_tc_gemm and K % 8 == 0 and N <= 128:
-            # few outputs in 32-bit for many rows (a router's logits over a prompt portion): one tile of weight rows, a block per 64 rows
+        if bf16 and out_dtype == torch.float32 and self.use_tc_gemm and K % 8 == 0 and N <= 520:
+            # few outputs in 32-bit for many rows (a router's logits over a prompt portion): a few tiles of weight rows, a block per 64 rows
             return self.linear_tc(x, w, bias=bias)
         if self.use_cublas and bf16 and out_dtype == torch.bfloat16:
             self.launches += 1
@@ -823,12 +860,17 @@ class CudaKernels:
         return self.paged_attention(qkv, k_pool, v_pool, block_table, token_seq, positions, num_heads, num_kv_heads, head_dim, page_size,
                                     scale, window, max_context, batch=batch)
 
-    def gate_up_act(self, x, w_gate_up, out_dtype=None, glu=None, activation="silu"):
+    def gate_up_act(self, x, w_gate_up, out_dtype=None, glu=None, activation="silu", row_scale=None):
         """``silu(x Wg^T) * (x Wu^T)`` for the fused matrix ``w_gate_up`` ``[2 I, K]`` (gate rows first). Prompt portions in
         bfloat16 take one tcgen05 kernel whose epilogue is the activation (the float32 sums stay in tensor memory; nothing of
         width 2 I is written); everything else is the product followed by ``silu_mul``. ``glu = (limit, alpha, shift)`` asks for
-        the clamped unit ``g sigmoid(alpha g) (u + shift)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)`` instead."""
+        the clamped unit ``g sigmoid(alpha g) (u + shift)`` with ``g = min(gate, limit)``, ``u = clamp(up, -limit, limit)`` instead.
+        ``row_scale`` (float32, one number per row): multiplies the row's results (with silu only)."""
         out_dtype = out_dtype or x.dtype
+        if row_scale is not None:
+            self._need(row_scale, "row_scale", torch.float32)
+            if row_scale.numel() != x.shape[0] or glu is not None or activation != "silu":
+                raise KernelError("gate_up_act: a scale per row needs one number per row, and is built with silu only")
         limit, alpha, shift = (float(v) for v in glu) if glu is not None else (0.0, 1.0, 0.0)
         if glu is not None and not limit > 0:
             raise KernelError("gate_up_act: the clamped unit needs a positive limit")
@@ -845,24 +887,24 @@ class CudaKernels:
             # three forms of the kernel: one block per tile of 128 rows; pairs of multiprocessors on tiles of 256 rows
             # (cta_group::2), the default for long portions; pairs of blocks that share their weight rows by TMA multicast,
             # where the library was built with that optional source file (off by default: measured no faster)
-            fn = self._gate_up_cluster if (self.use_cluster_gate_up and M > 128 and glu is None) else None
+            fn = self._gate_up_cluster if (self.use_cluster_gate_up and M > 128 and glu is None and row_scale is None) else None
             pair = self.use_pair_gate_up and self._gate_up_pair is not None and M >= self.pair_gate_up_min_rows
-            if pair and glu is None:
+            if pair and glu is None and row_scale is None:
                 fn = self._gate_up_pair
-            if fn is not None or glu is None:
+            if fn is not None or (glu is None and row_scale is None):
                 fn = fn or self.lib.llmie_gateup_silu_tc
                 self._check(fn(_ptr(x), _ptr(w_gate_up), _ptr(out), M, I, K_, self.num_sms, _ptr(self._errors(x.device)), self._stream()),
                             "gate_up_act (tcgen05)")
                 return out
             fn = self._gate_up_glu_pair if (pair and self._gate_up_glu_pair is not None) else self.lib.llmie_gateup_glu_tc
             self._check(fn(_ptr(x), _ptr(w_gate_up), _ptr(out), M, I, K_, self.num_sms, _ptr(self._errors(x.device)), ctypes.c_float(limit),
-                           ctypes.c_float(alpha), ctypes.c_float(shift), self._stream()), "gate_up_act (tcgen05, clamped unit)")
+                           ctypes.c_float(alpha), ctypes.c_float(shift), _ptr(row_scale), self._stream()), "gate_up_act (tcgen05, clamped unit)")
             return out
         if glu is not None:
             return self.glu_clamped(self.linear(x, w_gate_up, transient=True), limit, alpha, shift, out_dtype)
-        return self.silu_mul(self.linear(x, w_gate_up, transient=True), out_dtype)
+        return self.silu_mul(self.linear(x, w_gate_up, transient=True), out_dtype, row_scale)
 
-    def silu_mul(self, gu, out_dtype=None):
+    def silu_mul(self, gu, out_dtype=None, row_scale=None):
         """``silu(gate) * up`` of a fused gate/up projection ``[rows, 2 I]`` (gate first); a transient float32 input is consumed and cleared."""
         self._need(gu, "gate_up", None, 2)
         if gu.shape[1] % 2:
@@ -873,7 +915,7 @@ class CudaKernels:
         dirty, self._dirty_qkv = self._dirty_qkv, None
         self._check(self.lib.llmie_silu_mul(_ptr(gu), _ptr(out), N, I, int(self._is_transient(gu)), self._dt(gu, "gate_up"),
                                             self._dt(out, "out"), _ptr(dirty), ctypes.c_longlong(0 if dirty is None else dirty.numel()),
-                                            self._stream()), "silu_mul")
+                                            _ptr(row_scale), self._stream()), "silu_mul")
         return out
 
     # ------------------------------------------------------------------ several residual streams
@@ -977,7 +1019,7 @@ class CudaKernels:
     # ------------------------------------------------------------------ a product with an activation behind it
     def linear_act(self, x, w, activation, out_dtype=None):
         """``act(x w^T)``; the activation is computed in 32-bit on the product's sums where those are at hand (small batches)."""
-        kinds = {"gelu_tanh": 0, "gelu_erf": 2}
+        kinds = {"gelu_tanh": 0, "gelu_erf": 2, "relu2": 4}
         if activation not in kinds:
             raise KernelError(f"linear_act: activation '{activation}' is not built")
         out_dtype = out_dtype or x.dtype
@@ -987,7 +1029,7 @@ class CudaKernels:
             # prompt portions: one tcgen05 kernel whose epilogue is the activation (the gate/up kernels without a gate)
             out = torch.empty((M, w.shape[0]), dtype=torch.bfloat16, device=x.device)
             fn = self._up_gelu_pair if (self.use_pair_gate_up and self._up_gelu_pair is not None and M >= self.pair_gate_up_min_rows) else self.lib.llmie_up_gelu_tc
-            self._check(fn(_ptr(x), _ptr(w), _ptr(out), M, w.shape[0], K_, self.num_sms, _ptr(self._errors(x.device)), int(activation == "gelu_tanh"),
+            self._check(fn(_ptr(x), _ptr(w), _ptr(out), M, w.shape[0], K_, self.num_sms, _ptr(self._errors(x.device)), {"gelu_erf": 0, "gelu_tanh": 1, "relu2": 2}[activation],
                            self._stream()), "linear_act (tcgen05)")
             return out
         z = self.linear(x, w, transient=True)
@@ -1024,7 +1066,7 @@ class CudaKernels:
     def attention_ext(self, q, q_col, num_heads, num_kv_heads, head_dim, v_head_dim, k_pool, v_pool, block_table, token_seq, positions,
                       page_size, scale, window, max_context, temp=(0.0, 0), rel=None, rel_rows=None, sink=None, gate=None, gate_col=0,
                       gate_per_head=False, batch=None, num_splits=None, keep_first=0, chunk=0, softcap=0.0, talk=None,
-                      sigmoid_bias=None, log_distance=None, turn=None):
+                      sigmoid_bias=None, log_distance=None, turn=None, key_scale=None):
         """Paged attention with extras: the query heads are columns ``q_col ..`` of ``q``; ``v_pool=None`` reads the values out
         of the key rows (their first ``v_head_dim`` entries); ``temp=(coef, every)`` a query temperature by position;
         ``rel [rows, heads]`` with ``rel_rows`` (distance -> row) a bias by distance; ``sink [heads]`` joins the denominator;
@@ -1035,7 +1077,9 @@ class CudaKernels:
         ``log_distance = (r1, r2)`` (float32, one number per head each) takes ``r1 ln(1 + r2 (p - j))`` off the scaled score;
         ``sigmoid_bias [heads]`` (float32): no softmax, a visible key's weight is ``sigmoid(score + bias)``;
         ``turn = (cos, sin, neighbours)`` with ``[N, v_head_dim / 2]`` tables: every head's result is turned back by these angles (pairs half
-        the values apart, or neighbours), for values that were turned when they were cached."""
+        the values apart, or neighbours), for values that were turned when they were cached;
+        ``key_scale [pages, page_size]`` (float32): a number per cached token that multiplies its keys' scores (before cap and bias), not the
+        values that may lie in the same rows."""
         self._need(q, "q", None, 2)
         dt = self._dt(q, "q")
         N = q.shape[0]
@@ -1084,13 +1128,17 @@ class CudaKernels:
                 self._need(t, name, torch.float32, 2)
                 if v_head_dim % 2 or tuple(t.shape) != (N, v_head_dim // 2):
                     raise KernelError("attention_ext: the turn's tables must be [tokens, v_head_dim / 2] with v_head_dim even")
+        if key_scale is not None:
+            self._need(key_scale, "key_scale", torch.float32, 2)
+            if tuple(key_scale.shape) != (k_pool.shape[0], page_size):
+                raise KernelError(f"attention_ext: key_scale is {list(key_scale.shape)}, expected [{k_pool.shape[0]}, {page_size}]")
         more = (_ptr(sigmoid_bias), _ptr(log_distance[0] if log_distance is not None else None), _ptr(log_distance[1] if log_distance is not None else None),
-                _ptr(turn[0] if turn is not None else None), _ptr(turn[1] if turn is not None else None), int(bool(turn[2])) if turn is not None else 0)
+                _ptr(turn[0] if turn is not None else None), _ptr(turn[1] if turn is not None else None), int(bool(turn[2])) if turn is not None else 0, _ptr(key_scale))
         out = torch.empty((N, num_heads * v_head_dim), dtype=q.dtype, device=q.device)
         esize = q.element_size()
         if talk is not None:
-            if sigmoid_bias is not None or log_distance is not None or turn is not None:
-                raise KernelError("attention_ext: talking heads are not built together with sigmoid weights, a penalty by distance or turned values")
+            if sigmoid_bias is not None or log_distance is not None or turn is not None or key_scale is not None:
+                raise KernelError("attention_ext: talking heads are not built together with sigmoid weights, a penalty by distance, turned values or scaled keys")
             return self._attention_talk(q, q_col, num_heads, num_kv_heads, head_dim, v_head_dim, k_pool, v_pool, block_table, token_seq, positions,
                                         page_size, scale, window, max_context, talk, sink, gate, gate_col, gate_mode, keep_first, chunk, softcap,
                                         temp, rel, out, batch)
@@ -1098,7 +1146,7 @@ class CudaKernels:
             raise KernelError("attention_ext: keep_first needs a window, and keep_first, chunk and softcap cannot be negative")
         if (self.use_plain_attention_for_ext and self.use_mma_attention and dt == 1 and batch is not None and v_pool is not None and head_dim == v_head_dim
                 and head_dim in (64, 128) and q_col == 0 and q.shape[1] % 8 == 0 and not (keep_first or chunk or softcap or temp[1]) and rel is None
-                and sink is None and gate is None and (turn is None or not turn[2]) and (log_distance is None or sigmoid_bias is not None) and scale > 0
+                and key_scale is None and sink is None and gate is None and (turn is None or not turn[2]) and (log_distance is None or sigmoid_bias is not None) and scale > 0
                 and num_heads // num_kv_heads <= (16 if batch.max_seq_len == 1 else 64) and (num_splits is None or num_splits <= 16)):
             done = self._attention_mma(q, k_pool, v_pool, block_table, token_seq, positions, out, num_heads, num_kv_heads, head_dim, page_size, scale,
                                        int(window), min(max_context, window) if window else max_context, batch, num_splits, turn, sigmoid_bias, log_distance)
@@ -1106,12 +1154,13 @@ class CudaKernels:
                 return done
         max_rows = 0
         tensor_cores = dt == 1 and self.use_mma_attention_ext and batch is not None and (q_col * esize) % 16 == 0 and q.shape[1] % 8 == 0
-        masked = bool(keep_first or chunk or softcap)
+        masked = bool(keep_first or chunk or softcap or key_scale is not None)
         if sigmoid_bias is not None and (masked or rel is not None):
             tensor_cores = False   # (the tensor-core kernels know sigmoid weights under a causal mask and a window)
         if masked and not self.masked_attention_tensor_cores:
             tensor_cores = False
         if (tensor_cores and self.use_fa_attention_ext and batch.max_seq_len > 1
+                and (v_pool is not None or key_scale is not None)   # (latent rows, which all heads share, keep the other kernel)
                 and self.lib.llmie_attention_ext_fa_fits(head_dim, v_head_dim, int(v_pool is not None), num_heads // num_kv_heads)):
             # steps with prompt portions, heads of 64 or 128: tiles of 64 rows, a warp to 16 rows and all of a chunk's keys
             group = num_heads // num_kv_heads
@@ -1345,6 +1394,79 @@ class CudaKernels:
         self._need(weight, "weight", torch.float32, 1)
         self._pending_post = (residual, y, weight, 0.0, True)
 
+    # ------------------------------------------------------------------ a stream that is read as it is, results that are RMS-normed
+    def _rms_waits_for(self, residual) -> bool:
+        """True if a closing RMS norm of this stream waits and nothing else does, so that the stream's next reader can do both."""
+        return (self._pending_rms is not None and self._pending_rms[0] is residual and self._pending_add is None and self._pending_streams is None
+                and self._pending_post is None and self._pending_tanh is None and self._pending_mix is None)
+
+    def _post_rms(self, x, parts, w_post, eps, w_pre, rows, out_dtype, what):
+        """``x += u / rms(u) * w_post`` for the result ``u`` that ``parts`` describes (None: no addition), then, with ``out_dtype``, the
+        stream's rows rounded to it, or (``w_pre``) normed. With ``rows`` only those are computed, and the stream is not stored."""
+        self._need(x, "residual", torch.float32, 2)
+        N, H = x.shape
+        a = b = wa = wb = None
+        coef = 1.0
+        if parts is not None:
+            a, b, wa, wb, coef = parts
+            for name, t, w in (("the sublayer's result", a, None), ("the first result", None, wa), ("the second result", b, wb)):
+                if t is not None:
+                    self._need(t, name, None, 2)
+                    if tuple(t.shape) != (N, H):
+                        raise KernelError(f"{what}: {name} is {list(t.shape)}, the stream is {list(x.shape)}")
+                if w is not None:
+                    self._need(w, f"the weight of {name}", torch.float32, 1)
+        for w in (wa, wb, w_post, w_pre):
+            if w is not None:
+                self._need(w, "a norm's weight", torch.float32, 1)
+                if w.shape[0] != H:
+                    raise KernelError(f"{what}: a norm's weight has {w.shape[0]} entries, rows have {H}")
+        if rows is not None:
+            self._need(rows, "rows", torch.int32, 1)
+        n_out = N if rows is None else rows.shape[0]
+        out = torch.empty((n_out, H), dtype=out_dtype, device=x.device) if out_dtype is not None else None
+        mode = 0 if out is None else (1 if w_pre is None else 2)
+        clear = [t for t in (a, b) if t is not None and self._clears(t)]
+        self._check(self.lib.llmie_post_rms(_ptr(x), _ptr(a), 0 if a is None else self._dt(a, "a"), int(a is not None and self._clears(a)), _ptr(b),
+                                            0 if b is None else self._dt(b, "b"), int(b is not None and self._clears(b)), _ptr(wa), _ptr(wb),
+                                            ctypes.c_float(coef), _ptr(w_post if parts is not None else None), _ptr(w_pre), _ptr(out),
+                                            0 if out is None else _DT[out_dtype], mode, _ptr(rows), n_out, H, ctypes.c_float(eps), self._stream()), what)
+        if rows is not None:
+            for t in clear:   # only the chosen rows were read and cleared; the buffer must be zero for its next user
+                t.zero_()
+                self.launches += 1
+        return out
+
+    def stream_rows(self, residual, out_dtype):
+        """The stream's rows as they are, in ``out_dtype`` (float32: the stream itself). A closing norm that still waits (``post_rms_add``)
+        is carried out by the same kernel."""
+        parts = w_post = None
+        eps = 0.0
+        if self._rms_waits_for(residual):
+            _, parts, w_post, eps = self._pending_rms
+            self._pending_rms = None
+        else:
+            self.flush()
+        if out_dtype == torch.float32:
+            if parts is not None:
+                self._post_rms(residual, parts, w_post, eps, None, None, None, "stream_rows")
+            return residual
+        return self._post_rms(residual, parts, w_post, eps, None, None, out_dtype, "stream_rows")
+
+    def post_rms_add(self, residual, y, weight, eps):
+        """``residual += y / sqrt(mean(y^2) + eps) * weight``: put off until the stream is read next (``stream_rows``, ``rmsnorm_rows``) or
+        until ``flush``. ``y`` is a zeroed tensor of ``zeros_like_rows`` that the sublayer added its result into; two results that only
+        wait to be normed and summed into it (``dual_rmsnorm_mix``) are taken over as they are."""
+        self._flush_rms()
+        mix = self._pending_mix
+        if mix is not None and mix[0] is y and mix[5] == eps and self._pending_add is None:
+            self._pending_mix = None
+            self._unfresh(y)
+            self._pending_rms = (residual, (mix[1], mix[2], mix[3], mix[4], mix[6]), weight, float(eps))
+            return
+        y = self.take_result(y)
+        self._pending_rms = (residual, (y, None, None, None, 1.0), weight, float(eps))
+
     # ------------------------------------------------------------------ Dynamic Tanh in place of a norm
     def _dynamic_tanh(self, x, post, pre, rows, out_dtype, what):
         """``x += tanh(a y) * w + b`` for ``post = (y, a, w, b)``, then ``tanh(a x) * w + b`` for ``pre = (a, w, b)``; either may be None."""
@@ -1421,7 +1543,8 @@ class CudaKernels:
         return out
 
     def dual_rmsnorm_mix(self, a, b, weight_a, weight_b, eps, coef, add_to):
-        """``add_to += coef * (a / rms(a) * weight_a + b / rms(b) * weight_b)`` row by row (``add_to`` float32)."""
+        """``add_to += coef * (a / rms(a) * weight_a + b / rms(b) * weight_b)`` row by row (``add_to`` float32). Into a tensor of
+        ``zeros_like_rows`` that holds nothing yet it is put off: whoever takes that tensor's result may do it on the way."""
         self.flush()
         self._need(add_to, "add_to", torch.float32, 2)
         N, H = add_to.shape
@@ -1431,6 +1554,13 @@ class CudaKernels:
                 raise KernelError(f"dual_rmsnorm_mix: {name} is {list(t.shape)}, the target is {list(add_to.shape)}")
         self._need(weight_a, "weight_a", torch.float32, 1)
         self._need(weight_b, "weight_b", torch.float32, 1)
+        if self._is_fresh(add_to):
+            self._pending_mix = (add_to, a, b, weight_a, weight_b, float(eps), float(coef))
+            return
+        self._dual_mix_now(add_to, a, b, weight_a, weight_b, eps, coef)
+
+    def _dual_mix_now(self, add_to, a, b, weight_a, weight_b, eps, coef) -> None:
+        N, H = add_to.shape
         self._check(self.lib.llmie_dual_rmsnorm_mix(_ptr(a), self._dt(a, "a"), _ptr(b), self._dt(b, "b"), _ptr(weight_a), _ptr(weight_b), _ptr(add_to),
                                                     N, H, ctypes.c_float(eps), ctypes.c_float(coef), 1, int(self._clears(a)), int(self._clears(b)), self._stream()),
                     "dual_rmsnorm_mix")
@@ -1504,6 +1634,44 @@ class CudaKernels:
                                                       _ptr(k_pool if write_kv else None), _ptr(v_pool if write_kv else None), N, num_heads, num_kv_heads, head_dim,
                                                       v_head_dim, page_size, int(bool(write_kv)), int(clear), self._dt(z, "z"), _DT[out_dtype], self._stream()), "qk_norm_rope_store")
         return q
+
+    def qk_rows_norm_store(self, z, num_heads, num_kv_heads, head_dim, v_head_dim, q_weight, k_weight, eps, slot_mapping, k_pool, v_pool, key_scale,
+                           page_size, gate_cols=0, write_kv=True, out_dtype=None):
+        """From rows ``z = [query heads | key heads | value heads | gate columns]``: RMS norm of the whole query row and of the whole key
+        row, with a weight per entry. Keys and values go to the tokens' cache slots; returns rows ``[normed queries | gate columns | zeros]``
+        of a multiple of 8 entries. With ``key_scale [pages, page_size]`` the values ARE the keys: ``z`` has no value heads, the keys are
+        stored as they are before the norm, its reciprocal root mean square is stored in ``key_scale`` (the attention multiplies the
+        scores by it) and its weight is multiplied into the queries. ``z`` may be a product's transient sums, which are consumed and cleared."""
+        self._need(z, "z", None, 2)
+        N = z.shape[0]
+        Q, KW = num_heads * head_dim, num_kv_heads * head_dim
+        if num_heads % num_kv_heads or z.shape[1] < Q + KW + (0 if key_scale is not None else num_kv_heads * v_head_dim) + gate_cols:
+            raise KernelError("qk_rows_norm_store: the rows are too short for the heads")
+        for name, t, width in (("q_weight", q_weight, Q), ("k_weight", k_weight, KW)):
+            self._need(t, name, torch.float32, 1)
+            if t.shape[0] != width:
+                raise KernelError(f"qk_rows_norm_store: {name} needs one entry per element of the row ({width})")
+        out_dtype = out_dtype or z.dtype
+        clear = self._is_transient(z)
+        if write_kv:
+            self._need(slot_mapping, "slot_mapping", torch.int32, 1)
+            pools = [("k_pool", k_pool, head_dim)] + ([("v_pool", v_pool, v_head_dim)] if key_scale is None else [])
+            for name, pool, d in pools:
+                self._need(pool, name, out_dtype, 4)
+                if tuple(pool.shape[1:]) != (num_kv_heads, page_size, d):
+                    raise KernelError(f"qk_rows_norm_store: {name} is {list(pool.shape)}, expected [pages, {num_kv_heads}, {page_size}, {d}]")
+        if key_scale is not None:
+            self._need(key_scale, "key_scale", torch.float32, 2)
+            if key_scale.shape[1] != page_size:
+                raise KernelError("qk_rows_norm_store: key_scale must be [pages, page_size]")
+        width = Q + gate_cols + -(Q + gate_cols) % 8
+        out = torch.empty((N, width), dtype=out_dtype, device=z.device)
+        self._check(self.lib.llmie_qk_rows_norm_store(_ptr(z), z.shape[1], _ptr(out), width, _ptr(q_weight), _ptr(k_weight), ctypes.c_float(eps),
+                                                      _ptr(slot_mapping if write_kv else None), _ptr(k_pool if write_kv else None),
+                                                      _ptr(v_pool if write_kv and key_scale is None else None), _ptr(key_scale), N, num_heads,
+                                                      num_kv_heads, head_dim, v_head_dim, page_size, int(gate_cols), int(bool(write_kv)), int(clear),
+                                                      self._dt(z, "z"), _DT[out_dtype], self._stream()), "qk_rows_norm_store")
+        return out
 
     # ------------------------------------------------------------------ mixers with a state of fixed size
     def causal_conv(self, z, col, channels, weight, bias, state, batch, activation=None):
@@ -1596,6 +1764,25 @@ class CudaKernels:
                                             _ptr(out), H, G, NS, DV, batch.num_seqs, batch.max_seq_len, self._dt(xbc, "xbc"), self._stream()), "ssm_scan")
         return out
 
+    def linear_attention(self, z, q_col, k_col, v_col, num_heads, head_dim, v_head_dim, decay, state, batch):
+        """Linear attention with a fixed decay per head over the rows of each request: per head ``S <- decay[h] S + k v^T``, ``o = S^T q`` with
+        ``q``, ``k`` (``heads * head_dim`` columns of ``z`` from ``q_col``, ``k_col``) and ``v`` (``heads * v_head_dim`` from ``v_col``) passing silu
+        first; from ``state [slots, heads, v_head_dim, head_dim]`` (a head's ``S`` kept column by column), which is moved on. Returns float32
+        ``[N, heads * v_head_dim]``."""
+        self._need(z, "z", None, 2)
+        self._need(state, "state", torch.float32, 4)
+        self._need(decay, "decay", torch.float32, 1)
+        H, D, DV = num_heads, head_dim, v_head_dim
+        if max(q_col, k_col) + H * D > z.shape[1] or v_col + H * DV > z.shape[1] or D > 256 or decay.shape[0] != H:
+            raise KernelError("linear_attention: the rows or the decays do not fit the heads (head_dim at most 256)")
+        if tuple(state.shape[1:]) != (H, DV, D):
+            raise KernelError(f"linear_attention: state is {list(state.shape)}, expected [slots, {H}, {DV}, {D}]")
+        out = torch.empty((z.shape[0], H * DV), dtype=torch.float32, device=z.device)
+        self._check(self.lib.llmie_linear_attention_scan(_ptr(z), z.shape[1], int(q_col), int(k_col), int(v_col), _ptr(decay), _ptr(state),
+                                                         _ptr(batch.seq_starts_dev), _ptr(batch.seq_slots), _ptr(out), H, D, DV, batch.num_seqs,
+                                                         batch.max_seq_len, self._dt(z, "z"), self._stream()), "linear_attention")
+        return out
+
     def selective_scan(self, x, dt, bc, b_col, c_col, z, z_col, A_log, dt_bias, skip, state, batch):
         """The selective scan with a state per channel and state index over the rows of each request, from ``state [slots, channels,
         state_size]``: ``x [N, channels]`` (after convolution and activation), ``dt [N, channels]`` the step sizes' logits (``dt_bias`` is
@@ -1626,16 +1813,20 @@ class CudaKernels:
         return out
 
     # ------------------------------------------------------------------ routed experts
-    _SCORING = {"softmax": 0, "sigmoid": 1}
+    _SCORING = {"softmax": 0, "sigmoid": 1, "top_softmax": 2}
 
-    def moe_route(self, logits, correction, top: int, scoring: str = "softmax"):
+    def moe_route(self, logits, correction, top: int, scoring: str = "softmax", bias=None, gates: int = 0):
         """From float32 router logits ``[N, outputs]``: ``s = softmax(logits)``; the ``top`` outputs with the largest ``s + correction``
         (``correction`` may be None); returns ``(ids [N, top] int32, weights [N, top] float32)`` with the weights ``s / (sum of the chosen s + 1e-20)``.
-        ``scoring="sigmoid"``: ``s = sigmoid(logits)`` and the weights are the chosen ``s`` as they are."""
+        ``scoring="sigmoid"``: ``s = sigmoid(logits)`` and the weights are the chosen ``s`` as they are. ``scoring="top_softmax"``: the largest
+        logits are chosen, the weights are the softmax over those alone. ``bias`` (float32) is added to the logits first. ``gates``: the last
+        so many columns of ``logits`` are no outputs of the router but gates, and ``sigmoid`` of them is returned as a third tensor
+        (``bias`` or ``gates`` given: three results, the third maybe empty)."""
         self._need(logits, "logits", torch.float32, 2)
         if scoring not in self._SCORING:
             raise KernelError(f"moe_route: scoring '{scoring}' is not built")
-        N, total = logits.shape
+        N, total = logits.shape[0], logits.shape[1] - gates
+        self._check_router(bias, total)
         if correction is not None:
             self._need(correction, "correction", torch.float32, 1)
             if correction.shape[0] != total:
@@ -1644,22 +1835,32 @@ class CudaKernels:
             raise KernelError(f"moe_route: {top} of {total} router outputs cannot be chosen (at most 512 outputs)")
         ids = torch.empty((N, top), dtype=torch.int32, device=logits.device)
         weights = torch.empty((N, top), dtype=torch.float32, device=logits.device)
-        self._check(self.lib.llmie_moe_route(_ptr(logits), _ptr(correction), _ptr(ids), _ptr(weights), N, total, top, self._SCORING[scoring], self._stream()), "moe_route")
-        return ids, weights
+        out_gates = torch.empty((N, gates), dtype=torch.float32, device=logits.device)
+        self._check(self.lib.llmie_moe_route(_ptr(logits), _ptr(correction), _ptr(ids), _ptr(weights), N, total, top, self._SCORING[scoring], _ptr(bias),
+                                             int(gates), _ptr(out_gates if gates else None), self._stream()), "moe_route")
+        return (ids, weights, out_gates) if bias is not None or gates else (ids, weights)
 
-    def moe_router(self, h, w_router, correction, top: int, scoring: str = "softmax"):
+    def _check_router(self, bias, total: int) -> None:
+        if bias is not None:
+            self._need(bias, "bias", torch.float32, 1)
+            if bias.shape[0] != total:
+                raise KernelError("moe_route: the bias needs one entry per router output")
+
+    def moe_router(self, h, w_router, correction, top: int, scoring: str = "softmax", bias=None, gates: int = 0):
         """A router from the rows themselves: ``moe_route`` of the 32-bit logits ``h w_router^T`` (``h`` as it is stored). The few rows of
         a decode step, and float32 always, take one kernel that makes a token's logits and its choice (the sum over the inputs runs in one
-        order whatever the step holds); prompt portions in bfloat16 take the tensor-core product with 32-bit output and the choice kernel."""
+        order whatever the step holds); prompt portions in bfloat16 take the tensor-core product with 32-bit output and the choice kernel.
+        ``bias`` and ``gates`` as in ``moe_route`` (the gates' rows are the last ones of ``w_router``)."""
         self._need(h, "h", None, 2)
         self._need(w_router, "w_router", h.dtype, 2)
         if scoring not in self._SCORING:
             raise KernelError(f"moe_router: scoring '{scoring}' is not built")
         N, K = h.shape
-        total = w_router.shape[0]
-        fused = self.use_fused_router and (h.dtype == torch.float32 or N <= self.tc_max_rows) and (K + total + 4) * 4 <= 200 * 1024
+        total = w_router.shape[0] - gates
+        fused = self.use_fused_router and (h.dtype == torch.float32 or N <= self.tc_max_rows) and (K + total + gates + 4) * 4 <= 200 * 1024
         if not fused:
-            return self.moe_route(self.linear(h, w_router, out_dtype=torch.float32), correction, top, scoring)
+            return self.moe_route(self.linear(h, w_router, out_dtype=torch.float32), correction, top, scoring, bias, gates)
+        self._check_router(bias, total)
         if w_router.shape[1] != K:
             raise KernelError(f"moe_router: h has {K} columns, the router {w_router.shape[1]}")
         if correction is not None:
@@ -1670,9 +1871,10 @@ class CudaKernels:
             raise KernelError(f"moe_router: {top} of {total} router outputs cannot be chosen (at most 512 outputs)")
         ids = torch.empty((N, top), dtype=torch.int32, device=h.device)
         weights = torch.empty((N, top), dtype=torch.float32, device=h.device)
+        out_gates = torch.empty((N, gates), dtype=torch.float32, device=h.device)
         self._check(self.lib.llmie_moe_router(_ptr(h), _ptr(w_router), _ptr(correction), _ptr(ids), _ptr(weights), N, K, total, top, self._SCORING[scoring],
-                                              self._dt(h, "h"), self._stream()), "moe_router")
-        return ids, weights
+                                              _ptr(bias), int(gates), _ptr(out_gates if gates else None), self._dt(h, "h"), self._stream()), "moe_router")
+        return (ids, weights, out_gates) if bias is not None or gates else (ids, weights)
 
     def moe_experts(self, h, ids, weights, w_gate_up, w_down, add_to, glu=None, weight_inputs=False):
         """``add_to[t] += sum_k weights[t, k] * expert_(ids[t, k])(h[t])``: expert ``e < E`` is ``down_e(silu(gate_e x) * (up_e x))`` with

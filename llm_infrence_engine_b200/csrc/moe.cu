@@ -23,14 +23,18 @@ constexpr int SORT_MAX_EXPERTS = 4096;
 // chosen (of equal scores the lower index first); their weights are s / (sum of the chosen s + 1e-20).
 // (one warp: token n's row of logits, in global or shared memory)
 // `scoring` 1 instead: s = sigmoid(logits), every output by itself, and the weights are the chosen s as they are (not renormalised).
+// `scoring` 2: the `top` largest logits are chosen, and their weights are the softmax over the chosen ones alone.
+// `bias` [total] or null is added to the logits first.
 __device__ __forceinline__ void route_token(const float* __restrict__ row, const float* __restrict__ correction, int* __restrict__ ids,
-                                            float* __restrict__ weights, int n, int total, int top, int lane, int scoring) {
+                                            float* __restrict__ weights, int n, int total, int top, int lane, int scoring,
+                                            const float* __restrict__ bias) {
     float s[ROUTE_MAX_PER_LANE], c[ROUTE_MAX_PER_LANE];
     float mx = -INFINITY;
 #pragma unroll
     for (int j = 0; j < ROUTE_MAX_PER_LANE; ++j) {
         const int e = lane + 32 * j;
-        s[j] = e < total ? row[e] : -INFINITY;
+        s[j] = e < total ? row[e] + (bias ? bias[e] : 0.f) : -INFINITY;
+        c[j] = s[j];
         mx = fmaxf(mx, s[j]);
     }
     mx = warp_max(mx);
@@ -42,12 +46,12 @@ __device__ __forceinline__ void route_token(const float* __restrict__ row, const
         else s[j] = e < total ? expf(s[j] - mx) : 0.f;
         sum += s[j];
     }
-    sum = scoring == 1 ? 1.f : warp_sum(sum);
+    sum = scoring != 0 ? 1.f : warp_sum(sum);
 #pragma unroll
     for (int j = 0; j < ROUTE_MAX_PER_LANE; ++j) {
         const int e = lane + 32 * j;
         s[j] = s[j] / sum;
-        c[j] = e < total ? s[j] + (correction ? correction[e] : 0.f) : -INFINITY;
+        if (scoring != 2) c[j] = e < total ? s[j] + (correction ? correction[e] : 0.f) : -INFINITY;
     }
     float chosen_sum = 0.f;
     float my_w = 0.f;      // lane k keeps the k-th choice
@@ -80,17 +84,22 @@ __device__ __forceinline__ void route_token(const float* __restrict__ row, const
         }
     }
     __syncwarp();
-    const float inv = scoring == 1 ? 1.0f : 1.0f / (chosen_sum + 1e-20f);
+    const float inv = scoring == 1 ? 1.0f : 1.0f / (chosen_sum + (scoring == 0 ? 1e-20f : 0.f));   // (2: the largest logit's share is 1)
     for (int k = lane; k < top; k += 32) weights[(size_t)n * top + k] *= inv;
 }
 
+// Rows of `total + extra` logits; the extra ones are gates of their own: gates[n][j] = sigmoid(logit).
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ correction,
-                                                        int* __restrict__ ids, float* __restrict__ weights, int N, int total, int top, int scoring) {
+                                                        int* __restrict__ ids, float* __restrict__ weights, int N, int total, int top, int scoring,
+                                                        const float* __restrict__ bias, int extra, float* __restrict__ gates) {
     pdl_trigger();
     pdl_wait();
     const int n = blockIdx.x * 4 + (threadIdx.x >> 5);
     if (n >= N) return;
-    route_token(logits + (size_t)n * total, correction, ids, weights, n, total, top, threadIdx.x & 31, scoring);
+    const float* row = logits + (size_t)n * (total + extra);
+    const int lane = threadIdx.x & 31;
+    for (int j = lane; j < extra; j += 32) gates[(size_t)n * extra + j] = 1.0f / (1.0f + expf(-row[total + j]));
+    route_token(row, correction, ids, weights, n, total, top, lane, scoring, bias);
 }
 
 // The router's product and its choice in one kernel, a block per token: the token's row lies in shared memory as floats, the warps
@@ -100,8 +109,9 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
 constexpr int ROUTER_THREADS = 256;
 template <typename T>
 __global__ void __launch_bounds__(ROUTER_THREADS) moe_router_kernel(const T* __restrict__ h, const T* __restrict__ w, const float* __restrict__ correction,
-                                                                    int* __restrict__ ids, float* __restrict__ weights, int K, int total, int top, int scoring) {
-    extern __shared__ __align__(16) float router_smem[];   // [K] the row, then [total] the logits
+                                                                    int* __restrict__ ids, float* __restrict__ weights, int K, int total, int top, int scoring,
+                                                                    const float* __restrict__ bias, int extra, float* __restrict__ gates) {
+    extern __shared__ __align__(16) float router_smem[];   // [K] the row, then [total + extra] the logits
     constexpr int VN = Vec16<T>::N;
     float* row = router_smem;
     float* logits = router_smem + ((K + 3) & ~3);
@@ -121,7 +131,7 @@ __global__ void __launch_bounds__(ROUTER_THREADS) moe_router_kernel(const T* __r
         for (int k = threadIdx.x; k < K; k += ROUTER_THREADS) row[k] = to_f32(src[k]);
     }
     __syncthreads();
-    for (int e = warp; e < total; e += ROUTER_THREADS / 32) {
+    for (int e = warp; e < total + extra; e += ROUTER_THREADS / 32) {
         const T* we = w + (size_t)e * K;
         float acc = 0.f;
         if (vec) {
@@ -138,7 +148,9 @@ __global__ void __launch_bounds__(ROUTER_THREADS) moe_router_kernel(const T* __r
         if (lane == 0) logits[e] = acc;
     }
     __syncthreads();
-    if (warp == 0) route_token(logits, correction, ids, weights, n, total, top, lane, scoring);
+    if (warp == 1)
+        for (int j = lane; j < extra; j += 32) gates[(size_t)n * extra + j] = 1.0f / (1.0f + expf(-logits[total + j]));
+    if (warp == 0) route_token(logits, correction, ids, weights, n, total, top, lane, scoring, bias);
 }
 
 // One block: the step's (token, choice) pairs counted per expert, the experts' runs laid out one behind the other, every pair
@@ -379,20 +391,22 @@ __global__ void __launch_bounds__(256) moe_combine_kernel(float* __restrict__ re
 
 }  // namespace
 
+// logits [N, total + extra]; bias [total] or null; gates [N, extra] (extra 0: none).
 LLMIE_API int llmie_moe_route(const float* logits, const float* correction, int* ids, float* weights, int N, int total, int top, int scoring,
-                              cudaStream_t s) {
+                              const float* bias, int extra, float* gates, cudaStream_t s) {
     if (N <= 0) return 0;
-    if (total <= 0 || total > 32 * ROUTE_MAX_PER_LANE || top <= 0 || top > total) return LLMIE_ERR_BAD_ARGUMENT;
-    return launch_kernel(moe_route_kernel, dim3((N + 3) / 4), dim3(128), 0, s, logits, correction, ids, weights, N, total, top, scoring);
+    if (total <= 0 || total > 32 * ROUTE_MAX_PER_LANE || top <= 0 || top > total || extra < 0 || (extra && !gates)) return LLMIE_ERR_BAD_ARGUMENT;
+    return launch_kernel(moe_route_kernel, dim3((N + 3) / 4), dim3(128), 0, s, logits, correction, ids, weights, N, total, top, scoring, bias, extra,
+                         gates);
 }
 
-// ids, weights [N, top] from the rows h [N, K] and the router's matrix w [total, K] of the same type (float or bfloat16): the product in
+// ids, weights [N, top] from the rows h [N, K] and the router's matrix w [total + extra, K] of the same type (float or bfloat16): the product in
 // 32-bit and the choice, one launch. The row and the logits must fit the shared memory (K + total floats: up to about 50,000).
 LLMIE_API int llmie_moe_router(const void* h, const void* w, const float* correction, int* ids, float* weights, int N, int K, int total, int top,
-                               int scoring, int dtype, cudaStream_t s) {
+                               int scoring, const float* bias, int extra, float* gates, int dtype, cudaStream_t s) {
     if (N <= 0) return 0;
-    if (K <= 0 || total <= 0 || total > 32 * ROUTE_MAX_PER_LANE || top <= 0 || top > total) return LLMIE_ERR_BAD_ARGUMENT;
-    const size_t smem = ((size_t)((K + 3) & ~3) + total) * sizeof(float);
+    if (K <= 0 || total <= 0 || total > 32 * ROUTE_MAX_PER_LANE || top <= 0 || top > total || extra < 0 || (extra && !gates)) return LLMIE_ERR_BAD_ARGUMENT;
+    const size_t smem = ((size_t)((K + 3) & ~3) + total + extra) * sizeof(float);
     if (smem > 200 * 1024) return LLMIE_ERR_BAD_ARGUMENT;
     static size_t allowed_f = 48 * 1024, allowed_b = 48 * 1024;
     if (dtype == DT_F32) {
@@ -402,7 +416,7 @@ LLMIE_API int llmie_moe_router(const void* h, const void* w, const float* correc
             allowed_f = 200 * 1024;
         }
         return launch_kernel(moe_router_kernel<float>, dim3(N), dim3(ROUTER_THREADS), smem, s, (const float*)h, (const float*)w, correction, ids, weights, K,
-                             total, top, scoring);
+                             total, top, scoring, bias, extra, gates);
     }
     if (smem > allowed_b) {
         cudaError_t e = cudaFuncSetAttribute(moe_router_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
@@ -410,7 +424,7 @@ LLMIE_API int llmie_moe_router(const void* h, const void* w, const float* correc
         allowed_b = 200 * 1024;
     }
     return launch_kernel(moe_router_kernel<bf16>, dim3(N), dim3(ROUTER_THREADS), smem, s, (const bf16*)h, (const bf16*)w, correction, ids, weights, K, total,
-                         top, scoring);
+                         top, scoring, bias, extra, gates);
 }
 
 // Rows per tile of the grouped product on the CUDA cores for rows of K numbers: as many as fit the shared memory, at most MOE_TM;

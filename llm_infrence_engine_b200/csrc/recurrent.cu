@@ -350,7 +350,10 @@ __global__ void __launch_bounds__(SCAN_THREADS) delta_scan_kernel(const T* __res
 //   dt = softplus(dt_raw + dt_bias[h]);  S <- exp(-exp(A_log[h]) dt) S + dt B x^T;  y = S^T C + D[h] x
 // B and C belong to the head's group and come straight from the convolution's result (type T), so their tiles are filled with
 // plain loads a tile ahead; step size and decay are computed while a tile is loaded.
-template <typename T, int NMAX, int PARTS>
+// FIXED: linear attention with a fixed decay per head, S <- decay[h] S + k v^T; y = S^T q. q, k and v stand in the places of C, B
+// and x (a head of their own each: G = H), pass silu as they are loaded, and there are neither step sizes nor a skip; A_log holds
+// the decays themselves.
+template <typename T, int NMAX, int PARTS, bool FIXED>
 __global__ void __launch_bounds__(SCAN_THREADS) ssm_scan_kernel(const T* __restrict__ xbc, int x_stride, int x_col, int b_col, int c_col,
                                                                 const T* __restrict__ dt_raw, int dt_stride, const float* __restrict__ A_log,
                                                                 const float* __restrict__ dt_bias, const float* __restrict__ Dskip,
@@ -370,7 +373,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssm_scan_kernel(const T* __restr
     const int g = h / (H / G);
     const bool live = col < DV;
     const bool vec = (NS & 3) == 0;
-    const float rate = expf(A_log[h]), bias = dt_bias[h], skip = Dskip[h];
+    const float rate = FIXED ? A_log[h] : expf(A_log[h]), bias = FIXED ? 0.f : dt_bias[h], skip = FIXED ? 0.f : Dskip[h];
     pdl_wait();
     const int s0 = seq_starts[r], s1 = seq_starts[r + 1];
     float* st = state + (((size_t)seq_slots[r] * H + h) * DV + (live ? col : 0)) * NS;
@@ -392,7 +395,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssm_scan_kernel(const T* __restr
             pre_b[n] = in ? to_f32(xbc[row + b_col + g * NS + d]) : 0.f;
             pre_c[n] = in ? to_f32(xbc[row + c_col + g * NS + d]) : 0.f;
         }
-        if (threadIdx.x < count) pre_dt = to_f32(dt_raw[(size_t)(base + threadIdx.x) * dt_stride + h]);
+        if (!FIXED && threadIdx.x < count) pre_dt = to_f32(dt_raw[(size_t)(base + threadIdx.x) * dt_stride + h]);
 #pragma unroll
         for (int n = 0; n < XPT; ++n) {
             const int j = SCAN_THREADS - 1 - threadIdx.x + n * SCAN_THREADS;
@@ -405,11 +408,11 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssm_scan_kernel(const T* __restr
         for (int n = 0; n < BPT; ++n) {
             const int i = threadIdx.x + n * SCAN_THREADS;
             if (i < SCAN_TILE * NMAX) {
-                b_s[buf * SCAN_TILE * NMAX + i] = pre_b[n];
-                c_s[buf * SCAN_TILE * NMAX + i] = pre_c[n];
+                b_s[buf * SCAN_TILE * NMAX + i] = FIXED ? silu_f(pre_b[n]) : pre_b[n];   // (silu(0) = 0: the padding stays)
+                c_s[buf * SCAN_TILE * NMAX + i] = FIXED ? silu_f(pre_c[n]) : pre_c[n];
             }
         }
-        if (threadIdx.x < SCAN_TILE) {
+        if (!FIXED && threadIdx.x < SCAN_TILE) {
             const float dt = softplus_f(pre_dt + bias);
             dt_s[buf * SCAN_TILE + threadIdx.x] = dt;
             a_s[buf * SCAN_TILE + threadIdx.x] = expf(-rate * dt);
@@ -417,7 +420,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssm_scan_kernel(const T* __restr
 #pragma unroll
         for (int n = 0; n < XPT; ++n) {
             const int j = SCAN_THREADS - 1 - threadIdx.x + n * SCAN_THREADS;
-            if (j < SCAN_TILE * COLS) x_s[buf * SCAN_TILE * COLS + j] = pre_x[n];
+            if (j < SCAN_TILE * COLS) x_s[buf * SCAN_TILE * COLS + j] = FIXED ? silu_f(pre_x[n]) : pre_x[n];
         }
     };
     const int my_col = threadIdx.x / PARTS;
@@ -437,7 +440,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssm_scan_kernel(const T* __restr
         for (int t = 0; t < SCAN_TILE; ++t) {
             if (t < count) {
                 const float xv = x_s[(buf * SCAN_TILE + t) * COLS + my_col];
-                const float a = a_s[buf * SCAN_TILE + t], u = dt_s[buf * SCAN_TILE + t] * xv;
+                const float a = FIXED ? rate : a_s[buf * SCAN_TILE + t], u = FIXED ? xv : dt_s[buf * SCAN_TILE + t] * xv;
                 float y0 = 0.f, y1 = 0.f;
 #pragma unroll
                 for (int i = 0; i < DPL / 4; ++i) {
@@ -448,7 +451,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) ssm_scan_kernel(const T* __restr
                     y0 = fmaf(s[0], c4.x, y0); y1 = fmaf(s[1], c4.y, y1); y0 = fmaf(s[2], c4.z, y0); y1 = fmaf(s[3], c4.w, y1);
                 }
                 const float y = parts_sum<PARTS>(y0 + y1);
-                if (live && part == 0) out[(size_t)(base + t) * H * DV + h * DV + col] = fmaf(skip, xv, y);
+                if (live && part == 0) out[(size_t)(base + t) * H * DV + h * DV + col] = FIXED ? y : fmaf(skip, xv, y);
             }
         }
         if (more) store_tile(buf ^ 1);         // (the other stage: nobody reads it before the next barrier)
@@ -609,16 +612,27 @@ int launch_delta_scan_as(const T* v, int v_stride, int v_col, const float* qn, c
     return launch_delta_scan_one<T, DM, PARTS, false>(v, v_stride, v_col, qn, kn, kq, decay, beta, state, seq_starts, seq_slots, out, H, G, D, DV, R, alone, s);
 }
 
-template <typename T, int NM, int PARTS>
-int launch_ssm_scan_as(const T* xbc, int x_stride, int x_col, int b_col, int c_col, const T* dt_raw, int dt_stride, const float* A_log,
+template <typename T, int NM, int PARTS, bool FIXED>
+int launch_ssm_scan_one(const T* xbc, int x_stride, int x_col, int b_col, int c_col, const T* dt_raw, int dt_stride, const float* A_log,
                        const float* dt_bias, const float* Dskip, float* state, const int* seq_starts, const int* seq_slots, float* out, int H,
                        int G, int NS, int DV, int R, bool alone, cudaStream_t s) {
     constexpr int cols = SCAN_THREADS / PARTS;
     const dim3 grid((DV + cols - 1) / cols, H, R);
     const size_t smem = sizeof(float) * (2 * SCAN_TILE * (2 * NM + 2 + cols));
-    if (smem > 48 * 1024) cudaFuncSetAttribute(ssm_scan_kernel<T, NM, PARTS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    return launch_kernel_on(alone, ssm_scan_kernel<T, NM, PARTS>, grid, dim3(SCAN_THREADS), smem, s, xbc, x_stride, x_col, b_col, c_col, dt_raw,
+    if (smem > 48 * 1024) cudaFuncSetAttribute(ssm_scan_kernel<T, NM, PARTS, FIXED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    return launch_kernel_on(alone, ssm_scan_kernel<T, NM, PARTS, FIXED>, grid, dim3(SCAN_THREADS), smem, s, xbc, x_stride, x_col, b_col, c_col, dt_raw,
                             dt_stride, A_log, dt_bias, Dskip, state, seq_starts, seq_slots, out, H, G, NS, DV);
+}
+
+template <typename T, int NM, int PARTS>
+int launch_ssm_scan_as(const T* xbc, int x_stride, int x_col, int b_col, int c_col, const T* dt_raw, int dt_stride, const float* A_log,
+                       const float* dt_bias, const float* Dskip, float* state, const int* seq_starts, const int* seq_slots, float* out, int H,
+                       int G, int NS, int DV, int R, bool alone, cudaStream_t s) {
+    if (!dt_raw)   // no step sizes: the fixed decays of linear attention
+        return launch_ssm_scan_one<T, NM, PARTS, true>(xbc, x_stride, x_col, b_col, c_col, dt_raw, dt_stride, A_log, dt_bias, Dskip, state, seq_starts,
+                                                       seq_slots, out, H, G, NS, DV, R, alone, s);
+    return launch_ssm_scan_one<T, NM, PARTS, false>(xbc, x_stride, x_col, b_col, c_col, dt_raw, dt_stride, A_log, dt_bias, Dskip, state, seq_starts,
+                                                    seq_slots, out, H, G, NS, DV, R, alone, s);
 }
 
 // the padded size (16, 32, 64, 128 or 256) and the lanes per column (scan_parts) pick the instantiation
@@ -714,13 +728,28 @@ LLMIE_API int llmie_ssm_scan(const void* xbc, int x_stride, int x_col, int b_col
                              const float* A_log, const float* dt_bias, const float* Dskip, float* state, const int* seq_starts,
                              const int* seq_slots, float* out, int H, int G, int NS, int DV, int R, int max_rows, int dtype, cudaStream_t s) {
     if (R <= 0) return 0;
-    if (H <= 0 || G <= 0 || H % G || NS <= 0 || NS > 256 || DV <= 0 || H > 65535 || R > 65535) return LLMIE_ERR_BAD_ARGUMENT;
+    if (H <= 0 || G <= 0 || H % G || NS <= 0 || NS > 256 || DV <= 0 || H > 65535 || R > 65535 || !dt_raw) return LLMIE_ERR_BAD_ARGUMENT;
     const bool alone = max_rows >= SCAN_ALONE_ROWS;
     if (dtype == DT_F32)
         return launch_ssm_scan<float>((const float*)xbc, x_stride, x_col, b_col, c_col, (const float*)dt_raw, dt_stride, A_log, dt_bias, Dskip,
                                       state, seq_starts, seq_slots, out, H, G, NS, DV, R, alone, s);
     return launch_ssm_scan<bf16>((const bf16*)xbc, x_stride, x_col, b_col, c_col, (const bf16*)dt_raw, dt_stride, A_log, dt_bias, Dskip, state,
                                  seq_starts, seq_slots, out, H, G, NS, DV, R, alone, s);
+}
+
+// Linear attention with a fixed decay per head: z holds q and k (H heads of D columns from q_col, k_col) and v (H heads of DV from
+// v_col), before silu; decay [H]; state [slots][H][DV][D] float (column by column); out [N][H * DV] float
+LLMIE_API int llmie_linear_attention_scan(const void* z, int z_stride, int q_col, int k_col, int v_col, const float* decay, float* state,
+                                          const int* seq_starts, const int* seq_slots, float* out, int H, int D, int DV, int R, int max_rows, int dtype,
+                                          cudaStream_t s) {
+    if (R <= 0) return 0;
+    if (H <= 0 || D <= 0 || D > 256 || DV <= 0 || H > 65535 || R > 65535) return LLMIE_ERR_BAD_ARGUMENT;
+    const bool alone = max_rows >= SCAN_ALONE_ROWS;
+    if (dtype == DT_F32)
+        return launch_ssm_scan<float>((const float*)z, z_stride, v_col, k_col, q_col, nullptr, 0, decay, nullptr, nullptr, state, seq_starts, seq_slots, out,
+                                      H, H, D, DV, R, alone, s);
+    return launch_ssm_scan<bf16>((const bf16*)z, z_stride, v_col, k_col, q_col, nullptr, 0, decay, nullptr, nullptr, state, seq_starts, seq_slots, out, H, H,
+                                 D, DV, R, alone, s);
 }
 
 // x, dt_raw, z: [N] rows of C channels (the caller offsets the pointers to their first column); bc: rows that hold B from column

@@ -40,6 +40,9 @@ def build_runner(folder: Union[str, Path], config: EngineConfig, kernels=None):
     spec = build_model_spec(read_config_json(folder))
     dtype = _TORCH_DTYPE[config.dtype]
     load_weights(spec, folder, dtype, config.device)
+    limit = spec.embedding.position_limit()
+    if limit is not None and config.max_len > limit:   # (a table of positions: no request can become longer)
+        config.max_len = limit
     specs = spec.cache_specs()
     groups, of_entry = group_layout(specs)
     num_pages = config.pool_blocks()

@@ -43,6 +43,7 @@ class PagedKVBinding:
     k: torch.Tensor  # [num_pages, num_kv_heads, page_size, head_dim]
     v: Optional[torch.Tensor]  # [num_pages, num_kv_heads, page_size, v_head_dim]; None where values are read out of the key rows
     write: bool = True
+    scalar: Optional[torch.Tensor] = None  # [num_pages, page_size] float32, where the mixer keeps a number per token
 
 
 @dataclass
@@ -119,7 +120,9 @@ class ModelRunner:
                 k = torch.zeros((num_pages, cs.num_kv_heads, page_size, cs.head_dim), dtype=dtype, device=self.device)
                 v = torch.zeros((num_pages, cs.num_kv_heads, page_size, v_dim), dtype=dtype, device=self.device) if v_dim else None
                 self.kv_bytes_per_token += cs.num_kv_heads * (cs.head_dim + v_dim) * k.element_size()
-                return PagedKVBinding(group, k, v)
+                scalar = torch.zeros((num_pages, page_size), dtype=torch.float32, device=self.device) if cs.token_scalar else None
+                self.kv_bytes_per_token += 4 if cs.token_scalar else 0
+                return PagedKVBinding(group, k, v, scalar=scalar)
             if isinstance(cs, FixedStateSpec):
                 b = StateBinding(torch.zeros((max_seqs + 1,) + tuple(cs.shape), dtype=torch.float32, device=self.device))
                 self.all_states.append(b)

@@ -6,7 +6,8 @@ from typing import Dict, Optional
 import torch
 
 from ..cache.spec import FixedStateSpec, PagedKVSpec
-from .base import INIT_EYE, INIT_NORM, INIT_PROJ, INIT_RATE, INIT_SMALL, INIT_TAPS, MATRIX, VECTOR, Mixer, ParamSpec, PositionEncoding, Source
+from .attention_biased import distance_rows
+from .base import ANY, INIT_EYE, INIT_NORM, INIT_PROJ, INIT_RATE, INIT_SMALL, INIT_TAPS, MATRIX, VECTOR, Mixer, ParamSpec, PositionEncoding, Source
 
 
 class MaskedAttention(Mixer):
@@ -17,6 +18,12 @@ class MaskedAttention(Mixer):
     * ``conv_taps``: a short causal convolution per channel on q, k and v right after their projection (no bias, no
       activation); a request's last ``conv_taps - 1`` projected rows are part of its state;
     * ``qk_norm``: RMS norm of every query and key head with a weight of ``head_dim`` entries shared by the heads, before rotation;
+      ``qk_norm="rows"``: of the whole query projection and of the whole key projection at once, with a weight per row of them;
+    * ``values_are_keys`` (with ``qk_norm="rows"``, without rotation): there is no value projection, the values are the keys as they
+      are before the norm. The cache holds that row ONCE, with one number per token beside it, its reciprocal root mean square:
+      the norm's weight is moved to the queries, ``q . (w k rms^-1) = rms^-1 (w q) . k``, and the number multiplies the score;
+    * ``bias_far``: a bias ``rel[row(i - j), head]`` (``{prefix}.rel``) is added to the (capped) score, its row chosen by the distance
+      (``distance_rows``), the last row from ``bias_far`` on; the number of rows is the checkpoint's;
     * ``position``: a rotary encoding with ``dims`` and ``tables`` (cos, sin of ``[N, dims / 2]``); the first ``dims`` entries of a
       head turn, the rest pass; pairs are ``(i, i + dims/2)``, or neighbours ``(2i, 2i+1)`` when ``interleaved``;
     * ``window`` with ``keep_first``: position i sees ``j <= i`` with ``i - j < window`` or ``j < keep_first``;
@@ -42,9 +49,10 @@ class MaskedAttention(Mixer):
 
     def __init__(self, hidden: int, num_heads: int, num_kv_heads: int, head_dim: int, v_head_dim: int, scale: float, prefix: str,
                  position: Optional[PositionEncoding] = None, interleaved: bool = False, window: Optional[int] = None, keep_first: int = 0,
-                 chunk: Optional[int] = None, softcap: Optional[float] = None, conv_taps: int = 0, qk_norm: bool = False, eps: float = 1e-6,
+                 chunk: Optional[int] = None, softcap: Optional[float] = None, conv_taps: int = 0, qk_norm=False, eps: float = 1e-6,
                  talking_heads: bool = False, sink: bool = False, head_gate: bool = False, bias: bool = False,
-                 value_position: Optional[PositionEncoding] = None, log_distance: bool = False, scoring: str = "softmax"):
+                 value_position: Optional[PositionEncoding] = None, log_distance: bool = False, scoring: str = "softmax",
+                 values_are_keys: bool = False, bias_far: Optional[float] = None, random_rel_rows: int = 16):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads cannot share {num_kv_heads} key/value heads")
         if keep_first and not window:
@@ -59,7 +67,18 @@ class MaskedAttention(Mixer):
         self.window, self.keep_first, self.chunk = window, int(keep_first), chunk
         self.softcap = float(softcap) if softcap else 0.0
         self.conv_taps, self.qk_norm, self.eps = int(conv_taps), bool(qk_norm), float(eps)
-        self.channels = (num_heads + num_kv_heads) * head_dim + num_kv_heads * v_head_dim
+        self.norm_rows = qk_norm == "rows"
+        if self.norm_rows and (conv_taps or position is not None or value_position is not None):
+            raise ValueError("queries and keys normed as whole projections are not built together with convolutions or rotation")
+        self.values_are_keys = bool(values_are_keys)
+        if values_are_keys and (not self.norm_rows or v_head_dim != head_dim):
+            raise ValueError("values that are the keys need keys normed as a whole projection, and heads of one size")
+        if bias_far is not None and (scoring == "sigmoid" or talking_heads):
+            raise ValueError("a bias by distance is not built together with sigmoid weights or talking heads")
+        self.bias_far, self.random_rel_rows = bias_far, int(random_rel_rows)
+        self.rel: Optional[torch.Tensor] = None
+        self.rel_rows: Optional[torch.Tensor] = None   # int32 [ceil(bias_far)]: distance -> row of ``rel``
+        self.channels = (num_heads + num_kv_heads) * head_dim + (0 if values_are_keys else num_kv_heads * v_head_dim)
         self.talking_heads, self.has_sink, self.head_gate = bool(talking_heads), bool(sink), bool(head_gate)
         if scoring not in ("softmax", "sigmoid"):
             raise ValueError(f"scoring '{scoring}' is not 'softmax' or 'sigmoid'")
@@ -84,7 +103,8 @@ class MaskedAttention(Mixer):
         self.k_norm: Optional[torch.Tensor] = None
 
     def _rows(self):
-        return (("q", self.num_heads * self.head_dim), ("k", self.num_kv_heads * self.head_dim), ("v", self.num_kv_heads * self.v_head_dim))
+        rows = (("q", self.num_heads * self.head_dim), ("k", self.num_kv_heads * self.head_dim))
+        return rows if self.values_are_keys else rows + (("v", self.num_kv_heads * self.v_head_dim),)
 
     def params(self) -> Dict[str, ParamSpec]:
         p, h = self.prefix, self.hidden
@@ -94,8 +114,6 @@ class MaskedAttention(Mixer):
         out = {"w_qkv": ParamSpec(joined, MATRIX),
                "w_o": ParamSpec((Source(f"{p}.o", (h, self.num_heads * self.v_head_dim), INIT_PROJ),), MATRIX)}
         if self.has_bias:   # (biases are kept in the type of the products they are added to)
-            if self.head_gate:
-                raise ValueError("biases are not built together with a gate per head")
             out["b_qkv"] = ParamSpec(tuple(Source(f"{p}.{n}.b", (r,), INIT_SMALL) for n, r in self._rows()), MATRIX)
             out["b_o"] = ParamSpec((Source(f"{p}.o.b", (h,), INIT_SMALL),), MATRIX)
         if self.log_distance:
@@ -110,8 +128,11 @@ class MaskedAttention(Mixer):
         if self.conv_taps:
             out["conv_w"] = ParamSpec(tuple(Source(f"{p}.{n}.conv", (r, self.conv_taps), INIT_TAPS) for n, r in self._rows()), VECTOR)
         if self.qk_norm:
-            out["q_norm"] = ParamSpec((Source(f"{p}.q.norm", (self.head_dim,), INIT_NORM),), VECTOR)
-            out["k_norm"] = ParamSpec((Source(f"{p}.k.norm", (self.head_dim,), INIT_NORM),), VECTOR)
+            heads_q, heads_k = (self.num_heads, self.num_kv_heads) if self.norm_rows else (1, 1)
+            out["q_norm"] = ParamSpec((Source(f"{p}.q.norm", (heads_q * self.head_dim,), INIT_NORM),), VECTOR)
+            out["k_norm"] = ParamSpec((Source(f"{p}.k.norm", (heads_k * self.head_dim,), INIT_NORM),), VECTOR)
+        if self.bias_far is not None:
+            out["rel"] = ParamSpec((Source(f"{p}.rel", (ANY, self.num_heads), INIT_SMALL, free=self.random_rel_rows),), VECTOR)
         return out
 
     def bind(self, tensors) -> None:
@@ -119,17 +140,23 @@ class MaskedAttention(Mixer):
         pad = -self.w_qkv.shape[0] % 8   # (rows of the product that start on a 16-byte boundary)
         if pad:
             self.w_qkv = torch.cat([self.w_qkv, self.w_qkv.new_zeros((pad, self.w_qkv.shape[1]))]).contiguous()
-            if self.b_qkv is not None:
-                self.b_qkv = torch.cat([self.b_qkv, self.b_qkv.new_zeros(pad)]).contiguous()
+        if self.b_qkv is not None and self.b_qkv.shape[0] < self.w_qkv.shape[0]:   # (the rows of a gate, and the padding, have no bias)
+            self.b_qkv = torch.cat([self.b_qkv, self.b_qkv.new_zeros(self.w_qkv.shape[0] - self.b_qkv.shape[0])]).contiguous()
+        if self.rel is not None:
+            self.rel = self.rel.contiguous()
+            self.rel_rows = torch.tensor(distance_rows(self.rel.shape[0], self.bias_far), dtype=torch.int32, device=self.rel.device)
 
     def cache_spec(self):
-        pages = PagedKVSpec(self.num_kv_heads, self.head_dim, self.window, self.v_head_dim, self.keep_first, self.chunk)
+        pages = PagedKVSpec(self.num_kv_heads, self.head_dim, self.window, 0 if self.values_are_keys else self.v_head_dim, self.keep_first, self.chunk,
+                            token_scalar=self.values_are_keys)
         if self.conv_taps:
             return (pages, FixedStateSpec((self.conv_taps - 1, self.channels)))
         return pages
 
     def forward(self, ctx, h, cache, residual):
         K = ctx.K
+        if self.norm_rows:
+            return self._forward_rows(ctx, h, cache, residual)
         kv, conv_state = cache if self.conv_taps else (cache, None)
         # where nothing else reads the projections, a small batch leaves its float32 sums to the kernel that turns and stores them
         more = {"transient": True} if not (self.head_gate or self.conv_taps) else {}
@@ -151,6 +178,8 @@ class MaskedAttention(Mixer):
         more = {}
         if v_turn is not None:
             more["turn"] = (*v_turn, self.interleaved)
+        if self.rel is not None:
+            more["rel"], more["rel_rows"] = self.rel, self.rel_rows
         if self.log_distance:
             more["log_distance"] = (self.r1, self.r2)
         if self.scoring == "sigmoid":
@@ -163,3 +192,23 @@ class MaskedAttention(Mixer):
             K.linear(attn, self.w_o, add_to=residual, bias=self.b_o)
         else:
             K.linear(attn, self.w_o, add_to=residual)
+
+    def _forward_rows(self, ctx, h, kv, residual):
+        """Queries and keys normed as whole projections: one kernel norms both rows of a token, stores its keys (and values) and
+        hands the gate's columns on behind the queries, so the projections' sums have no other reader."""
+        K = ctx.K
+        z = K.linear(h, self.w_qkv, out_dtype=ctx.dtype, transient=True, **({"bias": self.b_qkv} if self.has_bias else {}))
+        q = K.qk_rows_norm_store(z, self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim, self.q_norm, self.k_norm, self.eps,
+                                 ctx.slot_mapping[kv.group], kv.k, kv.v, kv.scalar, ctx.page_size, gate_cols=self.num_heads if self.head_gate else 0,
+                                 write_kv=kv.write, out_dtype=ctx.dtype)
+        more = {}
+        if self.log_distance:
+            more["log_distance"] = (self.r1, self.r2)
+        if self.scoring == "sigmoid":
+            more["sigmoid_bias"] = self.pb
+        attn = K.attention_ext(q, 0, self.num_heads, self.num_kv_heads, self.head_dim, self.v_head_dim, kv.k, kv.v, ctx.block_tables[kv.group],
+                               ctx.token_seq, ctx.positions, ctx.page_size, self.scale, self.window or 0, ctx.max_context, batch=ctx,
+                               keep_first=self.keep_first, chunk=self.chunk or 0, softcap=self.softcap, sink=self.sink,
+                               gate=q if self.head_gate else None, gate_col=self.num_heads * self.head_dim, gate_per_head=True, talk=self.talk,
+                               rel=self.rel, rel_rows=self.rel_rows, key_scale=kv.scalar, **more)
+        K.linear(attn, self.w_o, add_to=residual, **({"bias": self.b_o} if self.has_bias else {}))

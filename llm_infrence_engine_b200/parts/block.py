@@ -103,6 +103,40 @@ class SandwichBlock(Part):
             self.norm2b.add_normed(ctx, residual, y)
 
 
+class PostNormBlock(Part):
+    """``x += norm1(mixer(x)); x += norm2(ff(x))``: the sublayers read the stream itself (rounded to the compute dtype, nothing else),
+    and a norm stands on their results alone; a layer may be a mixer alone.
+
+    A sublayer adds its result into a zeroed tensor as in ``SandwichBlock``; the norms have ``add_normed(ctx, residual, y)``, whose
+    addition is put off until the stream is read next, by a kernel that adds and rounds in one pass.
+    """
+
+    graph_safe = True
+
+    def __init__(self, mixer: Mixer, norm1: Norm, ff: Optional[FeedForward] = None, norm2: Optional[Norm] = None):
+        if (norm2 is None) != (ff is None):
+            raise ValueError("a feed-forward comes with its norm, or neither is there")
+        self.mixer, self.norm1, self.ff, self.norm2 = mixer, norm1, ff, norm2
+
+    def children(self) -> Sequence[Part]:
+        return tuple(p for p in (self.mixer, self.norm1, self.ff, self.norm2) if p is not None)
+
+    def cache_spec(self):
+        return self.mixer.cache_spec()
+
+    def forward(self, ctx, residual: torch.Tensor, cache) -> None:
+        K = ctx.K
+        h = K.stream_rows(residual, ctx.dtype)
+        y = K.zeros_like_rows(residual)
+        self.mixer.forward(ctx, h, cache, y)
+        self.norm1.add_normed(ctx, residual, y)
+        if self.ff is not None:
+            h = K.stream_rows(residual, ctx.dtype)
+            y = K.zeros_like_rows(residual)
+            self.ff.forward(ctx, h, y)
+            self.norm2.add_normed(ctx, residual, y)
+
+
 class ParallelBlock(Part):
     """``h = norm(x); x += mixer(h) + ff(h)``: one norm, and both sublayers read its output. Each sublayer adds its result into
     the 32-bit stream itself, so the sum of the two is never a tensor of its own; a layer may be a mixer alone."""

@@ -6,7 +6,7 @@ from typing import Dict, Optional
 import torch
 
 from ..cache.spec import FixedStateSpec
-from .base import MATRIX, ParamSpec, Part, Source
+from .base import ANY, MATRIX, ParamSpec, Part, Source
 
 
 class TokenEmbedding(Part):
@@ -26,6 +26,10 @@ class TokenEmbedding(Part):
         """What the embedding keeps per request (as a mixer's ``cache_spec``); nothing here."""
         return None
 
+    def position_limit(self) -> Optional[int]:
+        """The most positions a request may have, or None where the embedding sets no limit."""
+        return None
+
     def forward(self, ctx, cache=None) -> torch.Tensor:
         if self.scale == 1.0:
             return ctx.K.embed(ctx.token_ids, self.table)
@@ -34,6 +38,30 @@ class TokenEmbedding(Part):
     def add_into(self, ctx, residual: torch.Tensor) -> None:
         """``residual += table[token] * scale``: the step's embedding once more, for a model that feeds it in again on the way."""
         ctx.K.embed_add(ctx.token_ids, self.table, residual, self.scale)
+
+
+class PositionedEmbedding(TokenEmbedding):
+    """``x = table[token] * scale + positions[p]`` for the token at position p of its request, the sum in 32-bit. ``max_positions`` rows
+    (None: the checkpoint's tensor decides): no request can become longer than that."""
+
+    def __init__(self, vocab: int, hidden: int, name: str, position_name: str, max_positions: Optional[int] = None, scale: float = 1.0,
+                 random_positions: int = 256):
+        super().__init__(vocab, hidden, name, scale)
+        self.position_name, self.max_positions, self.random_positions = position_name, max_positions, int(random_positions)
+        self.position_table: Optional[torch.Tensor] = None
+
+    def params(self) -> Dict[str, ParamSpec]:
+        rows = self.max_positions if self.max_positions else ANY
+        return {**super().params(), "position_table": ParamSpec((Source(self.position_name, (rows, self.hidden), free=self.random_positions),), MATRIX)}
+
+    def position_limit(self) -> Optional[int]:
+        return self.max_positions if self.position_table is None else self.position_table.shape[0]
+
+    def forward(self, ctx, cache=None) -> torch.Tensor:
+        return ctx.K.embed_positions(ctx.token_ids, self.table, ctx.positions, self.position_table, self.scale)
+
+    def add_into(self, ctx, residual: torch.Tensor) -> None:
+        raise ValueError("an embedding with positions is not fed in again on the way")
 
 
 class BigramEmbedding(TokenEmbedding):

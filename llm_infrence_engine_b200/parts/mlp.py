@@ -41,11 +41,11 @@ class GatedMLP(FeedForward):
 
 class DenseMLP(FeedForward):
     """``down(act(up(x)))`` without biases; ``act`` is the tanh form of GELU,
-    ``0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))``, or the exact one (``gelu_erf``), ``0.5 z (1 + erf(z / sqrt(2)))``, computed in
-    32-bit on the product's sums."""
+    ``0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))``, the exact one (``gelu_erf``), ``0.5 z (1 + erf(z / sqrt(2)))``, or the square
+    of the positive part (``relu2``), ``max(z, 0)^2``, computed in 32-bit on the product's sums."""
 
     graph_safe = True
-    ACTIVATIONS = ("gelu_tanh", "gelu_erf")
+    ACTIVATIONS = ("gelu_tanh", "gelu_erf", "relu2")
 
     def __init__(self, hidden: int, intermediate: int, up_name: str, down_name: str, activation: str = "gelu_tanh"):
         if activation not in self.ACTIVATIONS:
@@ -111,9 +111,11 @@ class GatedUnit(FeedForward):
         return {"w_gate_up": ParamSpec((Source(self.gate_name, (i, h), INIT_PROJ), Source(self.up_name, (i, h), INIT_PROJ)), MATRIX),
                 "w_down": ParamSpec((Source(self.down_name, (h, i), INIT_PROJ),), MATRIX)}
 
-    def forward(self, ctx, h, residual):
+    def forward(self, ctx, h, residual, row_scale: Optional[torch.Tensor] = None):
+        """``row_scale`` (float32, one number per row, or None): the result of a row is multiplied by it (on its way into ``down``)."""
         K = ctx.K
-        K.linear(K.gate_up_act(h, self.w_gate_up, ctx.dtype, activation=self.activation), self.w_down, add_to=residual)
+        more = {"row_scale": row_scale} if row_scale is not None else {}
+        K.linear(K.gate_up_act(h, self.w_gate_up, ctx.dtype, activation=self.activation, **more), self.w_down, add_to=residual)
 
 
 class RoutedExperts(FeedForward):
@@ -131,7 +133,12 @@ class RoutedExperts(FeedForward):
     Other routers and experts, each a constructor argument:
 
     * ``scoring="sigmoid"``: ``s = sigmoid(W_router x)``, every output by itself, and the weights are the chosen ``s`` as they are;
+    * ``scoring="top_softmax"``: the ``top`` largest outputs of the router are taken as they are, their weights are the softmax over
+      the taken ones alone;
     * ``correction=False``: no correction vector in the checkpoint;
+    * ``router_bias``: a bias (``{prefix}.router.b``) is added to the router's outputs, in 32-bit;
+    * ``shared_gate``: names a row ``[1, hidden]``; the shared feed-forward's result is multiplied by ``sigmoid(row x)``, one number per
+      token. The row rides behind the router's own rows, so the gate comes out of the router's product;
     * ``weight_inputs``: the weight multiplies the expert's INPUT, the output is ``sum_k expert(w_k x)``;
     * ``expert_glu=(limit, alpha, shift)``: the experts are clamped units, ``down(g sigmoid(alpha g) (u + shift))`` with
       ``g = min(gate x, limit)`` and ``u = clamp(up x, -limit, limit)``."""
@@ -140,17 +147,23 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, hidden: int, intermediate: int, num_experts: int, num_identity: int, top: int, prefix: str,
                  shared: Optional[FeedForward] = None, scoring: str = "softmax", correction: bool = True, weight_inputs: bool = False,
-                 expert_glu: Optional[tuple] = None):
+                 expert_glu: Optional[tuple] = None, router_bias: bool = False, shared_gate: Optional[str] = None):
         if not 1 <= top <= num_experts + num_identity:
             raise ValueError(f"{top} of {num_experts + num_identity} router outputs cannot be chosen")
-        if scoring not in ("softmax", "sigmoid"):
-            raise ValueError(f"a router scores by 'softmax' or 'sigmoid', got {scoring!r}")
+        if scoring not in ("softmax", "sigmoid", "top_softmax"):
+            raise ValueError(f"a router scores by 'softmax', 'sigmoid' or 'top_softmax', got {scoring!r}")
+        if scoring == "top_softmax" and correction:
+            raise ValueError("logits that are chosen as they are have no correction")
+        if shared_gate and shared is None:
+            raise ValueError("a gate of the shared feed-forward needs one")
         if weight_inputs and num_identity:
             raise ValueError("weights on the experts' inputs are not built together with identity experts")
         self.hidden, self.intermediate, self.num_experts, self.num_identity, self.top = hidden, intermediate, num_experts, num_identity, top
         self.prefix, self.shared = prefix, shared
         self.scoring, self.has_correction, self.weight_inputs = scoring, bool(correction), bool(weight_inputs)
         self.expert_glu = None if expert_glu is None else tuple(float(v) for v in expert_glu)
+        self.has_router_bias, self.shared_gate = bool(router_bias), shared_gate
+        self.router_bias = None
         self.w_router = self.correction = self.w_gate_up = self.w_down = None
 
     def children(self):
@@ -160,11 +173,16 @@ class RoutedExperts(FeedForward):
         p, h, i, E = self.prefix, self.hidden, self.intermediate, self.num_experts
         total = E + self.num_identity
         gate_up = tuple(Source(f"{p}.e{e}.{n}", (i, h), INIT_PROJ) for e in range(E) for n in ("gate", "up"))
-        out = {"w_router": ParamSpec((Source(f"{p}.router", (total, h), INIT_PROJ),), MATRIX),
+        router = (Source(f"{p}.router", (total, h), INIT_PROJ),)
+        if self.shared_gate:   # the shared feed-forward's gate is one more row of the router's product
+            router += (Source(self.shared_gate, (1, h), INIT_PROJ),)
+        out = {"w_router": ParamSpec(router, MATRIX),
                "w_gate_up": ParamSpec(gate_up, MATRIX),
                "w_down": ParamSpec(tuple(Source(f"{p}.e{e}.down", (h, i), INIT_PROJ) for e in range(E)), MATRIX)}
         if self.has_correction:
             out["correction"] = ParamSpec((Source(f"{p}.correction", (total,), INIT_SMALL),), VECTOR)
+        if self.has_router_bias:
+            out["router_bias"] = ParamSpec((Source(f"{p}.router.b", (total,), INIT_SMALL),), VECTOR)
         return out
 
     def bind(self, tensors) -> None:
@@ -175,9 +193,16 @@ class RoutedExperts(FeedForward):
 
     def forward(self, ctx, h, residual):
         K = ctx.K
-        if self.scoring == "softmax" and not self.weight_inputs and self.expert_glu is None:
+        if self.scoring == "softmax" and not (self.weight_inputs or self.expert_glu or self.has_router_bias or self.shared_gate):
             ids, weights = K.moe_router(h, self.w_router, self.correction, self.top)
             K.moe_experts(h, ids, weights, self.w_gate_up, self.w_down, add_to=residual)
+        elif self.has_router_bias or self.shared_gate:
+            ids, weights, gates = K.moe_router(h, self.w_router, self.correction, self.top, scoring=self.scoring, bias=self.router_bias,
+                                               gates=1 if self.shared_gate else 0)
+            K.moe_experts(h, ids, weights, self.w_gate_up, self.w_down, add_to=residual, glu=self.expert_glu, weight_inputs=self.weight_inputs)
+            if self.shared is not None:
+                self.shared.forward(ctx, h, residual, **({"row_scale": gates} if self.shared_gate else {}))
+            return
         else:
             ids, weights = K.moe_router(h, self.w_router, self.correction, self.top, scoring=self.scoring)
             K.moe_experts(h, ids, weights, self.w_gate_up, self.w_down, add_to=residual, glu=self.expert_glu, weight_inputs=self.weight_inputs)

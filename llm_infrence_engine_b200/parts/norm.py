@@ -17,6 +17,9 @@ class RMSNorm(Norm):
     ``offset``: what is added to the stored weight before it is used. A checkpoint that keeps its norm weights around zero
     (the scaling is ``1 + w``) has ``offset = 1``; the sum is made once, in 32-bit, when the weights are bound.
 
+    ``add_normed(ctx, residual, y)`` closes a sublayer, ``residual += weight * y / sqrt(mean(y^2) + eps)`` in 32-bit, put off until
+    the stream is read next.
+
     ``norm_streams``: the norm of a weighted sum of several residual streams ``[N, streams, dim]``, everything in 32-bit up
     to the one rounding of the result (the kernel also carries out a stream update that was put off until now).
     """
@@ -45,6 +48,9 @@ class RMSNorm(Norm):
 
     def norm_rows(self, ctx, residual, rows):
         return ctx.K.rmsnorm_rows(residual, None, self.weight, self.eps, rows, ctx.dtype)
+
+    def add_normed(self, ctx, residual, y) -> None:
+        ctx.K.post_rms_add(residual, y, self.weight, self.eps)
 
 
 class LayerNorm(Norm):

@@ -368,6 +368,62 @@ class MatrixMemoryMixer(Mixer):
         K.linear(y, self.w_o, add_to=residual)
 
 
+class DecayedLinearAttention(Mixer):
+    """Linear attention with a fixed decay per head (lightning attention). With ``q = silu(W_q x)`` and ``k = silu(W_k x)`` of
+    ``num_heads x head_dim`` and ``v = silu(W_v x)`` of ``num_heads x v_head_dim``, per head and in the order of the tokens:
+
+        S <- decay[h] S + k v^T;   o = S^T q
+
+    with ``S [head_dim, v_head_dim]`` starting at zero. The heads side by side are divided by their common root mean square and
+    multiplied by a weight of ``heads * v_head_dim`` entries and by ``sigmoid(W_g x)``; then the output projection. The decays are
+    constants of the model, not tensors. The four projections are one matrix; the state is a request's own, in 32-bit, kept column by
+    column. Checkpoint names: ``{prefix}.q / k / v / g / o``, ``.norm``."""
+
+    graph_safe = True
+
+    def __init__(self, hidden: int, num_heads: int, head_dim: int, v_head_dim: int, decay: Sequence[float], eps: float, prefix: str):
+        if len(decay) != num_heads:
+            raise ValueError(f"{num_heads} heads need a decay each, got {len(decay)}")
+        if head_dim > 256:
+            raise ValueError(f"the recurrence's kernel keeps a column of the state in registers: head_dim {head_dim} is more than 256")
+        self.hidden, self.num_heads, self.head_dim, self.v_head_dim = hidden, num_heads, head_dim, v_head_dim
+        self.decay_values, self.eps, self.prefix = tuple(float(d) for d in decay), float(eps), prefix
+        self.q_col = self.k_col = self.v_col = self.g_col = 0     # columns of the joined projection's sections: set when the weights are bound
+        self.w_in = self.w_o = self.norm_w = self.decay = None
+
+    def params(self) -> Dict[str, ParamSpec]:
+        p, h, H, D, DV = self.prefix, self.hidden, self.num_heads, self.head_dim, self.v_head_dim
+        return {
+            "w_in": ParamSpec(tuple(Source(f"{p}.{n}", (c, h), INIT_PROJ) for n, c in (("q", H * D), ("k", H * D), ("v", H * DV), ("g", H * DV))), MATRIX),
+            "w_o": ParamSpec((Source(f"{p}.o", (h, H * DV), INIT_PROJ),), MATRIX),
+            "norm_w": ParamSpec((Source(f"{p}.norm", (H * DV,), INIT_NORM),), VECTOR),
+        }
+
+    def bind(self, tensors) -> None:
+        super().bind(tensors)
+        H, D, DV = self.num_heads, self.head_dim, self.v_head_dim
+        # every section of the joined projection starts on a multiple of 8 rows: its columns of the product then start on a 16-byte boundary
+        pieces, starts, at = [], [], 0
+        for part in torch.split(self.w_in, (H * D, H * D, H * DV, H * DV)):
+            starts.append(at)
+            pieces.append(_padded(part))
+            at += pieces[-1].shape[0]
+        self.q_col, self.k_col, self.v_col, self.g_col = starts
+        self.w_in = torch.cat(pieces).contiguous()
+        self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=self.w_in.device)
+
+    def cache_spec(self):
+        return FixedStateSpec((self.num_heads, self.v_head_dim, self.head_dim))   # S column by column
+
+    def forward(self, ctx, h, cache, residual):
+        K = ctx.K
+        H, D, DV = self.num_heads, self.head_dim, self.v_head_dim
+        z = K.linear(h, self.w_in, out_dtype=ctx.dtype)
+        o = K.linear_attention(z, self.q_col, self.k_col, self.v_col, H, D, DV, self.decay, cache.state, ctx)
+        y = K.group_rmsnorm_gate(o, z, self.g_col, self.norm_w, H * DV, self.eps, gate_first=False, out_dtype=ctx.dtype)
+        K.linear(y, self.w_o, add_to=residual)
+
+
 class ParallelMixer(Mixer):
     """Two mixers side by side on the same input, each with its own cache or state. Two ways of joining their outputs:
 

@@ -23,6 +23,9 @@ class TorchKernels:
     def embed(self, token_ids, table, scale=1.0):
         return table[token_ids.long()].float() * scale
 
+    def embed_positions(self, token_ids, table, positions, position_table, scale=1.0):
+        return table[token_ids.long()].float() * scale + position_table[positions.long()].float()
+
     def embed_bigram(self, token_ids, table, bigram, buckets, mul_prev, mul_cur, positions, token_seq, seq_starts, num_seqs, last, scale=1.0):
         out = table[token_ids.long()].float() * scale
         for r in range(num_seqs):
@@ -140,7 +143,9 @@ class TorchKernels:
                 out[t, h] = pr @ v[:, h // rep]
         return out.reshape(N, num_heads * d).to(qkv.dtype)
 
-    def gate_up_act(self, x, w_gate_up, out_dtype=None, glu=None, activation="silu"):
+    def gate_up_act(self, x, w_gate_up, out_dtype=None, glu=None, activation="silu", row_scale=None):
+        if row_scale is not None:
+            return (self.gate_up_act(x.float(), w_gate_up.float(), torch.float32, glu, activation) * row_scale.view(-1, 1)).to(out_dtype or x.dtype)
         if activation == "gelu_tanh":
             gu = self.linear(x, w_gate_up, out_dtype=torch.float32)
             i = gu.shape[1] // 2
@@ -182,6 +187,8 @@ class TorchKernels:
         z = x.float() @ w.float().T
         if activation == "gelu_erf":
             return (0.5 * z * (1.0 + torch.erf(z / math.sqrt(2.0)))).to(out_dtype or x.dtype)
+        if activation == "relu2":
+            return (z.clamp(min=0) ** 2).to(out_dtype or x.dtype)
         if activation != "gelu_tanh":
             raise ValueError(activation)
         y = 0.5 * z * (1.0 + torch.tanh(math.sqrt(2.0 / math.pi) * (z + 0.044715 * z ** 3)))
@@ -197,7 +204,7 @@ class TorchKernels:
     def attention_ext(self, q, q_col, num_heads, num_kv_heads, head_dim, v_head_dim, k_pool, v_pool, block_table, token_seq, positions,
                       page_size, scale, window, max_context, temp=(0.0, 0), rel=None, rel_rows=None, sink=None, gate=None, gate_col=0,
                       gate_per_head=False, batch=None, num_splits=None, keep_first=0, chunk=0, softcap=0.0, talk=None,
-                      sigmoid_bias=None, log_distance=None, turn=None):
+                      sigmoid_bias=None, log_distance=None, turn=None, key_scale=None):
         N = q.shape[0]
         rep = num_heads // num_kv_heads
         qs = q[:, q_col:q_col + num_heads * head_dim].float().view(N, num_heads, head_dim)
@@ -212,6 +219,8 @@ class TorchKernels:
             offs = (keys % page_size).long()
             k = k_pool[pages, :, offs].float()                                   # [S, kv heads, head_dim]
             v = v_pool[pages, :, offs].float() if v_pool is not None else k[..., :v_head_dim]
+            if key_scale is not None:   # a number per token multiplies its keys (not the values inside them)
+                k = k * key_scale[pages, offs][:, None, None]
             factor = scale
             if temp[1]:
                 factor = scale * (1.0 + temp[0] * math.log((p + 1) // temp[1] + 1))
@@ -251,6 +260,56 @@ class TorchKernels:
             else:
                 out = out * torch.sigmoid(gate[:, gate_col:gate_col + num_heads * v_head_dim].float()).view(N, num_heads, v_head_dim)
         return out.reshape(N, num_heads * v_head_dim).to(q.dtype)
+
+    # ------------------------------------------------------------------ a stream that is read as it is, results that are normed
+    def stream_rows(self, residual, out_dtype):
+        return residual.to(out_dtype)
+
+    def post_rms_add(self, residual, y, weight, eps):
+        y = y.float()
+        residual += y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps) * weight.float()
+
+    def qk_rows_norm_store(self, z, num_heads, num_kv_heads, head_dim, v_head_dim, q_weight, k_weight, eps, slot_mapping, k_pool, v_pool, key_scale,
+                           page_size, gate_cols=0, write_kv=True, out_dtype=None):
+        N = z.shape[0]
+        nq, nk = num_heads * head_dim, num_kv_heads * head_dim
+        zf = z.float()
+        q, k = zf[:, :nq], zf[:, nq:nq + nk]
+        q = q * torch.rsqrt(q.pow(2).mean(-1, keepdim=True) + eps) * q_weight.float()
+        rk = torch.rsqrt(k.pow(2).mean(-1, keepdim=True) + eps)
+        page, off = (slot_mapping // page_size).long(), (slot_mapping % page_size).long()
+        if key_scale is not None:    # values are keys: the keys as they are, their number beside them, their weight on the queries
+            w = k_weight.float().view(num_kv_heads, 1, head_dim).expand(-1, num_heads // num_kv_heads, -1)
+            q = q * w.reshape(1, nq)
+            g0 = nq + nk
+            if write_kv:
+                key_scale[page, off] = rk[:, 0]
+        else:
+            v = zf[:, nq + nk:nq + nk + num_kv_heads * v_head_dim]
+            g0 = nq + nk + v.shape[1]
+            k = k * rk * k_weight.float()
+            if write_kv:
+                v_pool[page, :, off] = v.reshape(N, num_kv_heads, v_head_dim).to(v_pool.dtype)
+        if write_kv:
+            k_pool[page, :, off] = k.reshape(N, num_kv_heads, head_dim).to(k_pool.dtype)
+        out = torch.cat([q, zf[:, g0:g0 + gate_cols]], dim=1)
+        out = torch.cat([out, out.new_zeros(N, -out.shape[1] % 8)], dim=1)
+        return out.to(out_dtype or z.dtype)
+
+    def linear_attention(self, z, q_col, k_col, v_col, num_heads, head_dim, v_head_dim, decay, state, batch):
+        N = z.shape[0]
+        H, D, DV = num_heads, head_dim, v_head_dim
+        a = z.float()
+        a = a * torch.sigmoid(a)
+        q, k, v = (a[:, c:c + H * n].view(N, H, n) for c, n in ((q_col, D), (k_col, D), (v_col, DV)))
+        out = torch.zeros(N, H, DV)
+        for slot, s0, s1 in self._requests(batch):
+            S = state[slot].clone()                     # kept column by column: [heads, v_head_dim, head_dim]
+            for n in range(s0, s1):
+                S = decay[:, None, None] * S + v[n][:, :, None] * k[n][:, None, :]
+                out[n] = torch.einsum("hcd,hd->hc", S, q[n])
+            state[slot] = S
+        return out.reshape(N, H * DV)
 
     # ------------------------------------------------------------------ layer norm before and after a sublayer
     @staticmethod
@@ -422,7 +481,16 @@ class TorchKernels:
         return out.to(x.dtype)
 
     # ------------------------------------------------------------------ routed experts
-    def moe_route(self, logits, correction, top, scoring="softmax"):
+    def moe_route(self, logits, correction, top, scoring="softmax", bias=None, gates=0):
+        if bias is not None or gates or scoring == "top_softmax":
+            total = logits.shape[1] - gates
+            z = logits[:, :total].float() + (0.0 if bias is None else bias.float())
+            if scoring == "top_softmax":
+                values, ids = torch.topk(z, top, dim=-1)
+                out = ids.to(torch.int32), torch.softmax(values, dim=-1)
+            else:
+                out = self.moe_route(z, correction, top, scoring)
+            return (*out, torch.sigmoid(logits[:, total:].float()))
         if scoring == "sigmoid":
             s = torch.sigmoid(logits.float())
         else:
@@ -432,8 +500,8 @@ class TorchKernels:
         w = torch.gather(s, 1, ids)
         return ids.to(torch.int32), w if scoring == "sigmoid" else w / (w.sum(-1, keepdim=True) + 1e-20)
 
-    def moe_router(self, h, w_router, correction, top, scoring="softmax"):
-        return self.moe_route(h.float() @ w_router.float().T, correction, top, scoring)
+    def moe_router(self, h, w_router, correction, top, scoring="softmax", bias=None, gates=0):
+        return self.moe_route(h.float() @ w_router.float().T, correction, top, scoring, bias, gates)
 
     def moe_experts(self, h, ids, weights, w_gate_up, w_down, add_to, glu=None, weight_inputs=False):
         E, F = w_gate_up.shape[0], w_gate_up.shape[1] // 2
