@@ -20,8 +20,8 @@ batch of 8 requests and a context of 8192 tokens. A "step" is one decode step of
 ``roofline``  bytes a decode step must read (every weight once + the live requests' cache) / its time.
 ``points``    decode tokens per second at batch 1 and 64, same method as ``value``.
 
-``--workload serving | luvutar | zepalorn | mufotar | memilorn | sinorax`` measure other things (a stream of requests through the engine; the other architectures
-beside Qwen2 of equal size, Mufotar beside Zepalorn, with ``--kernels`` also kernel by kernel) and print lines of their own; the default line is
+``--workload serving | luvutar | zepalorn | mufotar | memilorn | sinorax | putelix`` measure other things (a stream of requests through the engine; the other
+architectures beside Qwen2 of equal size, Mufotar and Putelix beside Zepalorn, with ``--kernels`` also kernel by kernel) and print lines of their own; the default line is
 unchanged by them.
 
 Peaks come from MEASURED_PEAKS.json beside this file when it exists, else 6.65 TB/s and 1.59 PFLOP/s.
@@ -572,6 +572,8 @@ def model_points(folder: Path, vocab: int, batch: int, context: int, prefill_tok
             b.k.normal_(0, 0.5)
             if b.v is not None:
                 b.v.normal_(0, 0.5)
+            if b.scalar is not None:
+                b.scalar.fill_(2.0)
 
     for b in runner.bindings:
         fill(b)
@@ -606,7 +608,7 @@ def model_points(folder: Path, vocab: int, batch: int, context: int, prefill_tok
             seen = min(seen, (context - 1) % g.chunk + 1)
         if getattr(g, "window", None):
             seen = min(context, seen + getattr(g, "keep_first", 0))
-        return 2 * seen * g.num_kv_heads * (g.head_dim + (g.head_dim if g.v_head_dim is None else g.v_head_dim))
+        return seen * (2 * g.num_kv_heads * (g.head_dim + (g.head_dim if g.v_head_dim is None else g.v_head_dim)) + (4 if g.token_scalar else 0))
 
     held = sum(live(g) for cs in spec.cache_specs() for g in flatten_specs(cs))
     out = {"decode_ms": round(dec_ms, 4), "decode_tok_s": round(batch / dec_ms * 1e3, 1), "launches_per_step": cap.launches,
@@ -1481,6 +1483,204 @@ def sinorax_workload(a) -> int:
     return 0
 
 
+# ---------------------------------------------------------------------------------------------------------------------
+# ``--workload putelix``: the Putelix decoder at layer sizes of real models, beside the Zepalorn decoder (the closest of the engine's
+# other models: chunked, capped attention beside a recurrence in every layer) of equal width, heads, state and weights per token.
+
+PUTELIX_SIZES = {
+    # name: (width, heads, kv heads, head_dim, chunk, linear-attention heads, key size, value size, dense ff, experts, chosen, expert ff,
+    #        shared ff, layers, vocab)
+    "1b-like": (1024, 8, 2, 128, 2048, 8, 128, 128, 4224, 16, 4, 512, 768, 8, 32768),
+    "3b-like": (2048, 16, 4, 128, 4096, 16, 128, 128, 8256, 32, 4, 768, 2432, 8, 32768),
+}
+PUTELIX_NAMES = ("width", "heads", "kv_heads", "head_dim", "chunk", "linear_heads", "linear_dim", "linear_vdim", "dense_ff", "experts", "top", "expert_ff",
+                 "shared_ff", "layers", "vocab")
+
+
+def putelix_config(size: str) -> dict:
+    """Every layer both halves of the mixer; dense feed-forwards and routed experts in turn."""
+    W, H, G, d, chunk, lh, ld, lv, ff, E, top, eff, sff, layers, vocab = PUTELIX_SIZES[size]
+    left = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "softcap": 50.0, "bias_max": 1024, "mask": {"size": chunk}}
+    right = {"heads": lh, "dim": ld, "vdim": lv, "decay": [1.0 - 2.0 ** -(1 + 8 * (h + 1) / lh) for h in range(lh)]}
+    moe = {"kind": "moe", "expert": {"ff": eff}, "router": {"experts": E, "top": top}, "shared": {"ff": sff}}
+    return {"architecture": "Putelix", "vocab": vocab, "width": W, "norm": {"eps": 1e-6}, "max_positions": 8192,
+            "layers": [{"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": moe if i % 2 else {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
+def zepalorn_beside_putelix(size: str) -> dict:
+    """The same attention (with a value pool and short convolutions), a state-space mixer whose state is as large, and gated
+    feed-forwards of the weights that a Putelix token reads."""
+    W, H, G, d, chunk, lh, ld, lv, ff, E, top, eff, sff, layers, vocab = PUTELIX_SIZES[size]
+    left = {"heads": H, "kv_heads": G, "dim": d, "vdim": d, "scale": d ** -0.5, "conv": 4, "softcap": 50.0, "mask": {"size": chunk}}
+    right = {"heads": lh * lv // 64, "vdim": 64, "state": ld, "groups": 1, "norm_groups": 1, "conv": 4}
+    return {"architecture": "Zepalorn", "vocab": vocab, "width": W, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+            "layers": [{"type": "parallel", "mixer": {"left": left, "right": right},
+                        "mlp": {"kind": "dense", "ff": top * eff + sff if i % 2 else ff * 2 // 3, "limit": 7.0}} for i in range(layers)]}
+
+
+def putelix_kernel_points(torch, pk, size: str) -> dict:
+    """Putelix's kernels one by one, each beside the kernel of the engine's other models that does the like job at the same size:
+    microseconds, and the fraction of its roofline (bytes that must move / copy peak, or flops / bf16 peak)."""
+    from types import SimpleNamespace
+
+    from llm_infrence_engine_b200.csrc import get_kernels
+
+    K = get_kernels()
+    W, H, G, d, chunk, lh, ld, lv, ff, E, top, eff, sff, _, vocab = PUTELIX_SIZES[size]
+    bf, dev = torch.bfloat16, "cuda"
+    hbm, tf = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    out = {}
+
+    def entry(us, bytes_=None, flops=None):
+        e = {"us": round(us, 2)}
+        if bytes_ is not None:
+            e["frac_of_copy_peak"] = round(bytes_ / (us * 1e-6) / hbm, 4)
+        if flops is not None:
+            e["frac_of_bf16_peak"] = round(flops / (us * 1e-6) / tf, 4)
+        return e
+
+    r = lambda *n: torch.randn(*n, device=dev)
+    one = torch.ones(W, device=dev)
+    for what, batch, ctx, T in (("decode", 8, 4096, 1), ("decode_b64", 64, 4096, 1), ("prefill", 1, 2048, 2048)):
+        per = -(-ctx // BLOCK)
+        table = torch.zeros((batch + 1, per), dtype=torch.int32, device=dev)
+        table[:batch] = (torch.randperm(batch * per, device=dev).to(torch.int32) + 1).view(batch, per)
+        N = batch * T
+        seq = torch.arange(batch, dtype=torch.int32, device=dev).repeat_interleave(T)
+        pos = (torch.arange(T, dtype=torch.int32, device=dev) + (ctx - T)).repeat(batch)
+        starts = torch.arange(0, N + 1, T, dtype=torch.int32, device=dev)
+        b = SimpleNamespace(seq_lens=[T] * batch, seq_starts_dev=starts, num_seqs=batch, max_seq_len=T, _tables={},
+                            seq_slots=torch.arange(batch, dtype=torch.int32, device=dev))
+        kp, vp = r(batch * per + 1, G, BLOCK, d).to(bf), r(batch * per + 1, G, BLOCK, d).to(bf)
+        scalar = torch.full((batch * per + 1, BLOCK), 1.0, device=dev)
+        q = r(N, H * d + H + -H % 8).to(bf)
+        rel, rows = r(32, H) * 0.1, torch.tensor([min(31, i) for i in range(1024)], dtype=torch.int32, device=dev)
+        seen = min(ctx, chunk)
+        if T == 1:
+            moved = lambda pools: batch * seen * (pools * G * d * 2)
+            fl = None
+        else:
+            moved = lambda pools: None
+            fl = 4.0 * H * d * sum(p % chunk + 1 for p in range(ctx - T, ctx)) * batch
+
+        def attention(v, **kw):
+            b._tables.clear()
+            K.attention_ext(q, 0, H, G, d, d, kp, v, table, seq, pos, BLOCK, d ** -0.5, 0, ctx, batch=b, chunk=chunk, softcap=50.0, **kw)
+
+        out[f"attention_{what}_zepalorn"] = entry(_time_graph(lambda: attention(vp), torch), moved(2), fl)
+        out[f"attention_{what}_putelix"] = entry(_time_graph(lambda: attention(None, key_scale=scalar, rel=rel, rel_rows=rows, gate=q, gate_col=H * d, gate_per_head=True), torch),
+                                                 moved(1), fl)
+        # what lies between the projection and the attention
+        slots = torch.randperm(batch * per * BLOCK, device=dev)[:N].to(torch.int32)
+        zq = r(N, (H + 2 * G) * d).to(bf)
+        wh, wq, wk = torch.ones(d, device=dev), torch.ones(H * d, device=dev), torch.ones(G * d, device=dev)
+        cos, sin = r(N, d // 2), r(N, d // 2)
+        out[f"heads_{what}_zepalorn"] = entry(_time_graph(lambda: K.qk_norm_rope_store(zq, H, G, d, d, wh, wh, 1e-6, cos, sin, d, True, slots, kp, vp, BLOCK), torch), N * 4 * (H + 2 * G) * d)
+        zk = r(N, (H + G) * d + H + -H % 8).to(bf)
+        out[f"heads_{what}_putelix"] = entry(_time_graph(lambda: K.qk_rows_norm_store(zk, H, G, d, d, wq, wk, 1e-6, slots, kp, None, scalar, BLOCK, gate_cols=H), torch),
+                                             N * 4 * ((H + G) * d + H))
+        del kp, vp
+        # the recurrences
+        sh = lh * lv // 64
+        xbc, dt = r(N, sh * 64 + 2 * ld).to(bf) * 0.5, r(N, sh).to(bf)
+        A3, b3, k3 = torch.zeros(sh, device=dev), torch.full((sh,), -3.0, device=dev), torch.ones(sh, device=dev)
+        st3 = torch.zeros(batch + 1, sh, 64, ld, device=dev)
+        held = batch * 2 * 4 * lh * ld * lv
+        out[f"recurrence_{what}_zepalorn"] = entry(_time_graph(lambda: K.ssm_scan(xbc, sh, 1, ld, 64, dt, 0, A3, b3, k3, st3, b), torch),
+                                                   held + N * (2 * (sh * 64 + 2 * ld) + 4 * sh * 64), 6.0 * N * sh * 64 * ld)
+        zl = r(N, 2 * lh * ld + 2 * lh * lv).to(bf)
+        decay, st4 = torch.full((lh,), 0.99, device=dev), torch.zeros(batch + 1, lh, lv, ld, device=dev)
+        out[f"recurrence_{what}_putelix"] = entry(_time_graph(lambda: K.linear_attention(zl, 0, lh * ld, 2 * lh * ld, lh, ld, lv, decay, st4, b, activated=T > 1), torch),
+                                                  held + N * (2 * (2 * lh * ld + lh * lv) + 4 * lh * lv), 6.0 * N * lh * lv * ld)
+        o, gw = r(N, lh * lv), torch.ones(lh * lv, device=dev)
+        out[f"gated_norm_{what}_zepalorn"] = entry(_time_graph(lambda: K.group_rmsnorm_gate(o, zl, 0, gw, lh * lv, 1e-6, True, bf), torch), N * lh * lv * (4 + 2 + 2))
+        out[f"gated_norm_{what}_putelix"] = entry(_time_graph(lambda: K.group_rmsnorm_gate(o, zl, 2 * lh * ld + lh * lv, gw, lh * lv, 1e-6, False, bf), torch), N * lh * lv * (4 + 2 + 2))
+        # the join of the two halves, the closing norm, the rows of the next sublayer
+        few = N <= K.tc_max_rows
+        ta = torch.float32 if few else bf
+        res, ya, yb, y = r(N, W), r(N, W).to(ta), r(N, W).to(ta), torch.zeros(N, W, device=dev)
+        es = 4 if few else 2
+
+        def zepalorn_join():
+            K.dual_rmsnorm_mix(ya, yb, one, one, 1e-6, 0.5, y)
+            K.post_norm_add(res, y, one, 1e-6)
+            return K.layernorm(res, one, 1e-6, bf)
+
+        def putelix_join():
+            t = K.zeros_like_rows(res)
+            K.dual_rmsnorm_mix(ya, yb, one, one, 1e-6, 0.5, t)
+            K.post_rms_add(res, t, one, 1e-6)
+            return K.stream_rows(res, bf)
+
+        out[f"join_{what}_zepalorn"] = entry(_time_graph(zepalorn_join, torch), N * W * (2 * es + 4 + 4 + 2))
+        out[f"join_{what}_putelix"] = entry(_time_graph(putelix_join, torch), N * W * (2 * es + 4 + 4 + 2))
+
+        # the feed-forwards at equal weights
+        h = r(N, W).to(bf)
+        ffg = ff * 2 // 3 // 8 * 8
+        wup, wgu = r(ff, W).to(bf) * 0.02, r(2 * ffg, W).to(bf) * 0.02
+        out[f"ff_in_{what}_zepalorn"] = entry(_time_graph(lambda: K.gate_up_act(h, wgu, bf, glu=(7.0, 1.702, 1.0)), torch),
+                                              2 * ffg * W * 2 if T == 1 else None, 2.0 * N * W * 2 * ffg if T > 1 else None)
+        out[f"ff_in_{what}_putelix"] = entry(_time_graph(lambda: K.linear_act(h, wup, "relu2", bf), torch), ff * W * 2 if T == 1 else None,
+                                             2.0 * N * W * ff if T > 1 else None)
+        del wup, wgu
+        w_router, bias = r(E + 1, W).to(bf) * 0.05, torch.zeros(E, device=dev)
+        we_gu, we_dn = r(E, 2 * eff, W).to(bf) * 0.02, r(E, W, eff).to(bf) * 0.02
+        ws_gu, ws_dn = r(2 * sff, W).to(bf) * 0.02, r(W, sff).to(bf) * 0.02
+        ids, wts, gates = K.moe_router(h, w_router, None, top, scoring="top_softmax", bias=bias, gates=1)
+        used = int(torch.unique(ids).numel())
+        out[f"router_{what}_mufotar"] = entry(_time_graph(lambda: K.moe_router(h, w_router[:E], None, top), torch), N * W * 2 + E * W * 2)
+        out[f"router_{what}_putelix"] = entry(_time_graph(lambda: K.moe_router(h, w_router, None, top, scoring="top_softmax", bias=bias, gates=1), torch), N * W * 2 + (E + 1) * W * 2)
+
+        def shared(scale):
+            K.linear(K.gate_up_act(h, ws_gu, bf, **({"row_scale": scale} if scale is not None else {})), ws_dn, add_to=y)
+            K._pending_add = None
+
+        fl = 6.0 * N * W * sff if T > 1 else None
+        out[f"shared_{what}_mufotar"] = entry(_time_graph(lambda: shared(None), torch), 3 * sff * W * 2 if T == 1 else None, fl)
+        out[f"shared_{what}_putelix"] = entry(_time_graph(lambda: shared(gates), torch), 3 * sff * W * 2 if T == 1 else None, fl)
+        out[f"experts_{what}_both"] = entry(_time_graph(lambda: K.moe_experts(h, ids, wts, we_gu, we_dn, add_to=y), torch),
+                                            used * 3 * eff * W * 2 + N * W * (2 + 4), 6.0 * N * top * W * eff)
+        del we_gu, we_dn
+        toks = torch.randint(0, vocab, (N,), device=dev, dtype=torch.int32)
+        te, tp = r(vocab, W).to(bf), r(8192, W).to(bf)
+        out[f"embedding_{what}_zepalorn"] = entry(_time_graph(lambda: K.embed(toks, te), torch), N * W * (2 + 4))
+        out[f"embedding_{what}_putelix"] = entry(_time_graph(lambda: K.embed_positions(toks, te, pos, tp), torch), N * W * (2 + 2 + 4))
+    K.check_device_errors()
+    return out
+
+
+def putelix_workload(a) -> int:
+    import torch
+
+    from llm_infrence_engine_b200.weights import write_random_model
+
+    pk = peaks()
+    sampler = ClockSampler()
+    sampler.start()
+    sizes = {}
+    steps = min(a.steps, 256)
+    for size in PUTELIX_SIZES:
+        row = {}
+        for name, config in (("putelix", putelix_config(size)), ("zepalorn", zepalorn_beside_putelix(size))):
+            with tempfile.TemporaryDirectory() as tmp:
+                folder = write_random_model(config, Path(tmp) / "model", seed=0, store_dtype="bfloat16")
+                pt = model_points(folder, PUTELIX_SIZES[size][-1], a.batch, a.context or 4096, a.prefill_tokens, steps, max(a.warmup, 3), torch)
+            pt["decode_frac_of_copy_peak"] = round(pt["decode_bytes"] / (pt["decode_ms"] * 1e-3) / 1e9 / pk["hbm_gbs"], 4)
+            row[name] = pt
+        sizes[size] = row
+    line = {"metric": f"Putelix beside Zepalorn of equal size: decode (batch {a.batch}, context {a.context or 4096}) and prefill ({a.prefill_tokens} tokens), bf16, random weights",
+            "unit": "ms and tokens/s per size", "n_gpus": 1, "impl": "ours", "dtype": "bf16", "steps": steps, "warmup": max(a.warmup, 3),
+            "data": "synthetic: random weights (seed 0), uniform random token ids, synthetic cache contents",
+            "config": {"sizes": {k: dict(zip(PUTELIX_NAMES, v)) for k, v in PUTELIX_SIZES.items()}, "block_size": BLOCK, "peaks": pk["source"],
+                       "l2": "weights + cache per step larger than L2, no flush"},
+            "clocks": sampler.stop(), "sizes": sizes}
+    if a.kernels:
+        line["kernels"] = {size: putelix_kernel_points(torch, pk, size) for size in PUTELIX_SIZES}
+    print(json.dumps(line))
+    return 0
+
+
 def luvutar_workload(a) -> int:
     import torch
 
@@ -1528,13 +1728,14 @@ def main() -> int:
     ap.add_argument("--skip-e2e", action="store_true")
     ap.add_argument("--no-graphs", action="store_true", help="launch every kernel of a decode step from the host instead of replaying a CUDA graph")
     ap.add_argument("--only", default="all", choices=["all", "decode", "prefill"], help="measure one part only (for profiling); the JSON line then lacks the rest")
-    ap.add_argument("--workload", default="steps", choices=["steps", "serving", "luvutar", "zepalorn", "mufotar", "memilorn", "sinorax"],
+    ap.add_argument("--workload", default="steps", choices=["steps", "serving", "luvutar", "zepalorn", "mufotar", "memilorn", "sinorax", "putelix"],
                     help="serving: continuous batching of --requests requests (prompts U[128,2048], outputs U[64,512]) through Engine; "
                          "luvutar, zepalorn: that decoder at two layer sizes beside the Qwen2 decoder of equal size (decode and prefill); "
                          "mufotar: that decoder at two layer sizes beside the Zepalorn decoder of equal size; "
                          "memilorn: that decoder at two layer sizes beside the Mufotar decoder of equal size; "
-                         "sinorax: that decoder at two layer sizes beside the Qwen2 decoder of equal size")
-    ap.add_argument("--kernels", action="store_true", help="luvutar, zepalorn, mufotar, memilorn, sinorax: also time its kernels one by one beside their counterparts")
+                         "sinorax: that decoder at two layer sizes beside the Qwen2 decoder of equal size; "
+                         "putelix: that decoder at two layer sizes beside the Zepalorn decoder of equal size")
+    ap.add_argument("--kernels", action="store_true", help="luvutar, zepalorn, mufotar, memilorn, sinorax, putelix: also time its kernels one by one beside their counterparts")
     ap.add_argument("--requests", type=int, default=64)
     ap.add_argument("--token-budget", type=int, default=2048, help="serving: tokens per step (max_num_batched_tokens)")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="length of the timed prompt")
@@ -1554,6 +1755,8 @@ def main() -> int:
         return sinorax_workload(a)
     if a.workload == "memilorn":
         return memilorn_workload(a)
+    if a.workload == "putelix":
+        return putelix_workload(a)
     PREFILL_TOKENS = a.prefill_tokens
     shape_name, changes, shape_context = SHAPES[a.shape]
     MODEL.update(changes)

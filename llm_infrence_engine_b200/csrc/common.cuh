@@ -117,10 +117,11 @@ __device__ __forceinline__ float gelu_tanh_fast(float z) {
 
 // What a feed-forward's first product ends in; a compile-time choice, so that an epilogue's elements stand in one straight run of
 // instructions (a branch per element, even a uniform one, would leave nothing to overlap their latencies with).
-enum { UNIT_SILU = 0, UNIT_CLAMPED = 1, UNIT_GELU_TANH = 2, PLAIN_GELU_ERF = 3, PLAIN_GELU_TANH = 4, PLAIN_RELU2 = 5 };
+enum { UNIT_SILU = 0, UNIT_CLAMPED = 1, UNIT_GELU_TANH = 2, PLAIN_GELU_ERF = 3, PLAIN_GELU_TANH = 4, PLAIN_RELU2 = 5, PLAIN_SILU = 6 };
 template <int UNIT>
 __device__ __forceinline__ float plain_unit(float z) {
     if constexpr (UNIT == PLAIN_GELU_TANH) return gelu_tanh_fast(z);
+    if constexpr (UNIT == PLAIN_SILU) return __fdividef(z, 1.0f + __expf(-z));
     if constexpr (UNIT == PLAIN_RELU2) { const float r = fmaxf(z, 0.f); return r * r; }
     return gelu_erf_fast(z);
 }

@@ -609,12 +609,13 @@ LLMIE_API int llmie_kv_store(const void* z, int z_stride, int k_col, int v_col, 
 // ------------------------------------------------------------------------------------------------
 // out = act(in), elementwise in 32-bit. kind 0: the tanh form of GELU, 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)));
 // kind 1: a soft cap on a scaled input, param * tanh(scale z / param); kind 2: the exact GELU, 0.5 z (1 + erf(z / sqrt 2)); kind 3: scale z;
-// kind 4: the square of the positive part, max(z, 0)^2.
+// kind 4: the square of the positive part, max(z, 0)^2; kind 5: silu, z / (1 + exp(-z)).
 // With `clear_in` the input is set to zero after it was read (a float32 accumulation buffer of a split-K product).
 __device__ __forceinline__ float act_of(float z, int kind, float param, float scale) {
     if (kind == 1) return param * tanhf(scale * z / param);
     if (kind == 2) return 0.5f * z * (1.0f + erff(0.7071067811865476f * z));
     if (kind == 3) return scale * z;
+    if (kind == 5) return z / (1.0f + expf(-z));
     if (kind == 4) { const float r = fmaxf(z, 0.f); return r * r; }
     return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
@@ -653,7 +654,7 @@ __global__ void __launch_bounds__(128) act_vec_kernel(float* __restrict__ in, TO
 }
 
 // bfloat16 in and out, 8 elements (16 bytes) per thread. The result is rounded to bfloat16 (8 bits), so the hyperbolic tangent is
-// the fast 32-bit form (errors of about 1e-7). KIND: as in act_of, 0, 2 or 4.
+// the fast 32-bit form (errors of about 1e-7). KIND: as in act_of, 0, 2, 4 or 5.
 template <int KIND>
 __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict__ in, bf16* __restrict__ out, long long items) {
     pdl_trigger();
@@ -670,7 +671,7 @@ __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict_
 #pragma unroll
         for (int k = 0; k < 2; ++k) {
             const float v = z[2 * j + k];
-            y[k] = KIND == 4 ? fmaxf(v, 0.f) * fmaxf(v, 0.f) : (KIND == 2 ? gelu_erf_fast(v) : gelu_tanh_fast(v));
+            y[k] = KIND == 5 ? __fdividef(v, 1.0f + __expf(-v)) : KIND == 4 ? fmaxf(v, 0.f) * fmaxf(v, 0.f) : (KIND == 2 ? gelu_erf_fast(v) : gelu_tanh_fast(v));
         }
         const __nv_bfloat162 v2 = __floats2bfloat162_rn(y[0], y[1]);
         w[j] = *reinterpret_cast<const uint32_t*>(&v2);
@@ -681,10 +682,11 @@ __global__ void __launch_bounds__(256) act_bf16x8_kernel(const bf16* __restrict_
 LLMIE_API int llmie_act(void* in, void* out, long long total, int kind, int clear_in, float param, float scale, int in_dtype,
                         int out_dtype, cudaStream_t s) {
     if (total <= 0) return 0;
-    if (kind < 0 || kind > 4 || (kind == 1 && !(param > 0.f))) return LLMIE_ERR_BAD_ARGUMENT;
-    if ((kind == 0 || kind == 2 || kind == 4) && in_dtype == DT_BF16 && out_dtype == DT_BF16 && !clear_in && total % 8 == 0 && ((uintptr_t)in % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
+    if (kind < 0 || kind > 5 || (kind == 1 && !(param > 0.f))) return LLMIE_ERR_BAD_ARGUMENT;
+    if ((kind == 0 || kind == 2 || kind >= 4) && in_dtype == DT_BF16 && out_dtype == DT_BF16 && !clear_in && total % 8 == 0 && ((uintptr_t)in % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
         const dim3 blocks((unsigned)((total / 8 + 255) / 256));
         if (kind == 2) return launch_kernel(act_bf16x8_kernel<2>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
+        if (kind == 5) return launch_kernel(act_bf16x8_kernel<5>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
         if (kind == 4) return launch_kernel(act_bf16x8_kernel<4>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
         return launch_kernel(act_bf16x8_kernel<0>, blocks, dim3(256), 0, s, (const bf16*)in, (bf16*)out, total / 8);
     }

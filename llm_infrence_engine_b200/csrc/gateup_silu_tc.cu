@@ -263,10 +263,11 @@ LLMIE_API int llmie_gateup_silu_tc(const bf16* x, const bf16* w, bf16* out, int 
     return llmie_gateup_glu_tc(x, w, out, M, I, K, num_blocks, error_flag, 0.f, 1.f, 0.f, nullptr, s);
 }
 
-// act(x w^T) for w [N, K]: the same product without a gate; N a multiple of 16. form 0: the exact GELU, 1: its tanh form, 2: max(z, 0)^2.
+// act(x w^T) for w [N, K]: the same product without a gate; N a multiple of 16. form 0: the exact GELU, 1: its tanh form, 2: max(z, 0)^2, 3: silu.
 LLMIE_API int llmie_up_gelu_tc(const bf16* x, const bf16* w, bf16* out, int M, int N, int K, int num_blocks, int* error_flag, int form,
                                  cudaStream_t s) {
     if (N % 16) return LLMIE_ERR_BAD_ARGUMENT;
+    if (form == 3) return dispatch_single<PLAIN_SILU>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, nullptr, s);
     if (form == 2) return dispatch_single<PLAIN_RELU2>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, nullptr, s);
     if (form == 1) return dispatch_single<PLAIN_GELU_TANH>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, nullptr, s);
     return dispatch_single<PLAIN_GELU_ERF>(x, w, out, M, N / 2, K, num_blocks, error_flag, 0.f, 1.f, 0.f, nullptr, s);

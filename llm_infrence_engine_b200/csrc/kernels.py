@@ -76,6 +76,9 @@ class CudaKernels:
         self.use_plain_attention_for_ext = True
         self.masked_attention_tensor_cores = True    # kept first tokens, chunks and soft caps on the tensor-core kernels too
         self.use_fa_attention_ext = True     # prompt portions with heads of 64 / 128: the kernel in which a warp owns 16 rows and all keys of a chunk
+        # linear attention with fixed decays, bfloat16: steps whose longest request brings this many rows take the tensor-core form, on
+        # projections that are activated by the product that makes them; below, the scan activates them as it reads them
+        self.linear_attention_mma_rows = 24
         self.use_mma_attention_talk = True   # heads that talk, steps with prompt portions in bfloat16: plain scores and P V on the tensor cores
         self.head_matmul_library_rows = 64   # per-head products of latent attention: from this many rows on, one batched library product
         self.slice_keys = 1024         # generic attention: keys per slice, at fixed places of a request (a multiple of 32)
@@ -124,7 +127,8 @@ class CudaKernels:
                    "llmie_moe_tile_rows", "llmie_moe_router", "llmie_moe_gather", "llmie_moe_grouped_tc", "llmie_moe_grouped_tc_rows",
                    "llmie_embed_add", "llmie_mlstm_prepare", "llmie_mlstm_scan", "llmie_mlstm_finish", "llmie_paged_attention_talk",
                    "llmie_attention_talk_slice", "llmie_attention_talk_mma_fits", "llmie_paged_attention_talk_mma", "llmie_embed_bigram",
-                   "llmie_dynamic_tanh", "llmie_embed_positions", "llmie_post_rms", "llmie_qk_rows_norm_store", "llmie_linear_attention_scan"):
+                   "llmie_dynamic_tanh", "llmie_embed_positions", "llmie_post_rms", "llmie_qk_rows_norm_store", "llmie_linear_attention_scan",
+                   "llmie_linear_attention_mma", "llmie_linear_attention_mma_fits"):
             getattr(self.lib, fn).restype = ctypes.c_int
         # two forms of the gate/up kernel live in source files of their own, and the library also builds without them
         self._gate_up_cluster = self._gate_up_pair = self._gate_up_glu_pair = self._up_gelu_pair = None
@@ -1019,7 +1023,7 @@ class CudaKernels:
     # ------------------------------------------------------------------ a product with an activation behind it
     def linear_act(self, x, w, activation, out_dtype=None):
         """``act(x w^T)``; the activation is computed in 32-bit on the product's sums where those are at hand (small batches)."""
-        kinds = {"gelu_tanh": 0, "gelu_erf": 2, "relu2": 4}
+        kinds = {"gelu_tanh": 0, "gelu_erf": 2, "relu2": 4, "silu": 5}
         if activation not in kinds:
             raise KernelError(f"linear_act: activation '{activation}' is not built")
         out_dtype = out_dtype or x.dtype
@@ -1029,7 +1033,7 @@ class CudaKernels:
             # prompt portions: one tcgen05 kernel whose epilogue is the activation (the gate/up kernels without a gate)
             out = torch.empty((M, w.shape[0]), dtype=torch.bfloat16, device=x.device)
             fn = self._up_gelu_pair if (self.use_pair_gate_up and self._up_gelu_pair is not None and M >= self.pair_gate_up_min_rows) else self.lib.llmie_up_gelu_tc
-            self._check(fn(_ptr(x), _ptr(w), _ptr(out), M, w.shape[0], K_, self.num_sms, _ptr(self._errors(x.device)), {"gelu_erf": 0, "gelu_tanh": 1, "relu2": 2}[activation],
+            self._check(fn(_ptr(x), _ptr(w), _ptr(out), M, w.shape[0], K_, self.num_sms, _ptr(self._errors(x.device)), {"gelu_erf": 0, "gelu_tanh": 1, "relu2": 2, "silu": 3}[activation],
                            self._stream()), "linear_act (tcgen05)")
             return out
         z = self.linear(x, w, transient=True)
@@ -1764,11 +1768,20 @@ class CudaKernels:
                                             _ptr(out), H, G, NS, DV, batch.num_seqs, batch.max_seq_len, self._dt(xbc, "xbc"), self._stream()), "ssm_scan")
         return out
 
-    def linear_attention(self, z, q_col, k_col, v_col, num_heads, head_dim, v_head_dim, decay, state, batch):
+    def linear_attention_inputs(self, h, w_in, rows, head_dim, v_head_dim, batch, out_dtype):
+        """The projections of linear attention from one matrix ``w_in = [q, k, v: rows | gate]``: returns ``(z, activated, gate, gate_col)``. A
+        step with prompt portions in bfloat16 gets q, k and v through silu as their product's epilogue and the gate from a product of its
+        own; any other step gets one product of everything, and ``linear_attention`` activates what it reads."""
+        if (h.dtype == torch.bfloat16 and out_dtype == torch.bfloat16 and batch.max_seq_len >= self.linear_attention_mma_rows and rows % 8 == 0
+                and self.lib.llmie_linear_attention_mma_fits(head_dim, v_head_dim)):
+            return self.linear_act(h, w_in[:rows], "silu", out_dtype), True, self.linear(h, w_in[rows:], out_dtype=out_dtype), 0
+        return (z := self.linear(h, w_in, out_dtype=out_dtype)), False, z, rows
+
+    def linear_attention(self, z, q_col, k_col, v_col, num_heads, head_dim, v_head_dim, decay, state, batch, activated=False):
         """Linear attention with a fixed decay per head over the rows of each request: per head ``S <- decay[h] S + k v^T``, ``o = S^T q`` with
         ``q``, ``k`` (``heads * head_dim`` columns of ``z`` from ``q_col``, ``k_col``) and ``v`` (``heads * v_head_dim`` from ``v_col``) passing silu
-        first; from ``state [slots, heads, v_head_dim, head_dim]`` (a head's ``S`` kept column by column), which is moved on. Returns float32
-        ``[N, heads * v_head_dim]``."""
+        first (``activated``, bfloat16: they have passed it already, and the tensor-core form runs); from ``state [slots, heads, v_head_dim,
+        head_dim]`` (a head's ``S`` kept column by column), which is moved on. Returns float32 ``[N, heads * v_head_dim]``."""
         self._need(z, "z", None, 2)
         self._need(state, "state", torch.float32, 4)
         self._need(decay, "decay", torch.float32, 1)
@@ -1778,6 +1791,12 @@ class CudaKernels:
         if tuple(state.shape[1:]) != (H, DV, D):
             raise KernelError(f"linear_attention: state is {list(state.shape)}, expected [slots, {H}, {DV}, {D}]")
         out = torch.empty((z.shape[0], H * DV), dtype=torch.float32, device=z.device)
+        if activated:
+            self._need(z, "z", torch.bfloat16)
+            self._check(self.lib.llmie_linear_attention_mma(_ptr(z), z.shape[1], int(q_col), int(k_col), int(v_col), _ptr(decay), _ptr(state),
+                                                            _ptr(batch.seq_starts_dev), _ptr(batch.seq_slots), _ptr(out), H, D, DV, batch.num_seqs,
+                                                            self._stream()), "linear_attention (tensor cores)")
+            return out
         self._check(self.lib.llmie_linear_attention_scan(_ptr(z), z.shape[1], int(q_col), int(k_col), int(v_col), _ptr(decay), _ptr(state),
                                                          _ptr(batch.seq_starts_dev), _ptr(batch.seq_slots), _ptr(out), H, D, DV, batch.num_seqs,
                                                          batch.max_seq_len, self._dt(z, "z"), self._stream()), "linear_attention")

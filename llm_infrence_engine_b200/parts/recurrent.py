@@ -418,9 +418,9 @@ class DecayedLinearAttention(Mixer):
     def forward(self, ctx, h, cache, residual):
         K = ctx.K
         H, D, DV = self.num_heads, self.head_dim, self.v_head_dim
-        z = K.linear(h, self.w_in, out_dtype=ctx.dtype)
-        o = K.linear_attention(z, self.q_col, self.k_col, self.v_col, H, D, DV, self.decay, cache.state, ctx)
-        y = K.group_rmsnorm_gate(o, z, self.g_col, self.norm_w, H * DV, self.eps, gate_first=False, out_dtype=ctx.dtype)
+        z, activated, gate, gate_col = K.linear_attention_inputs(h, self.w_in, self.g_col, D, DV, ctx, ctx.dtype)
+        o = K.linear_attention(z, self.q_col, self.k_col, self.v_col, H, D, DV, self.decay, cache.state, ctx, activated=activated)
+        y = K.group_rmsnorm_gate(o, gate, gate_col, self.norm_w, H * DV, self.eps, gate_first=False, out_dtype=ctx.dtype)
         K.linear(y, self.w_o, add_to=residual)
 
 

@@ -115,8 +115,17 @@ def route(logits, top: int):
     return ids, torch.softmax(values, dim=-1)
 
 
-def routed_experts(mlp: dict, W: Dict[str, torch.Tensor], p: str, h):
-    ids, weights = route(h @ W[f"{p}.router"].T + W[f"{p}.router.b"], int(mlp["router"]["top"]))
+def routed_experts(mlp: dict, W: Dict[str, torch.Tensor], p: str, h, forced=None, regret_out: Optional[list] = None):
+    """``forced [T, top]``: these experts are taken instead of the router's own choice (their weights are still the softmax over the
+    router's logits for them); ``regret_out`` then collects, per token, how far the smallest logit taken lies below the smallest of the
+    router's own choice."""
+    logits = h @ W[f"{p}.router"].T + W[f"{p}.router.b"]
+    ids, weights = route(logits, int(mlp["router"]["top"]))
+    if forced is not None:
+        taken = logits.gather(1, forced)
+        if regret_out is not None:
+            regret_out.append(logits.gather(1, ids).min(-1).values - taken.min(-1).values)
+        ids, weights = forced, torch.softmax(taken, dim=-1)
     out = torch.zeros_like(h)
     for t in range(h.shape[0]):
         for e, w in zip(ids[t].tolist(), weights[t]):
@@ -127,22 +136,26 @@ def routed_experts(mlp: dict, W: Dict[str, torch.Tensor], p: str, h):
 
 
 # ------------------------------------------------------------------------------------------------------------ the model
-def layer(cfg: dict, W: Dict[str, torch.Tensor], i: int, x):
+def layer(cfg: dict, W: Dict[str, torch.Tensor], i: int, x, forced: Optional[list] = None, regret_out: Optional[list] = None):
     lc, p, eps = cfg["layers"][i], f"l{i}", float(cfg["norm"]["eps"])
     x = x + rms_norm(parallel_mixer(lc["mixer"], W, f"{p}.mix", x, eps), W[f"{p}.norm1"], eps)
     mlp = lc.get("mlp")
     if mlp:
-        y = routed_experts(mlp, W, f"{p}.mlp", x) if mlp["kind"] == "moe" else dense_unit(W, f"{p}.mlp", x)
+        y = routed_experts(mlp, W, f"{p}.mlp", x, forced.pop(0) if forced else None, regret_out) if mlp["kind"] == "moe" else dense_unit(W, f"{p}.mlp", x)
         x = x + rms_norm(y, W[f"{p}.norm2"], eps)
     return x
 
 
-def forward(cfg: dict, tensors: Dict[str, torch.Tensor], tokens: List[int], dtype=torch.float64, streams: Optional[list] = None):
-    """Logits [T, vocab]; ``streams`` collects the residual after every layer."""
+def forward(cfg: dict, tensors: Dict[str, torch.Tensor], tokens: List[int], dtype=torch.float64, streams: Optional[list] = None,
+            forced: Optional[list] = None, regret_out: Optional[list] = None):
+    """Logits [T, vocab]; ``streams`` collects the residual after every layer. ``forced`` (a list over the layers with experts of ``[T, top]``):
+    the experts to take instead of the routers' own choice, what another implementation chose, so that the two can be compared where
+    a choice hung on rounding."""
     W = {k: v.to(dtype) for k, v in tensors.items()}
     x = embed(W, list(tokens))
+    forced = list(forced) if forced else None
     for i in range(len(cfg["layers"])):
-        x = layer(cfg, W, i, x)
+        x = layer(cfg, W, i, x, forced, regret_out)
         if streams is not None:
             streams.append(x.clone())
     return rms_norm(x, W["final.norm"], float(cfg["norm"]["eps"])) @ W["embed"].T

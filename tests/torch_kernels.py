@@ -187,6 +187,8 @@ class TorchKernels:
         z = x.float() @ w.float().T
         if activation == "gelu_erf":
             return (0.5 * z * (1.0 + torch.erf(z / math.sqrt(2.0)))).to(out_dtype or x.dtype)
+        if activation == "silu":
+            return (z * torch.sigmoid(z)).to(out_dtype or x.dtype)
         if activation == "relu2":
             return (z.clamp(min=0) ** 2).to(out_dtype or x.dtype)
         if activation != "gelu_tanh":
@@ -296,11 +298,16 @@ class TorchKernels:
         out = torch.cat([out, out.new_zeros(N, -out.shape[1] % 8)], dim=1)
         return out.to(out_dtype or z.dtype)
 
-    def linear_attention(self, z, q_col, k_col, v_col, num_heads, head_dim, v_head_dim, decay, state, batch):
+    def linear_attention_inputs(self, h, w_in, rows, head_dim, v_head_dim, batch, out_dtype):
+        z = self.linear(h, w_in, out_dtype=out_dtype)
+        return z, False, z, rows
+
+    def linear_attention(self, z, q_col, k_col, v_col, num_heads, head_dim, v_head_dim, decay, state, batch, activated=False):
         N = z.shape[0]
         H, D, DV = num_heads, head_dim, v_head_dim
         a = z.float()
-        a = a * torch.sigmoid(a)
+        if not activated:
+            a = a * torch.sigmoid(a)
         q, k, v = (a[:, c:c + H * n].view(N, H, n) for c, n in ((q_col, D), (k_col, D), (v_col, DV)))
         out = torch.zeros(N, H, DV)
         for slot, s0, s1 in self._requests(batch):
