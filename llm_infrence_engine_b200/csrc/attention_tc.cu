@@ -30,6 +30,13 @@
 // by their positions when they were cached: a row's outputs are turned back by the row's own position before they leave the
 // block (a slice's partial outputs too: the turn is linear and the same for all slices of a row).
 //
+// Extras (EXT), for mixers whose scores are more than a scaled product: chunks of positions, a soft cap, a bias by distance, a gate per
+// head on the outputs, and (SHARED) values that ARE the keys, with a number per cached token that multiplies its keys' scores. A row
+// thread turns its 64 scores into finished ones in units of log2 before the softmax step sees them. The bias of the nearest distances
+// lies in shared memory as a table [distance][head of the group], in which the 64 biases of a row stand at a fixed stride. With SHARED
+// a chunk of keys is fetched once and is the B operand of both products (as it lies, K-major for the scores, MN-major for P V); both
+// rings' space is one ring, and a stage is free when its P V product is over; the tokens' numbers come with the keys by a plain bulk copy.
+//
 // A launch follows a plan made once per step on the device (attn_tc_plan_kernel): which pieces of work there are (a tile,
 // or one slice of a long tile's keys, whose partial result the last slice merges), long pieces first.
 //
@@ -82,7 +89,26 @@ struct TcParams {
     const float* sig_bias;  // SIG: [nq]
     const float* log_r1;    // SIG: [nq] or null, with log_r2
     const float* log_r2;
+    // EXT:
+    int chunk;              // > 0: only keys of the row's own run of `chunk` positions are seen
+    float cap;              // > 0: scores are bounded by cap tanh(s / cap)
+    float x_scale;          // what a raw score is multiplied by: scale log2(e), or with a cap 2 scale log2(e) / cap
+    const float* rel;       // [rel_rows][nq] or null
+    const int* rows_of;     // [n_rows_of]
+    int n_rows_of, rel_rows;
+    int table;              // distances whose biases lie in shared memory
+    const bf16* gate;       // row n at gate + n * gate_stride: a number per head; or null
+    int gate_stride;
+    const float* key_scale; // SHARED: [pages][page_size]
 };
+
+enum { KIND_PLAIN = 0, KIND_SIG = 1, KIND_EXT = 2 };
+
+// `bytes` (a multiple of 16, both addresses on 16-byte boundaries) from global to shared memory, counted on `bar`
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, uint32_t bytes, uint64_t* bar) {
+    asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];\n" ::"r"(smem_u32(dst)), "l"(src), "r"(bytes),
+                 "r"(smem_u32(bar)) : "memory");
+}
 
 __device__ __forceinline__ float fast_exp2(float x) {
     float y;
@@ -141,21 +167,30 @@ __device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
     asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];\n" ::"r"(smem_u32(bar)) : "memory");
 }
 
-template <int D, bool SIG>
+// stages of the one ring where values are keys, and the bytes behind the ring(s) that the barriers may take
+template <int D> constexpr int SHARED_STAGES = D == 64 ? 6 : 4;
+constexpr int BARRIER_BYTES = 512;
+
+template <int D, int KIND, bool SHARED>
 __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __grid_constant__ CUtensorMap tmap_k,
                                                                                           const __grid_constant__ CUtensorMap tmap_v, const TcParams p) {
-    constexpr int ATOMS = Sizes<D>::ATOMS, STAGES = Sizes<D>::STAGES, Q_BYTES = Sizes<D>::Q_BYTES, K_BYTES = Sizes<D>::K_BYTES;
+    constexpr bool SIG = KIND == KIND_SIG, EXT = KIND == KIND_EXT;
+    static_assert(EXT || !SHARED, "values that are keys belong to the extras");
+    constexpr int ATOMS = Sizes<D>::ATOMS, STAGES = SHARED ? SHARED_STAGES<D> : Sizes<D>::STAGES, Q_BYTES = Sizes<D>::Q_BYTES, K_BYTES = Sizes<D>::K_BYTES;
     constexpr int TMEM_COLS = Sizes<D>::TMEM_COLS, S_BUFS = Sizes<D>::S_BUFS;
     extern __shared__ unsigned char raw[];
     unsigned char* base = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(raw) + 1023) & ~(uintptr_t)1023);
     unsigned char* q_s = base;
     unsigned char* k_s = base + Q_BYTES;           // [STAGES] key chunks
-    unsigned char* v_s = k_s + STAGES * K_BYTES;  // [STAGES] value chunks
+    unsigned char* v_s = SHARED ? k_s : k_s + STAGES * K_BYTES;  // [STAGES] value chunks, or the keys themselves
+    unsigned char* rings_end = v_s + STAGES * K_BYTES;
+    float* scale_s = reinterpret_cast<float*>(rings_end + BARRIER_BYTES);   // SHARED: [STAGES][BN] numbers of the chunks' tokens
+    float* bias_s = scale_s + (SHARED ? STAGES * BN : 0);                   // EXT: [table][G]
     // Keys and values have rings of their own: a key chunk is free again as soon as its scores are made, long before the
     // values of the same chunk have been used, so the next keys are on their way that much earlier.
-    uint64_t* k_full = reinterpret_cast<uint64_t*>(v_s + STAGES * K_BYTES);
+    uint64_t* k_full = reinterpret_cast<uint64_t*>(rings_end);
     uint64_t* k_empty = k_full + STAGES;
-    uint64_t* v_full = k_empty + STAGES;
+    uint64_t* v_full = k_empty + STAGES;   // (SHARED: the tokens' numbers)
     uint64_t* v_empty = v_full + STAGES;
     uint64_t* s_ready = v_empty + STAGES;  // [S_BUFS]
     uint64_t* p_ready = s_ready + S_BUFS;     // [2], taken in turn: the row threads may hand over P(c + 1) before the MMA thread has looked at P(c)'s barrier
@@ -198,6 +233,14 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
     const uint32_t tmem = *tmem_slot;
 
     pdl_trigger();
+    if constexpr (EXT) {   // weights of the model: fetched before the wait for the kernel before
+        if (p.rel) {
+            const int g_all = p.nq / p.nkv, n = p.table * g_all;
+#pragma unroll 4
+            for (int i = tid; i < n; i += THREADS) bias_s[i] = LOG2E * p.rel[(size_t)p.rows_of[i / g_all] * p.nq + kvh * g_all + i % g_all];
+        }
+        __syncthreads();
+    }
     pdl_wait();  // queries, keys, values and the step's tables all come from kernels before this one
 
     // everything about the piece comes in one trip to memory: the plan has looked up the tile, its position and its request
@@ -211,7 +254,8 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
     const int nrows = ntok * G;  // <= BM
     const int pos0 = ntok > 0 ? where.z : 0;
     const int hi = pos0 + ntok;  // one past the last visible key
-    const int lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+    int lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+    if (EXT && p.chunk > 0) lo = max(lo, pos0 / p.chunk * p.chunk);
     const int lo_al = lo / p.box_rows * p.box_rows;  // chunks start where a TMA box starts
     // this block's slice of the tile's chunks: [chunk0, chunk0 + chunks), empty for the later slices of a short tile
     const int all_chunks = ntok > 0 ? (hi - lo_al + BN - 1) / BN : 0;
@@ -248,7 +292,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 rows_now = rows_next;
                 rows_next = group_rows((c >> group_shift) + 1);
             }
-            const bool keys = c < chunks, values = c > 0;
+            const bool keys = c < chunks, values = !SHARED && c > 0;
             const int kst = c % STAGES, vst = (c + STAGES - 1) % STAGES;  // stage of chunk c, of chunk c - 1
             const int row_k = __shfl_sync(0xffffffffu, rows_now, (((c & (group - 1)) << box_shift) + my_box) & 31);
             const int cv = c > 0 ? c - 1 : 0;
@@ -259,6 +303,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 if (keys && c >= STAGES) ok = mbar_wait(k_empty + kst, ((c / STAGES) & 1) ^ 1, abort_flag, p.error_flag, 11);
                 if (ok && values && c - 1 >= STAGES) ok = mbar_wait(v_empty + vst, (((c - 1) / STAGES) & 1) ^ 1, abort_flag, p.error_flag, 11);
                 if (ok && keys) mbar_expect_tx(k_full + kst, K_BYTES);
+                if (SHARED && ok && keys) mbar_expect_tx(v_full + kst, BN * 4);
                 if (ok && values) mbar_expect_tx(v_full + vst, K_BYTES);
             }
             ok = __shfl_sync(0xffffffffu, (int)ok, 0) != 0;
@@ -267,11 +312,16 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
             const int atom = (lane >> box_shift) % ATOMS;
             if (lane < boxes * ATOMS) {
                 if (keys) tma_load_2d(k_s + kst * K_BYTES + atom * (BN * 128) + my_box * p.box_rows * 128, &tmap_k, atom * 64, row_k, k_full + kst);
+            } else if (SHARED) {
+                if (keys && lane < boxes * (ATOMS + 1)) {
+                    const int page = row_k / (p.nkv * p.page_size);
+                    bulk_load(scale_s + kst * BN + my_box * p.box_rows, p.key_scale + (size_t)page * p.page_size + row_k % p.page_size, p.box_rows * 4, v_full + kst);
+                }
             } else if (lane < 2 * boxes * ATOMS) {
                 if (values) tma_load_2d(v_s + vst * K_BYTES + atom * (BN * 128) + my_box * p.box_rows * 128, &tmap_v, atom * 64, row_v, v_full + vst);
             }
             __syncwarp();
-            if (lane == 0) { if (keys) issued[0] = c + 1; if (values) issued[1] = c; }
+            if (lane == 0) { if (keys) issued[0] = c + 1; if (SHARED && keys) issued[1] = c + 1; if (values) issued[1] = c; }
         }
     } else if (warp == 5) {
         // ---------------------------------------------------------------- MMA issuer
@@ -286,7 +336,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                     umma_bf16(tmem + (c % S_BUFS) * BN, umma_desc(smem_u32(q_s) + (k / 4) * (BM * 128)) + 2 * (k % 4),
                               umma_desc(k_addr + (k / 4) * (BN * 128)) + 2 * (k % 4), idesc_s, k > 0 ? 1u : 0u);
                 umma_commit(s_ready + c % S_BUFS);
-                umma_commit(k_empty + c % STAGES);
+                if (!SHARED) umma_commit(k_empty + c % STAGES);
             };
             // Scores are made as early as their keys and a buffer allow: S(n) goes into the buffer in which P(n - S_BUFS) took the
             // place of S(n - S_BUFS); the product that reads that P was issued by this thread before, and a thread's MMAs run in
@@ -323,7 +373,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 bool p_there = false;
                 for (uint32_t i = 0; i < SPIN_LIMIT && !p_there; ++i) {
                     more_scores(c + S_BUFS - 1, false);
-                    p_there = mbar_try_wait(p_ready + (c & 1), (c >> 1) & 1) && mbar_try_wait(v_full + c % STAGES, (c / STAGES) & 1);
+                    p_there = mbar_try_wait(p_ready + (c & 1), (c >> 1) & 1) && (SHARED || mbar_try_wait(v_full + c % STAGES, (c / STAGES) & 1));
                     if (*abort_flag) break;
                     if (!p_there && i > 64) __nanosleep(40);
                 }
@@ -341,7 +391,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 }
                 umma_commit(o_ready);
                 if (c == chunks - 1) umma_commit(o_done);
-                umma_commit(v_empty + c % STAGES);
+                umma_commit((SHARED ? k_empty : v_empty) + c % STAGES);
             }
         }
     } else {
@@ -374,6 +424,9 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
             ref = 0.f;
             l = split == 0 ? 1.f : 0.f;   // (what the outputs are divided by in the end: one)
         }
+        const float to_log2 = EXT ? 1.f : p.scale_log2;   // from the scores to units of log2 (EXT: they are)
+        const int my_head = kvh * G + (row_ok ? row % G : 0);
+        const float rel_last = (EXT && p.rel) ? LOG2E * p.rel[(size_t)(p.rel_rows - 1) * p.nq + my_head] : 0.f;
         const uint32_t lane_base = tmem + ((uint32_t)(warp * 32) << 16);
         const uint32_t o_addr = lane_base + S_BUFS * BN;
         // the scores of chunk c are waited for during chunk c - 1 (see below): only the first ones here
@@ -392,7 +445,72 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
             const int key0 = lo_al + (chunk0 + c) * BN;
             // A chunk that every row of the tile sees in full needs no mask arithmetic (rows beyond the tile have zero
             // queries and collect numbers nobody reads). The scale is positive: the maximum is taken over the raw scores.
-            const bool interior = key0 >= lo && key0 + BN - 1 <= pos0 && (p.window <= 0 || key0 > hi - 1 - p.window);
+            bool interior = key0 >= lo && key0 + BN - 1 <= pos0 && (p.window <= 0 || key0 > hi - 1 - p.window);
+            if (EXT && p.chunk > 0) interior = interior && (hi - 1) / p.chunk * p.chunk <= key0;
+            if constexpr (EXT) {
+                // the row's 64 finished scores in units of log2: times the token's number, scaled, capped, biased by distance. (Columns the
+                // row does not see come out as anything; they are replaced below.)
+                if (SHARED) {
+                    ok = __all_sync(0xffffffffu, mbar_wait(v_full + c % STAGES, (c / STAGES) & 1, abort_flag, p.error_flag, 18));
+                    if (!ok) break;
+                }
+                const float* ks = scale_s + (c % STAGES) * BN;
+                const int nearest = pos0 - (key0 + BN - 1), farthest = hi - 1 - key0;   // distances of the tile's rows to the chunk's keys
+                const bool in_table = p.rel && farthest < p.table, all_far = p.rel && nearest >= p.n_rows_of;
+                const float add = (p.cap > 0.f ? p.cap * LOG2E : 0.f) + (all_far ? rel_last : 0.f);
+                const uint64_t zero2 = pair_of(0.f, 0.f), x2 = pair_of(p.x_scale, p.x_scale), add2_ = pair_of(add, add);
+                if (p.cap > 0.f) {
+                    // cap tanh(v) = cap - 2 cap / (e^(2 v) + 1), two of them per division; e^(2 v) is bounded so that the product stays finite
+                    const float m2cap = -2.f * LOG2E * p.cap;
+                    const uint64_t one2 = pair_of(1.f, 1.f), m2cap2 = pair_of(m2cap, m2cap);
+#pragma unroll
+                    for (int j = 0; j < BN; j += 4) {
+                        float kk[4] = {1.f, 1.f, 1.f, 1.f};
+                        if (SHARED) load4(ks + j, kk);
+#pragma unroll
+                        for (int i = 0; i < 4; i += 2) {
+                            float a, b, t0, t1;
+                            uint64_t v = pair_of(__uint_as_float(s[j + i]), __uint_as_float(s[j + i + 1]));
+                            if (SHARED) v = fma2(v, pair_of(kk[i], kk[i + 1]), zero2);
+                            unpair(fma2(v, x2, zero2), a, b);
+                            unpair(add2(pair_of(fast_exp2(fminf(a, 60.f)), fast_exp2(fminf(b, 60.f))), one2), t0, t1);
+                            const float r = __fdividef(1.0f, t0 * t1);
+                            unpair(fma2(pair_of(r * t1, r * t0), m2cap2, add2_), a, b);
+                            s[j + i] = __float_as_uint(a);
+                            s[j + i + 1] = __float_as_uint(b);
+                        }
+                    }
+                } else {
+#pragma unroll
+                    for (int j = 0; j < BN; j += 4) {
+                        float kk[4] = {1.f, 1.f, 1.f, 1.f};
+                        if (SHARED) load4(ks + j, kk);
+#pragma unroll
+                        for (int i = 0; i < 4; i += 2) {
+                            float a, b;
+                            uint64_t v = pair_of(__uint_as_float(s[j + i]), __uint_as_float(s[j + i + 1]));
+                            if (SHARED) v = fma2(v, pair_of(kk[i], kk[i + 1]), zero2);
+                            unpair(fma2(v, x2, add2_), a, b);
+                            s[j + i] = __float_as_uint(a);
+                            s[j + i + 1] = __float_as_uint(b);
+                        }
+                    }
+                }
+                if (in_table) {
+                    // entry (distance, head of the group) of this row and key j: (pos - key0 - j) G + row % G = (pos0 - key0) G + row - j G.
+                    // (A key behind the row's position reads what lies before the table in shared memory: the ring; see above.)
+                    const float* tb = bias_s + (pos0 - key0) * G + (row_ok ? row : 0);
+#pragma unroll
+                    for (int j = 0; j < BN; ++j) s[j] = __float_as_uint(__uint_as_float(s[j]) + tb[-j * G]);
+                } else if (p.rel && !all_far) {
+#pragma unroll
+                    for (int j = 0; j < BN; ++j) {
+                        const int dist = max(pos - key0 - j, 0);
+                        const int br = dist < p.n_rows_of ? p.rows_of[dist] : p.rel_rows - 1;
+                        s[j] = __float_as_uint(fmaf(LOG2E, p.rel[(size_t)br * p.nq + my_head], __uint_as_float(s[j])));
+                    }
+                }
+            }
             uint32_t keep_lo = 0xffffffffu, keep_hi = 0xffffffffu;
             if (__builtin_expect(!interior, 0)) {
                 // The columns this row sees are a run [first, last] of the chunk's 64: two words of bits say which, and a
@@ -400,7 +518,8 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 // instructions a column) and marked unlikely: this code sits in the middle of the loop that every chunk runs,
                 // and what the loop's instructions occupy of the instruction cache shows in its time.
                 const int last = row_ok ? min(pos - key0, BN - 1) : -1;
-                const int first = p.window > 0 ? max(pos - p.window + 1 - key0, 0) : 0;
+                int first = p.window > 0 ? max(pos - p.window + 1 - key0, 0) : 0;
+                if (EXT && p.chunk > 0) first = max(first, pos / p.chunk * p.chunk - key0);
                 const uint64_t upto = last < 0 ? 0ull : (last >= 63 ? ~0ull : ((1ull << (last + 1)) - 1ull));
                 const uint64_t seen = first >= 64 ? 0ull : upto & ~((1ull << first) - 1ull);
                 const uint32_t seen_lo = (uint32_t)seen, seen_hi = (uint32_t)(seen >> 32);
@@ -449,7 +568,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 for (int k = 0; k < 4; ++k) mx4[k] = max3(mx4[k], __uint_as_float(s[j + k]), __uint_as_float(s[j + 4 + k]));
             }
             const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-            m = fmaxf(m, mx * p.scale_log2);
+            m = fmaxf(m, mx * to_log2);
             // The reference follows the maximum only when it lags too far behind: then this row of O and the row's sum are
             // scaled down. The first keys a row sees set its reference for free (everything so far was zero).
             bool rescale = false;
@@ -489,7 +608,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
             }
             // all 64 exponentials first, in place and independent of each other (the special-function unit is the narrow
             // place of this loop and must not wait for the sums and stores that follow)
-            const uint64_t scale2 = pair_of(p.scale_log2, p.scale_log2), shift2 = pair_of(-use, -use);
+            const uint64_t scale2 = pair_of(to_log2, to_log2), shift2 = pair_of(-use, -use);
 #pragma unroll
             for (int j = 0; j < BN; j += 2) {
                 float x0, x1;
@@ -528,8 +647,10 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 // the chunk reaches behind the last key: those value rows may hold anything; they become zeros
                 unsigned char* v_c = v_s + (c % STAGES) * K_BYTES;
                 const int first_bad = hi - key0;
-                ok = __all_sync(0xffffffffu, mbar_wait(v_full + c % STAGES, (c / STAGES) & 1, abort_flag, p.error_flag, 18));  // the values have landed
-                if (!ok) break;
+                if (!SHARED) {   // (keys that are values have landed: their scores are made)
+                    ok = __all_sync(0xffffffffu, mbar_wait(v_full + c % STAGES, (c / STAGES) & 1, abort_flag, p.error_flag, 18));  // the values have landed
+                    if (!ok) break;
+                }
                 for (int i = tid; i < (BN - first_bad) * 8 * ATOMS; i += BM) {
                     const int in_block = i % ((BN - first_bad) * 8);  // which 16 bytes of the bad rows of a block of 64 dims
                     *reinterpret_cast<uint4*>(v_c + (i / ((BN - first_bad) * 8)) * (BN * 128) + (first_bad + (in_block >> 3)) * 128 + ((in_block & 7) << 4)) =
@@ -563,7 +684,10 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
             fm[row] = ref;  // what the sum and the outputs are relative to
             fl[row] = l;
         }
-        const float inv = l > 0.f ? 1.f / l : 0.f;
+        float inv = l > 0.f ? 1.f / l : 0.f;
+        float gate = 1.f;   // on the outputs of a slice as on those of the whole: the merge is linear in them
+        if (EXT && p.gate && row_ok) gate = 1.f / (1.f + __expf(-to_f32(p.gate[(size_t)(n0 + tok) * p.gate_stride + my_head])));
+        inv *= gate;
 #pragma unroll 1
         for (int part = 0; part < D / 2 && ok; part += 32) {   // 32 entries of either half: both partners of every pair that may turn
             float o[64];
@@ -607,7 +731,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 }
             } else {
 #pragma unroll
-                for (int i = 0; i < 64; i += 4) *reinterpret_cast<float4*>(fo + row * D + (i < 32 ? part + i : D / 2 + part + i - 32)) = make_float4(o[i], o[i + 1], o[i + 2], o[i + 3]);
+                for (int i = 0; i < 64; i += 4) *reinterpret_cast<float4*>(fo + row * D + (i < 32 ? part + i : D / 2 + part + i - 32)) = make_float4(o[i] * gate, o[i + 1] * gate, o[i + 2] * gate, o[i + 3] * gate);
             }
         }
     }
@@ -649,7 +773,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
 constexpr int MIN_SLICE = 8, SLICE_COST = 8, MAX_SLICES = 16, PLAN_THREADS = 256;
 
 __global__ void __launch_bounds__(PLAN_THREADS) attn_tc_plan_kernel(const int* __restrict__ tile_info, int num_tiles, const int* __restrict__ positions,
-                                                                    const int* __restrict__ token_seq, int window, int box_rows, int capacity, int fixed_splits, int max_items,
+                                                                    const int* __restrict__ token_seq, int window, int chunk, int box_rows, int capacity, int fixed_splits, int max_items,
                                                                     int* __restrict__ work, int* __restrict__ tmp) {
     pdl_trigger();
     pdl_wait();
@@ -665,7 +789,8 @@ __global__ void __launch_bounds__(PLAN_THREADS) attn_tc_plan_kernel(const int* _
         int c = 0;
         if (ntok > 0) {
             const int pos0 = positions[n0], hi = pos0 + ntok;
-            const int lo = window > 0 ? max(0, pos0 - window + 1) : 0;
+            int lo = window > 0 ? max(0, pos0 - window + 1) : 0;
+            if (chunk > 0) lo = max(lo, pos0 / chunk * chunk);
             c = (hi - lo / box_rows * box_rows + BN - 1) / BN;
         }
         chunks[t] = c;
@@ -738,13 +863,13 @@ __global__ void __launch_bounds__(PLAN_THREADS) attn_tc_plan_kernel(const int* _
 
 // The plan for llmie_paged_attention_tc (see attn_tc_plan_kernel): work [8 * max_items + 1] receives the pieces and their number,
 // tmp [3 * num_tiles] is scratch. capacity: pieces that can run at once. max_items >= num_tiles * max(1, fixed_splits).
-LLMIE_API int llmie_attn_tc_plan(const int* tile_info, int num_tiles, const int* positions, const int* token_seq, int window, int page_size,
+LLMIE_API int llmie_attn_tc_plan(const int* tile_info, int num_tiles, const int* positions, const int* token_seq, int window, int chunk, int page_size,
                                  int capacity, int fixed_splits, int max_items, int* work, int* tmp, cudaStream_t s) {
     if (num_tiles <= 0) return 0;
     if (!tile_info || !positions || !token_seq || !work || !tmp || page_size <= 0 || capacity <= 0 || fixed_splits < 0 || fixed_splits > MAX_SLICES ||
         max_items < (long long)num_tiles * (fixed_splits > 0 ? fixed_splits : 1) || ((uintptr_t)work & 15))
         return LLMIE_ERR_BAD_ARGUMENT;
-    return launch_kernel(attn_tc_plan_kernel, dim3(1), dim3(PLAN_THREADS), 0, s, tile_info, num_tiles, positions, token_seq, window,
+    return launch_kernel(attn_tc_plan_kernel, dim3(1), dim3(PLAN_THREADS), 0, s, tile_info, num_tiles, positions, token_seq, window, chunk,
                          page_size < BN ? page_size : BN, capacity, fixed_splits, max_items, work, tmp);
 }
 
@@ -758,8 +883,13 @@ LLMIE_API int llmie_paged_attention_tc(const bf16* q, int q_stride, const bf16* 
                                        const int* block_table, int max_blocks, int num_tiles, const int* work, int max_items, bf16* out, float* scratch_o,
                                        float* scratch_ml, int* counters, int nq, int nkv, int d, int page_size, float scale, int window,
                                        int* error_flag, const float* turn_cos, const float* turn_sin, const float* sig_bias, const float* log_r1,
-                                       const float* log_r2, cudaStream_t s) {
+                                       const float* log_r2, int chunk, float softcap, const float* rel, const int* rows_of, int n_rows_of, int rel_rows,
+                                       const bf16* gate, int gate_stride, const float* key_scale, cudaStream_t s) {
     if (num_tiles <= 0) return 0;
+    const bool ext = chunk > 0 || softcap > 0.f || rel || gate || key_scale;
+    if ((ext && (sig_bias || turn_cos)) || (rel && (!rows_of || rel_rows < 1 || n_rows_of < 0)) || (v_pool == nullptr) != (key_scale != nullptr) ||
+        ((uintptr_t)key_scale & 15) || (!ext && !(scale > 0.f)))
+        return LLMIE_ERR_BAD_ARGUMENT;
     if ((turn_cos == nullptr) != (turn_sin == nullptr) || ((uintptr_t)turn_cos & 15) || ((uintptr_t)turn_sin & 15) || (log_r1 == nullptr) != (log_r2 == nullptr) ||
         (log_r1 && !sig_bias))
         return LLMIE_ERR_BAD_ARGUMENT;
@@ -774,23 +904,41 @@ LLMIE_API int llmie_paged_attention_tc(const bf16* q, int q_stride, const bf16* 
     p.q_stride = q_stride; p.max_blocks = max_blocks; p.nq = nq; p.nkv = nkv; p.page_size = page_size; p.num_tiles = num_tiles;
     p.window = window; p.box_rows = page_size < BN ? page_size : BN; p.scale_log2 = scale * LOG2E;
     p.turn_cos = turn_cos; p.turn_sin = turn_sin; p.sig_bias = sig_bias; p.log_r1 = log_r1; p.log_r2 = log_r2;
+    p.chunk = chunk; p.cap = softcap; p.x_scale = softcap > 0.f ? 2.f * LOG2E * scale / softcap : LOG2E * scale;
+    p.rel = rel; p.rows_of = rows_of; p.n_rows_of = n_rows_of; p.rel_rows = rel_rows; p.table = 0;
+    p.gate = gate; p.gate_stride = gate_stride; p.key_scale = key_scale;
     CUtensorMap mk, mv;
     const int rows = (int)(pool_pages * nkv * page_size);
     int rc = tensor_map(k_pool, rows, d, p.box_rows, &mk);
     if (rc) return rc;
-    rc = tensor_map(v_pool, rows, d, p.box_rows, &mv);
+    rc = tensor_map(v_pool ? v_pool : k_pool, rows, d, p.box_rows, &mv);
     if (rc) return rc;
     const long long blocks = (long long)max_items * nkv;
     if (blocks > 0x7fffffffLL) return LLMIE_ERR_BAD_ARGUMENT;
-    static bool set[4] = {false, false, false, false};
+    static size_t set[8] = {};
     auto launch = [&](auto kernel, size_t smem, int which) -> int {
-        if (!set[which]) {
+        if (smem > set[which]) {
             cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             if (e != cudaSuccess) return (int)e;
-            set[which] = true;
+            set[which] = smem;
         }
         return launch_kernel(kernel, dim3((unsigned)blocks), dim3(THREADS), smem, s, mk, mv, p);
     };
-    if (sig_bias) return d == 64 ? launch(attn_tc_prefill_kernel<64, true>, Sizes<64>::SMEM, 2) : launch(attn_tc_prefill_kernel<128, true>, Sizes<128>::SMEM, 3);
-    return d == 64 ? launch(attn_tc_prefill_kernel<64, false>, Sizes<64>::SMEM, 0) : launch(attn_tc_prefill_kernel<128, false>, Sizes<128>::SMEM, 1);
+    if (ext) {
+        // as many of the nearest distances' biases as leave two blocks to a multiprocessor
+        const int G = nq / nkv, k_bytes = BN * d * 2;
+        const int stages = key_scale ? (d == 64 ? SHARED_STAGES<64> : SHARED_STAGES<128>) : 2 * (d == 64 ? Sizes<64>::STAGES : Sizes<128>::STAGES);
+        size_t smem = (size_t)BM * d * 2 + (size_t)stages * k_bytes + 1024 + BARRIER_BYTES + (key_scale ? (size_t)stages * BN * 4 : 0);
+        if (rel) {
+            const long long room = ((long long)113 * 1024 - (long long)smem) / (4 * G);
+            p.table = (int)(room < n_rows_of ? (room > 0 ? room : 0) : n_rows_of);
+            smem += (size_t)p.table * G * 4;
+        }
+        if (key_scale)
+            return d == 64 ? launch(attn_tc_prefill_kernel<64, KIND_EXT, true>, smem, 4) : launch(attn_tc_prefill_kernel<128, KIND_EXT, true>, smem, 5);
+        return d == 64 ? launch(attn_tc_prefill_kernel<64, KIND_EXT, false>, smem, 6) : launch(attn_tc_prefill_kernel<128, KIND_EXT, false>, smem, 7);
+    }
+    if (sig_bias)
+        return d == 64 ? launch(attn_tc_prefill_kernel<64, KIND_SIG, false>, Sizes<64>::SMEM, 2) : launch(attn_tc_prefill_kernel<128, KIND_SIG, false>, Sizes<128>::SMEM, 3);
+    return d == 64 ? launch(attn_tc_prefill_kernel<64, KIND_PLAIN, false>, Sizes<64>::SMEM, 0) : launch(attn_tc_prefill_kernel<128, KIND_PLAIN, false>, Sizes<128>::SMEM, 1);
 }

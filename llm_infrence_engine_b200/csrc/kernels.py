@@ -55,6 +55,7 @@ class CudaKernels:
         self.sample_single_block = False   # sampling by one block per row instead of a cluster per row (the slower, older kernel)
         self.use_tc_attention = True   # prompt portions of head size 64 or 128: scores and outputs through tcgen05 and tensor memory
         self.cluster_merge = True      # decode attention: the key slices of a token form a cluster and merge in shared memory
+        self.use_tc_attention_ext = True   # ... also with chunks, a soft cap, a bias by distance, a gate per head, keys that are values
         self.use_tc_gemm = True
         self.use_cluster_gate_up = False  # ... by pairs of blocks that share their weight rows (TMA multicast within a cluster of two)
         self.use_pair_gate_up = True     # ... by pairs of multiprocessors on tiles of 256 rows (tcgen05 cta_group::2) ...
@@ -675,9 +676,10 @@ class CudaKernels:
         return tiles, batch._tables[key]
 
     def _attention_tc(self, qkv, k_pool, v_pool, block_table, token_seq, positions, out, num_heads, num_kv_heads, head_dim,
-                      page_size, scale, window, span, batch, num_splits, turn=None, sigmoid_bias=None, log_distance=None):
-        """The tcgen05 kernel for prompt portions, if it takes this case: returns ``out`` or None. (``turn``, ``sigmoid_bias``,
-        ``log_distance``: see ``attention_ext``.)"""
+                      page_size, scale, window, span, batch, num_splits, turn=None, sigmoid_bias=None, log_distance=None, chunk=0, softcap=0.0,
+                      rel=None, rel_rows=None, gate=None, gate_col=0, key_scale=None):
+        """The tcgen05 kernel for prompt portions, if it takes this case: returns ``out`` or None. (The extras: see ``attention_ext``; the
+        gate is one per head.)"""
         group = num_heads // num_kv_heads
         if not (self.use_tc_attention and head_dim in (64, 128) and batch.max_seq_len > 1 and group <= 128 and page_size % 8 == 0
                 and (64 % page_size == 0 or page_size % 64 == 0) and (num_splits is None or 1 <= num_splits <= 16)):
@@ -692,11 +694,11 @@ class CudaKernels:
         capacity = max(1, 2 * self.num_sms // num_kv_heads)   # two blocks per SM
         # (tiles of up to 16 chunks are never cut: a slice costs about 8 chunks' time and is at least 8 chunks long)
         max_items = tiles * fixed if fixed else max(tiles, min(capacity, 16 * tiles)) if span > 16 * 64 else tiles
-        key = ("tcgen05 attention plan", group, num_kv_heads, page_size, int(window), fixed)
+        key = ("tcgen05 attention plan", group, num_kv_heads, page_size, int(window), int(chunk), fixed)
         if key not in batch._tables:
             work = torch.empty((8 * max_items + 4,), dtype=torch.int32, device=qkv.device)
             tmp = torch.empty((3 * tiles,), dtype=torch.int32, device=qkv.device)
-            self._check(self.lib.llmie_attn_tc_plan(_ptr(tile_info), tiles, _ptr(positions), _ptr(token_seq), int(window), page_size, capacity, fixed,
+            self._check(self.lib.llmie_attn_tc_plan(_ptr(tile_info), tiles, _ptr(positions), _ptr(token_seq), int(window), int(chunk), page_size, capacity, fixed,
                                                     max_items, _ptr(work), _ptr(tmp), self._stream()), "attention plan (tcgen05)")
             batch._tables[key] = (work, tmp)
         work = batch._tables[key][0]
@@ -710,6 +712,8 @@ class CudaKernels:
             block_table.shape[1], tiles, _ptr(work), max_items, _ptr(out),
             _ptr(scratch_o), _ptr(scratch_ml), _ptr(self._attn_counters), num_heads, num_kv_heads, head_dim, page_size,
             ctypes.c_float(scale), int(window), _ptr(self._errors(qkv.device)), *self._turn_and_sigmoid(turn, sigmoid_bias, log_distance),
+            int(chunk), ctypes.c_float(softcap), _ptr(rel), _ptr(rel_rows), 0 if rel_rows is None else rel_rows.shape[0], 0 if rel is None else rel.shape[0],
+            ctypes.c_void_p(0 if gate is None else gate.data_ptr() + gate_col * gate.element_size()), 0 if gate is None else gate.shape[1], _ptr(key_scale),
             self._stream()), "paged_attention (tcgen05)")
         return out
 
@@ -1154,6 +1158,15 @@ class CudaKernels:
                 and num_heads // num_kv_heads <= (16 if batch.max_seq_len == 1 else 64) and (num_splits is None or num_splits <= 16)):
             done = self._attention_mma(q, k_pool, v_pool, block_table, token_seq, positions, out, num_heads, num_kv_heads, head_dim, page_size, scale,
                                        int(window), min(max_context, window) if window else max_context, batch, num_splits, turn, sigmoid_bias, log_distance)
+            if done is not None:
+                return done
+        if (self.use_tc_attention_ext and dt == 1 and batch is not None and batch.max_seq_len > 1 and head_dim == v_head_dim and q_col == 0 and q.shape[1] % 8 == 0
+                and not (keep_first or temp[1]) and sink is None and gate_mode != 2 and log_distance is None and sigmoid_bias is None and turn is None
+                and (v_pool is None) == (key_scale is not None)):
+            span = min(max_context, window or max_context, chunk or max_context)
+            done = self._attention_tc(q, k_pool, v_pool, block_table, token_seq, positions, out, num_heads, num_kv_heads, head_dim, page_size, scale,
+                                      int(window), span, batch, num_splits, chunk=chunk, softcap=softcap, rel=rel, rel_rows=rel_rows, gate=gate, gate_col=gate_col,
+                                      key_scale=key_scale)
             if done is not None:
                 return done
         max_rows = 0

@@ -236,11 +236,11 @@ def run_attention(K, how, q, q_col, common, seq, pos, page, scale, window, ctx_l
     if "five runs" in how:
         more = {"num_splits": 5}
     K.use_fa_attention_ext = not how.endswith("split-part kernel")
-    K.use_plain_attention_for_ext = not how.endswith("kernel")
+    K.use_plain_attention_for_ext = K.use_tc_attention_ext = not how.endswith("kernel")
     try:
         return K.attention_ext(q.cuda(), q_col, *common, seq.cuda(), pos.cuda(), page, scale, window, ctx_len, batch=batch, **kw, **more)
     finally:
-        K.use_fa_attention_ext = K.use_plain_attention_for_ext = True
+        K.use_fa_attention_ext = K.use_plain_attention_for_ext = K.use_tc_attention_ext = True
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
