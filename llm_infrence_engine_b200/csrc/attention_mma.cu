@@ -61,6 +61,31 @@ struct Params {
     const float* log_r2 = nullptr;
     const float* turn_cos = nullptr;
     const float* turn_sin = nullptr;
+    // Decode steps, EXT (see ExtTerms): chunks of positions, a soft cap, a bias by distance, a gate per head, keys that are values
+    int chunk = 0;                     // > 0: only keys of the token's own run of `chunk` positions are seen
+    float cap_log2 = 0.f;              // > 0: the soft cap times log2(e)
+    float x_scale = 0.f;               // what a raw score is multiplied by: scale log2(e), or with a cap 2 scale log2(e) / cap
+    const float* rel = nullptr;        // [rel_rows][nq] or null
+    const int* rows_of = nullptr;      // [n_rows_of]
+    int n_rows_of = 0, rel_rows = 0;
+    const bf16* gate = nullptr;        // row n at gate + n * gate_stride: a number per head; or null
+    int gate_stride = 0;
+    const float* key_scale = nullptr;  // [pages][page_size]: a number per cached token, on its scores (v_pool is then unused)
+};
+
+// A chunk's terms of the scores of the transposed form: per lane the biases (in units of log2) of its keys kt * 16 + lane / 4 (+ 8) for its
+// rows 2 (lane % 4) + j, and where the chunk's numbers per token lie in shared memory. With them a raw score becomes, in units of log2,
+//   x_scale (s n) + b, or, with a cap, cap_log2 tanh(..) + b by tanh(v) = 1 - 2 / (e^(2 v) + 1).
+template <int BN>
+struct ExtTerms {
+    float b[BN / 16][4];
+    const float* numbers;   // [BN] or null
+    float x_scale, cap_log2;
+    __device__ __forceinline__ float score(int kt, int e, float s, float number) const {
+        const float v = s * number * x_scale;
+        if (cap_log2 > 0.f) return fmaf(-2.f * cap_log2, __fdividef(1.0f, hw_exp2(fminf(v, 60.f)) + 1.0f), cap_log2) + b[kt][e];
+        return v + b[kt][e];
+    }
 };
 
 // A lane's two rows' terms of sigmoid weights: the weight of a key at distance d is 1 / (1 + 2^x), x = b - scale_log2 s + r1 log2(1 + r2 d).
@@ -80,6 +105,10 @@ struct SigRows {
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
     const uint32_t s = (uint32_t)__cvta_generic_to_shared(smem);
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(s), "l"(gmem));
+}
+__device__ __forceinline__ void cp_async4(void* smem, const void* gmem) {
+    const uint32_t s = (uint32_t)__cvta_generic_to_shared(smem);
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(s), "l"(gmem));
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::); }
 template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
@@ -148,9 +177,9 @@ __device__ __forceinline__ PoolRows<NKEYS> find_rows_warp(const Params& p, const
 }
 
 // Second half: the row numbers travel by shuffle to the lanes that copy that row's 16-byte pieces, 8 (or 16) neighbouring
-// lanes per row, into the swizzled K tile and V tile.
-template <int D, int NKEYS>
-__device__ __forceinline__ void copy_rows_warp(const Params& p, const PoolRows<NKEYS>& rows, int tile_row0, bf16* ks, bf16* vs, int lane) {
+// lanes per row, into the swizzled K tile and V tile. SHARED: keys are values: no V tile, but the tokens' numbers to `numbers`.
+template <int D, int NKEYS, bool SHARED = false>
+__device__ __forceinline__ void copy_rows_warp(const Params& p, const PoolRows<NKEYS>& rows, int tile_row0, bf16* ks, bf16* vs, int lane, float* numbers = nullptr) {
     constexpr int CH = D / 8, KPI = 32 / CH;
     const int ch = lane % CH, sub = lane / CH;
 #pragma unroll
@@ -161,14 +190,20 @@ __device__ __forceinline__ void copy_rows_warp(const Params& p, const PoolRows<N
         const int dst = trow * D + ((ch ^ (trow & 7)) << 3);
         const size_t src = (size_t)r * D + ch * 8;
         cp_async16(ks + dst, p.k_pool + src);
-        cp_async16(vs + dst, p.v_pool + src);
+        if (!SHARED) cp_async16(vs + dst, p.v_pool + src);
+    }
+    if constexpr (SHARED) {
+        static_assert(NKEYS <= 32, "one number per lane");
+        const int r = rows.idx[0];                       // (page * nkv + kvh) * page_size + offset
+        const int page = r / (p.nkv * p.page_size);
+        if (lane < NKEYS) cp_async4(numbers + tile_row0 + lane, p.key_scale + (size_t)page * p.page_size + r % p.page_size);
     }
 }
 
-template <int D, int NKEYS>
+template <int D, int NKEYS, bool SHARED = false>
 __device__ __forceinline__ void load_rows_warp(const Params& p, const int* table, int kvh, int key_abs0, int last_key, int tile_row0,
-                                               bf16* ks, bf16* vs, int lane) {
-    copy_rows_warp<D, NKEYS>(p, find_rows_warp<NKEYS>(p, table, kvh, key_abs0, last_key, lane), tile_row0, ks, vs, lane);
+                                               bf16* ks, bf16* vs, int lane, float* numbers = nullptr) {
+    copy_rows_warp<D, NKEYS, SHARED>(p, find_rows_warp<NKEYS>(p, table, kvh, key_abs0, last_key, lane), tile_row0, ks, vs, lane, numbers);
 }
 
 // One chunk of BN keys for one warp's 16 rows: S = Q K^T, masked online softmax, O += P V.
@@ -275,10 +310,10 @@ __device__ __forceinline__ uint32_t transpose_8x8(uint32_t a) {
     return d;
 }
 
-template <int D, int BN, bool MASKED, bool SIG = false>
+template <int D, int BN, bool MASKED, bool SIG = false, bool EXT = false>
 __device__ __forceinline__ void attend_chunk_t8(const uint32_t (&qb)[D / 16][2], const bf16* ks, const bf16* vs, float (&ot)[D / 16][4],
                                                 float (&m)[2], float (&l)[2], int key0, int pos, int nrows, int window, float scale_log2,
-                                                int lane, const SigRows* sig = nullptr) {
+                                                int lane, const SigRows* sig = nullptr, const ExtTerms<BN>* ext = nullptr) {
     float st[BN / 16][4];
 #pragma unroll
     for (int kt = 0; kt < BN / 16; ++kt) {
@@ -315,7 +350,9 @@ __device__ __forceinline__ void attend_chunk_t8(const uint32_t (&qb)[D / 16][2],
         for (int e = 0; e < 4; ++e) {
             const int key = key0 + kt * 16 + (lane >> 2) + ((e >> 1) << 3);
             const bool ok = !MASKED || (((lane & 3) << 1) + (e & 1) < nrows && key <= pos && (window <= 0 || key > pos - window));
-            const float x = ok ? st[kt][e] * scale_log2 : -INFINITY;
+            float x = st[kt][e] * scale_log2;
+            if constexpr (EXT) x = ext->score(kt, e, st[kt][e], ext->numbers ? ext->numbers[kt * 16 + (lane >> 2) + ((e >> 1) << 3)] : 1.f);
+            if (!ok) x = -INFINITY;
             st[kt][e] = x;
             mx[e & 1] = fmaxf(mx[e & 1], x);
         }
@@ -364,12 +401,17 @@ __device__ __forceinline__ void attend_chunk_t8(const uint32_t (&qb)[D / 16][2],
 // ---------------------------------------------------------------------------------------------- decode
 // T8: every tile has at most 8 rows and one token (a decode step of a model with up to 8 heads per group): the transposed form.
 // SIG: sigmoid weights; TURN: results are turned back (each compiled in only where it is asked for)
-template <int D, int BN, int STAGES, int DW, bool T8, bool SIG, bool TURN>
+// EXT: the extras of ExtTerms (T8 only); SHARED: keys are values, a chunk is one tile of the ring
+template <int D, int BN, int STAGES, int DW, bool T8, bool SIG, bool TURN, bool EXT = false, bool SHARED = false>
 __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p) {
     extern __shared__ __align__(128) unsigned char smem_raw[];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    static_assert((!EXT || (T8 && !SIG && !TURN)) && (!SHARED || EXT), "the extras are built for the transposed form");
     constexpr int TILE = BN * D;                       // elements of one K or V chunk
-    bf16* my = reinterpret_cast<bf16*>(smem_raw) + (size_t)warp * STAGES * 2 * TILE;
+    constexpr int SLOT = SHARED ? TILE : 2 * TILE;     // elements of a slot of the ring
+    constexpr int V_AT = SHARED ? 0 : TILE;            // where the values of a slot lie
+    bf16* my = reinterpret_cast<bf16*>(smem_raw) + (size_t)warp * STAGES * SLOT;
+    float* my_numbers = reinterpret_cast<float*>(smem_raw + (size_t)DW * STAGES * SLOT * sizeof(bf16)) + warp * STAGES * BN;   // SHARED: [STAGES][BN]
     __shared__ int flag;
 
     const int tile = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z;
@@ -388,7 +430,8 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
     const int pos0 = p.positions[n0];
     const int* table = p.block_table + (size_t)p.token_seq[n0] * p.max_blocks;
     const int hi = pos0 + ntok;  // one past the last visible key
-    const int lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+    int lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
+    if (EXT && p.chunk > 0) lo = max(lo, pos0 / p.chunk * p.chunk);
     const int chunks = (hi - lo + BN - 1) / BN;
     const int per = (chunks + p.num_splits - 1) / p.num_splits;
     const int c_begin = split * per, c_end = min(chunks, c_begin + per);
@@ -403,7 +446,7 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
     for (int s = 0; s < STAGES; ++s) {
         const int key0 = lo + (first + s * DW) * BN;
         fetched[s] = early && s < mine && key0 + BN <= pos0;  // wholly before the first new position
-        if (fetched[s]) load_rows_warp<D, BN>(p, table, kvh, key0, hi - 1, 0, my + s * 2 * TILE, my + s * 2 * TILE + TILE, lane);
+        if (fetched[s]) load_rows_warp<D, BN, SHARED>(p, table, kvh, key0, hi - 1, 0, my + s * SLOT, my + s * SLOT + V_AT, lane, my_numbers + s * BN);
     }
     if (early) pdl_wait();
 
@@ -523,19 +566,46 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
 
 #pragma unroll
     for (int s = 0; s < STAGES; ++s) {
-        if (s < mine && !fetched[s]) load_rows_warp<D, BN>(p, table, kvh, lo + (first + s * DW) * BN, hi - 1, 0, my + s * 2 * TILE, my + s * 2 * TILE + TILE, lane);
+        if (s < mine && !fetched[s])
+            load_rows_warp<D, BN, SHARED>(p, table, kvh, lo + (first + s * DW) * BN, hi - 1, 0, my + s * SLOT, my + s * SLOT + V_AT, lane, my_numbers + s * BN);
         cp_async_commit();  // stage 0's group may also hold later stages' early fetches: it then completes a little later, never too early
     }
     // where the chunk lies that refills the first slot: the block table is read now, not between a chunk's arithmetic and the
     // copies that refill its slot
     PoolRows<BN> refill;
     if (STAGES < mine) refill = find_rows_warp<BN>(p, table, kvh, lo + (first + STAGES * DW) * BN, hi - 1, lane);
+    ExtTerms<BN> ext;
+    float rel_last[2] = {0.f, 0.f};
+    if constexpr (EXT) {
+        ext.x_scale = p.x_scale;
+        ext.cap_log2 = p.cap_log2;
+        ext.numbers = nullptr;
+        if (p.rel) {
+#pragma unroll
+            for (int j = 0; j < 2; ++j) rel_last[j] = LOG2E * p.rel[(size_t)(p.rel_rows - 1) * p.nq + kvh * G + min(((lane & 3) << 1) + j, G - 1)];
+        }
+    }
     for (int it = 0; it < mine; ++it) {
+        if constexpr (EXT) {   // the chunk's biases, asked for before its keys are waited for
+            const int key0 = lo + (first + it * DW) * BN;
+            const bool near = p.rel && pos0 - (key0 + BN - 1) < p.n_rows_of;
+#pragma unroll
+            for (int kt = 0; kt < BN / 16; ++kt)
+#pragma unroll
+                for (int i = 0; i < 2; ++i) {
+                    const int dist = max(pos0 - (key0 + kt * 16 + (lane >> 2) + 8 * i), 0);
+                    const int row = (near && dist < p.n_rows_of) ? p.rows_of[dist] : -1;
+#pragma unroll
+                    for (int j = 0; j < 2; ++j)
+                        ext.b[kt][2 * i + j] = row < 0 ? rel_last[j] : LOG2E * p.rel[(size_t)row * p.nq + kvh * G + min(((lane & 3) << 1) + j, G - 1)];
+                }
+            if (SHARED) ext.numbers = my_numbers + (it % STAGES) * BN;
+        }
         // groups so far: STAGES from above and one per iteration before this one; chunk `it` is in group `it` (and the early
         // fetches in group 0): everything but the STAGES - 1 youngest groups must have landed
         cp_async_wait<STAGES - 1>();
         __syncwarp();
-        bf16* cur = my + (it % STAGES) * 2 * TILE;
+        bf16* cur = my + (it % STAGES) * SLOT;
         const int key0 = lo + (first + it * DW) * BN;
         if (it == own_it) {
             // The token's own position lies in this chunk, and the cache did not hold its key and value when the chunk was
@@ -557,7 +627,10 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
         // a chunk that lies wholly before the first token's position (and inside every window) needs no mask arithmetic;
         // rows beyond the tile then collect numbers nobody reads
         const bool interior = key0 + BN - 1 <= pos0 && (p.window <= 0 || key0 > hi - 1 - p.window);
-        if constexpr (T8) {
+        if constexpr (EXT) {
+            if (interior) attend_chunk_t8<D, BN, false, false, true>(qb, cur, cur + V_AT, o, m, l, key0, pos0, nrows, p.window, 1.f, lane, nullptr, &ext);
+            else attend_chunk_t8<D, BN, true, false, true>(qb, cur, cur + V_AT, o, m, l, key0, pos0, nrows, p.window, 1.f, lane, nullptr, &ext);
+        } else if constexpr (T8) {
             if (interior) attend_chunk_t8<D, BN, false, SIG>(qb, cur, cur + TILE, o, m, l, key0, pos0, nrows, p.window, p.scale_log2, lane, &sig);
             else attend_chunk_t8<D, BN, true, SIG>(qb, cur, cur + TILE, o, m, l, key0, pos0, nrows, p.window, p.scale_log2, lane, &sig);
         } else {
@@ -567,8 +640,8 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
         __syncwarp();  // every lane is done with the slot
         const int nxt = it + STAGES;
         if (nxt < mine) {
-            bf16* dst = my + (it % STAGES) * 2 * TILE;
-            copy_rows_warp<D, BN>(p, refill, 0, dst, dst + TILE, lane);
+            bf16* dst = my + (it % STAGES) * SLOT;
+            copy_rows_warp<D, BN, SHARED>(p, refill, 0, dst, dst + V_AT, lane, my_numbers + (it % STAGES) * BN);
             if (nxt + 1 < mine) refill = find_rows_warp<BN>(p, table, kvh, lo + (first + (nxt + 1) * DW) * BN, hi - 1, lane);
         }
         cp_async_commit();
@@ -657,6 +730,16 @@ __global__ void __launch_bounds__(DW * 32) attn_mma_decode_kernel(const Params p
             fo[r * D + D / 2 + k] = fmaf(-a, sn, b * c);
         }
         __syncthreads();
+    }
+    if constexpr (EXT) {
+        if (p.gate) {   // slice by slice (the merge is linear in the outputs)
+            for (int i = tid; i < nrows * D; i += DW * 32) {
+                const int r = i / D;
+                const float z = to_f32(p.gate[(size_t)n0 * p.gate_stride + kvh * G + r]);
+                fo[i] *= 1.0f / (1.0f + expf(-z));
+            }
+            __syncthreads();
+        }
     }
     if (p.cluster && p.num_splits > 1) {
         // The slices of this tile are the blocks of one cluster: block 0 reads every block's (max, sum, output) out of
@@ -823,15 +906,15 @@ __global__ void attn_plan_kernel(const int* __restrict__ starts, int num_seqs, i
     for (; t < max_tiles; ++t) { tile_info[2 * t] = 0; tile_info[2 * t + 1] = 0; }
 }
 
-template <int D, bool T8, int DW, bool SIG, bool TURN>
+template <int D, bool T8, int DW, bool SIG, bool TURN, bool EXT = false, bool SHARED = false>
 int launch_decode_as(const Params& p, dim3 grid, cudaStream_t s) {
-    constexpr int BN = D == 64 ? 32 : 16, STAGES = 3;  // DW warps, each with its own ring of 4 KB + 4 KB chunks
-    constexpr size_t ring = (size_t)DW * STAGES * 2 * BN * D * sizeof(bf16);
+    constexpr int BN = D == 64 ? 32 : 16, STAGES = SHARED ? 6 : 3;  // DW warps, each with its own ring of 4 KB + 4 KB chunks
+    constexpr size_t ring = (size_t)DW * STAGES * ((SHARED ? 1 : 2) * BN * D * sizeof(bf16) + (SHARED ? BN * sizeof(float) : 0));
     constexpr size_t merge = (size_t)(DW * 16 * (D + 8 + 3) + 16 * (D + 2)) * sizeof(float);
     constexpr size_t smem = ring > merge ? ring : merge;
     static bool set = false;
     if (!set) {
-        cudaError_t e = cudaFuncSetAttribute(attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG, TURN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG, TURN, EXT, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
         set = true;
     }
@@ -850,13 +933,17 @@ int launch_decode_as(const Params& p, dim3 grid, cudaStream_t s) {
         attr[1].val.programmaticStreamSerializationAllowed = 1;
         cfg.attrs = attr;
         cfg.numAttrs = llmie_pdl_flag ? 2 : 1;
-        return (int)cudaLaunchKernelEx(&cfg, attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG, TURN>, p);
+        return (int)cudaLaunchKernelEx(&cfg, attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG, TURN, EXT, SHARED>, p);
     }
-    return launch_kernel(attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG, TURN>, grid, dim3(DW * 32), smem, s, p);
+    return launch_kernel(attn_mma_decode_kernel<D, BN, STAGES, DW, T8, SIG, TURN, EXT, SHARED>, grid, dim3(DW * 32), smem, s, p);
 }
 
 template <int D, bool T8, int DW>
 int launch_decode(const Params& p, dim3 grid, cudaStream_t s) {
+    if (p.x_scale != 0.f) {   // (set for the extras only)
+        if constexpr (T8) return p.key_scale ? launch_decode_as<D, T8, DW, false, false, true, true>(p, grid, s) : launch_decode_as<D, T8, DW, false, false, true, false>(p, grid, s);
+        else return LLMIE_ERR_BAD_ARGUMENT;
+    }
     if (p.sig_bias) return p.turn_cos ? launch_decode_as<D, T8, DW, true, true>(p, grid, s) : launch_decode_as<D, T8, DW, true, false>(p, grid, s);
     return p.turn_cos ? launch_decode_as<D, T8, DW, false, true>(p, grid, s) : launch_decode_as<D, T8, DW, false, false>(p, grid, s);
 }
@@ -905,7 +992,7 @@ static int run_mma(const bf16* q, int q_stride, const bf16* k_pool, const bf16* 
                    bf16* out, float* scratch_o, float* scratch_ml, int* counters, int nq, int nkv, int d,
                    int page_size, float scale, int window, int num_splits, int decode_mode, int cluster, const float* qkv_acc,
                    int acc_stride, const float* bias, const float* cos_t, const float* sin_t, const int* slots, const float* turn_cos, const float* turn_sin,
-                   const float* sig_bias, const float* log_r1, const float* log_r2, cudaStream_t s) {
+                   const float* sig_bias, const float* log_r1, const float* log_r2, cudaStream_t s, const Params* extras = nullptr) {
     if (num_tiles <= 0) return 0;
     if ((turn_cos == nullptr) != (turn_sin == nullptr) || (log_r1 == nullptr) != (log_r2 == nullptr) || (log_r1 && !sig_bias) ||
         ((turn_cos || sig_bias) && !decode_mode))
@@ -927,6 +1014,11 @@ static int run_mma(const bf16* q, int q_stride, const bf16* k_pool, const bf16* 
     p.num_splits = num_splits; p.scale_log2 = scale * LOG2E; p.cluster = cluster;
     p.qkv_acc = qkv_acc; p.acc_stride = acc_stride; p.bias = bias; p.cos_t = cos_t; p.sin_t = sin_t; p.slots = slots;
     p.turn_cos = turn_cos; p.turn_sin = turn_sin; p.sig_bias = sig_bias; p.log_r1 = log_r1; p.log_r2 = log_r2;
+    if (extras) {
+        p.chunk = extras->chunk; p.cap_log2 = extras->cap_log2; p.x_scale = extras->x_scale; p.rel = extras->rel; p.rows_of = extras->rows_of;
+        p.n_rows_of = extras->n_rows_of; p.rel_rows = extras->rel_rows; p.gate = extras->gate; p.gate_stride = extras->gate_stride;
+        p.key_scale = extras->key_scale;
+    }
     p.k_pool_w = const_cast<bf16*>(k_pool); p.v_pool_w = const_cast<bf16*>(v_pool);
     return d == 64 ? launch<64>(p, num_tiles, decode_mode, s) : launch<128>(p, num_tiles, decode_mode, s);
 }
@@ -939,6 +1031,26 @@ LLMIE_API int llmie_paged_attention_mma(const bf16* q, int q_stride, const bf16*
     return run_mma(q, q_stride, k_pool, v_pool, block_table, max_blocks, token_seq, positions, tile_info, num_tiles, out, scratch_o, scratch_ml,
                    counters, nq, nkv, d, page_size, scale, window, num_splits, decode_mode, cluster, nullptr, 0, nullptr, nullptr, nullptr,
                    nullptr, turn_cos, turn_sin, sig_bias, log_r1, log_r2, s);
+}
+
+// Decode steps (tile i is token i, at most 8 query heads per key/value head) with chunks, a soft cap, a bias by distance (rel [rel_rows][nq],
+// rows_of [n_rows_of]: distance -> row), a gate per head (gate + n * gate_stride), and, with key_scale [pages][page_size] and no v_pool, values
+// that are the keys; each off when its pointer is null or its number 0. four_warps as decode_mode 2.
+LLMIE_API int llmie_paged_attention_mma_ext(const bf16* q, int q_stride, const bf16* k_pool, const bf16* v_pool, const int* block_table, int max_blocks,
+                                            const int* token_seq, const int* positions, int num_tokens, bf16* out, float* scratch_o, float* scratch_ml,
+                                            int* counters, int nq, int nkv, int d, int page_size, float scale, int window, int num_splits, int cluster,
+                                            int four_warps, int chunk, float softcap, const float* rel, const int* rows_of, int n_rows_of, int rel_rows,
+                                            const bf16* gate, int gate_stride, const float* key_scale, cudaStream_t s) {
+    if (num_tokens <= 0) return 0;
+    if (nkv <= 0 || nq / nkv > 8 || chunk < 0 || softcap < 0.f || scale == 0.f || (rel && (!rows_of || rel_rows < 1 || n_rows_of < 0)) ||
+        (v_pool == nullptr) != (key_scale != nullptr))
+        return LLMIE_ERR_BAD_ARGUMENT;
+    Params e;
+    e.chunk = chunk; e.cap_log2 = softcap * LOG2E; e.x_scale = softcap > 0.f ? 2.f * LOG2E * scale / softcap : LOG2E * scale;
+    e.rel = rel; e.rows_of = rows_of; e.n_rows_of = n_rows_of; e.rel_rows = rel_rows; e.gate = gate; e.gate_stride = gate_stride; e.key_scale = key_scale;
+    return run_mma(q, q_stride, k_pool, v_pool, block_table, max_blocks, token_seq, positions, nullptr, num_tokens, out, scratch_o, scratch_ml, counters,
+                   nq, nkv, d, page_size, scale, window, num_splits, four_warps ? 2 : 1, cluster, nullptr, 0, nullptr, nullptr, nullptr, nullptr, nullptr,
+                   nullptr, nullptr, nullptr, nullptr, s, &e);
 }
 
 // Decode steps (every tile one token, at most 8 query heads per key/value head): the same attention, with the queries, keys and

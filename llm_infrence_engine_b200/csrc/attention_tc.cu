@@ -96,7 +96,8 @@ struct TcParams {
     const float* rel;       // [rel_rows][nq] or null
     const int* rows_of;     // [n_rows_of]
     int n_rows_of, rel_rows;
-    int table;              // distances whose biases lie in shared memory
+    int table;              // distances whose biases lie in shared memory ...
+    int rows_s;             // ... and, for the ones beyond: 1 if rows_of (16-bit) and the group's columns of rel lie there too
     const bf16* gate;       // row n at gate + n * gate_stride: a number per head; or null
     int gate_stride;
     const float* key_scale; // SHARED: [pages][page_size]
@@ -238,6 +239,13 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
             const int g_all = p.nq / p.nkv, n = p.table * g_all;
 #pragma unroll 4
             for (int i = tid; i < n; i += THREADS) bias_s[i] = LOG2E * p.rel[(size_t)p.rows_of[i / g_all] * p.nq + kvh * g_all + i % g_all];
+            if (p.rows_s) {
+                float* val = bias_s + n;
+                unsigned short* row = reinterpret_cast<unsigned short*>(val + p.rel_rows * g_all);
+                for (int i = tid; i < p.rel_rows * g_all; i += THREADS) val[i] = LOG2E * p.rel[(size_t)(i / g_all) * p.nq + kvh * g_all + i % g_all];
+#pragma unroll 4
+                for (int i = tid; i < p.n_rows_of; i += THREADS) row[i] = (unsigned short)p.rows_of[i];
+            }
         }
         __syncthreads();
     }
@@ -502,6 +510,15 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                     const float* tb = bias_s + (pos0 - key0) * G + (row_ok ? row : 0);
 #pragma unroll
                     for (int j = 0; j < BN; ++j) s[j] = __float_as_uint(__uint_as_float(s[j]) + tb[-j * G]);
+                } else if (p.rel && !all_far && p.rows_s) {
+                    const float* val = bias_s + p.table * G + (row_ok ? row % G : 0);
+                    const unsigned short* row_of = reinterpret_cast<const unsigned short*>(bias_s + (p.table + p.rel_rows) * G);
+#pragma unroll
+                    for (int j = 0; j < BN; ++j) {
+                        const int dist = max(pos - key0 - j, 0);
+                        const int br = dist < p.n_rows_of ? row_of[dist] : p.rel_rows - 1;
+                        s[j] = __float_as_uint(__uint_as_float(s[j]) + val[br * G]);
+                    }
                 } else if (p.rel && !all_far) {
 #pragma unroll
                     for (int j = 0; j < BN; ++j) {
@@ -905,7 +922,7 @@ LLMIE_API int llmie_paged_attention_tc(const bf16* q, int q_stride, const bf16* 
     p.window = window; p.box_rows = page_size < BN ? page_size : BN; p.scale_log2 = scale * LOG2E;
     p.turn_cos = turn_cos; p.turn_sin = turn_sin; p.sig_bias = sig_bias; p.log_r1 = log_r1; p.log_r2 = log_r2;
     p.chunk = chunk; p.cap = softcap; p.x_scale = softcap > 0.f ? 2.f * LOG2E * scale / softcap : LOG2E * scale;
-    p.rel = rel; p.rows_of = rows_of; p.n_rows_of = n_rows_of; p.rel_rows = rel_rows; p.table = 0;
+    p.rel = rel; p.rows_of = rows_of; p.n_rows_of = n_rows_of; p.rel_rows = rel_rows; p.table = 0; p.rows_s = 0;
     p.gate = gate; p.gate_stride = gate_stride; p.key_scale = key_scale;
     CUtensorMap mk, mv;
     const int rows = (int)(pool_pages * nkv * page_size);
@@ -930,7 +947,14 @@ LLMIE_API int llmie_paged_attention_tc(const bf16* q, int q_stride, const bf16* 
         const int stages = key_scale ? (d == 64 ? SHARED_STAGES<64> : SHARED_STAGES<128>) : 2 * (d == 64 ? Sizes<64>::STAGES : Sizes<128>::STAGES);
         size_t smem = (size_t)BM * d * 2 + (size_t)stages * k_bytes + 1024 + BARRIER_BYTES + (key_scale ? (size_t)stages * BN * 4 : 0);
         if (rel) {
-            const long long room = ((long long)113 * 1024 - (long long)smem) / (4 * G);
+            long long room = (long long)113 * 1024 - (long long)smem;
+            const long long two_level = (long long)rel_rows * G * 4 + ((long long)n_rows_of * 2 + 3) / 4 * 4;
+            if (room / (4 * G) < n_rows_of && two_level <= room && rel_rows <= 65535) {   // not all of them: the rest through the rows' numbers
+                p.rows_s = 1;
+                room -= two_level;
+                smem += (size_t)two_level;
+            }
+            room /= 4 * G;
             p.table = (int)(room < n_rows_of ? (room > 0 ? room : 0) : n_rows_of);
             smem += (size_t)p.table * G * 4;
         }

@@ -129,7 +129,7 @@ class CudaKernels:
                    "llmie_embed_add", "llmie_mlstm_prepare", "llmie_mlstm_scan", "llmie_mlstm_finish", "llmie_paged_attention_talk",
                    "llmie_attention_talk_slice", "llmie_attention_talk_mma_fits", "llmie_paged_attention_talk_mma", "llmie_embed_bigram",
                    "llmie_dynamic_tanh", "llmie_embed_positions", "llmie_post_rms", "llmie_qk_rows_norm_store", "llmie_linear_attention_scan",
-                   "llmie_linear_attention_mma", "llmie_linear_attention_mma_fits"):
+                   "llmie_linear_attention_mma", "llmie_linear_attention_mma_fits", "llmie_paged_attention_mma_ext"):
             getattr(self.lib, fn).restype = ctypes.c_int
         # two forms of the gate/up kernel live in source files of their own, and the library also builds without them
         self._gate_up_cluster = self._gate_up_pair = self._gate_up_glu_pair = self._up_gelu_pair = None
@@ -1160,10 +1160,22 @@ class CudaKernels:
                                        int(window), min(max_context, window) if window else max_context, batch, num_splits, turn, sigmoid_bias, log_distance)
             if done is not None:
                 return done
-        if (self.use_tc_attention_ext and dt == 1 and batch is not None and batch.max_seq_len > 1 and head_dim == v_head_dim and q_col == 0 and q.shape[1] % 8 == 0
+        if (self.use_tc_attention_ext and dt == 1 and batch is not None and head_dim == v_head_dim and q_col == 0 and q.shape[1] % 8 == 0
                 and not (keep_first or temp[1]) and sink is None and gate_mode != 2 and log_distance is None and sigmoid_bias is None and turn is None
                 and (v_pool is None) == (key_scale is not None)):
             span = min(max_context, window or max_context, chunk or max_context)
+            group = num_heads // num_kv_heads
+            if batch.max_seq_len == 1 and group <= 8 and head_dim in (64, 128) and scale != 0 and self.use_mma_attention:
+                # single tokens: the decode kernel of plain attention
+                n_splits, cluster, scratch_o, scratch_ml, counters = self._decode_plan(N, num_kv_heads, head_dim, span, num_splits, q.device)
+                self._check(self.lib.llmie_paged_attention_mma_ext(
+                    _ptr(q), q.shape[1], _ptr(k_pool), _ptr(v_pool), _ptr(block_table), block_table.shape[1], _ptr(token_seq), _ptr(positions), N, _ptr(out),
+                    _ptr(scratch_o), _ptr(scratch_ml), _ptr(counters), num_heads, num_kv_heads, head_dim, page_size, ctypes.c_float(scale), int(window),
+                    n_splits, cluster, int(self._decode_four_warps), int(chunk), ctypes.c_float(softcap), _ptr(rel), _ptr(rel_rows),
+                    0 if rel_rows is None else rel_rows.shape[0], 0 if rel is None else rel.shape[0],
+                    ctypes.c_void_p(0 if gate is None else gate.data_ptr() + gate_col * esize), 0 if gate is None else gate.shape[1], _ptr(key_scale),
+                    self._stream()), "attention_ext (decode, tensor cores)")
+                return out
             done = self._attention_tc(q, k_pool, v_pool, block_table, token_seq, positions, out, num_heads, num_kv_heads, head_dim, page_size, scale,
                                       int(window), span, batch, num_splits, chunk=chunk, softcap=softcap, rel=rel, rel_rows=rel_rows, gate=gate, gate_col=gate_col,
                                       key_scale=key_scale)
