@@ -193,10 +193,12 @@ __device__ __forceinline__ void copy_rows_warp(const Params& p, const PoolRows<N
         if (!SHARED) cp_async16(vs + dst, p.v_pool + src);
     }
     if constexpr (SHARED) {
-        static_assert(NKEYS <= 32, "one number per lane");
-        const int r = rows.idx[0];                       // (page * nkv + kvh) * page_size + offset
-        const int page = r / (p.nkv * p.page_size);
-        if (lane < NKEYS) cp_async4(numbers + tile_row0 + lane, p.key_scale + (size_t)page * p.page_size + r % p.page_size);
+#pragma unroll
+        for (int h = 0; h < (NKEYS + 31) / 32; ++h) {
+            const int r = rows.idx[h];                   // (page * nkv + kvh) * page_size + offset
+            const int t = p.page_shift >= 0 ? r >> p.page_shift : r / p.page_size;
+            if (lane + 32 * h < NKEYS) cp_async4(numbers + tile_row0 + lane + 32 * h, p.key_scale + (size_t)(t / p.nkv) * p.page_size + (r - t * p.page_size));
+        }
     }
 }
 
@@ -908,7 +910,8 @@ __global__ void attn_plan_kernel(const int* __restrict__ starts, int num_seqs, i
 
 template <int D, bool T8, int DW, bool SIG, bool TURN, bool EXT = false, bool SHARED = false>
 int launch_decode_as(const Params& p, dim3 grid, cudaStream_t s) {
-    constexpr int BN = D == 64 ? 32 : 16, STAGES = SHARED ? 6 : 3;  // DW warps, each with its own ring of 4 KB + 4 KB chunks
+    // DW warps, each with its own ring of three slots of 8 KB: keys and values of BN of them, or twice as many keys that are values
+    constexpr int BN = (D == 64 ? 32 : 16) * (SHARED ? 2 : 1), STAGES = 3;
     constexpr size_t ring = (size_t)DW * STAGES * ((SHARED ? 1 : 2) * BN * D * sizeof(bf16) + (SHARED ? BN * sizeof(float) : 0));
     constexpr size_t merge = (size_t)(DW * 16 * (D + 8 + 3) + 16 * (D + 2)) * sizeof(float);
     constexpr size_t smem = ring > merge ? ring : merge;

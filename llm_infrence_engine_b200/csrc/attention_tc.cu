@@ -947,7 +947,7 @@ LLMIE_API int llmie_paged_attention_tc(const bf16* q, int q_stride, const bf16* 
         const int stages = key_scale ? (d == 64 ? SHARED_STAGES<64> : SHARED_STAGES<128>) : 2 * (d == 64 ? Sizes<64>::STAGES : Sizes<128>::STAGES);
         size_t smem = (size_t)BM * d * 2 + (size_t)stages * k_bytes + 1024 + BARRIER_BYTES + (key_scale ? (size_t)stages * BN * 4 : 0);
         if (rel) {
-            long long room = (long long)113 * 1024 - (long long)smem;
+            long long room = (long long)113 * 1024 - 512 - (long long)smem;   // (the kernel has a few static bytes too)
             const long long two_level = (long long)rel_rows * G * 4 + ((long long)n_rows_of * 2 + 3) / 4 * 4;
             if (room / (4 * G) < n_rows_of && two_level <= room && rel_rows <= 65535) {   // not all of them: the rest through the rows' numbers
                 p.rows_s = 1;

@@ -80,6 +80,7 @@ class CudaKernels:
         # linear attention with fixed decays, bfloat16: steps whose longest request brings this many rows take the tensor-core form, on
         # projections that are activated by the product that makes them; below, the scan activates them as it reads them
         self.linear_attention_mma_rows = 24
+        self.use_linear_attention_step = True   # ... and decoded tokens alone in bfloat16 a kernel that streams the states (float32: always the scan)
         self.use_mma_attention_talk = True   # heads that talk, steps with prompt portions in bfloat16: plain scores and P V on the tensor cores
         self.head_matmul_library_rows = 64   # per-head products of latent attention: from this many rows on, one batched library product
         self.slice_keys = 1024         # generic attention: keys per slice, at fixed places of a request (a multiple of 32)
@@ -129,7 +130,7 @@ class CudaKernels:
                    "llmie_embed_add", "llmie_mlstm_prepare", "llmie_mlstm_scan", "llmie_mlstm_finish", "llmie_paged_attention_talk",
                    "llmie_attention_talk_slice", "llmie_attention_talk_mma_fits", "llmie_paged_attention_talk_mma", "llmie_embed_bigram",
                    "llmie_dynamic_tanh", "llmie_embed_positions", "llmie_post_rms", "llmie_qk_rows_norm_store", "llmie_linear_attention_scan",
-                   "llmie_linear_attention_mma", "llmie_linear_attention_mma_fits", "llmie_paged_attention_mma_ext"):
+                   "llmie_linear_attention_mma", "llmie_linear_attention_mma_fits", "llmie_linear_attention_step", "llmie_paged_attention_mma_ext"):
             getattr(self.lib, fn).restype = ctypes.c_int
         # two forms of the gate/up kernel live in source files of their own, and the library also builds without them
         self._gate_up_cluster = self._gate_up_pair = self._gate_up_glu_pair = self._up_gelu_pair = None
@@ -1821,6 +1822,11 @@ class CudaKernels:
             self._check(self.lib.llmie_linear_attention_mma(_ptr(z), z.shape[1], int(q_col), int(k_col), int(v_col), _ptr(decay), _ptr(state),
                                                             _ptr(batch.seq_starts_dev), _ptr(batch.seq_slots), _ptr(out), H, D, DV, batch.num_seqs,
                                                             self._stream()), "linear_attention (tensor cores)")
+            return out
+        if batch.max_seq_len == 1 and z.dtype == torch.bfloat16 and D % 4 == 0 and self.use_linear_attention_step:
+            self._check(self.lib.llmie_linear_attention_step(_ptr(z), z.shape[1], int(q_col), int(k_col), int(v_col), _ptr(decay), _ptr(state),
+                                                             _ptr(batch.seq_starts_dev), _ptr(batch.seq_slots), _ptr(out), H, D, DV, batch.num_seqs,
+                                                             self._stream()), "linear_attention (decoded tokens)")
             return out
         self._check(self.lib.llmie_linear_attention_scan(_ptr(z), z.shape[1], int(q_col), int(k_col), int(v_col), _ptr(decay), _ptr(state),
                                                          _ptr(batch.seq_starts_dev), _ptr(batch.seq_slots), _ptr(out), H, D, DV, batch.num_seqs,

@@ -239,7 +239,8 @@ def test_linear_attention(K, dtype, H, D, DV):
     forms = [False] + ([True] if dtype == "bfloat16" and K.lib.llmie_linear_attention_mma_fits(D, DV) else [])
     for lens, slots in (([1, 1, 1], [2, 0, 3]), ([70, 1, 64, 3], [1, 3, 0, 2]), ([130], [2]), ([63, 65, 129, 2], [3, 2, 1, 0])):
         host, dev = ragged(lens, slots)
-        for activated in forms:
+        for activated, step_kernel in [(f, True) for f in forms] + ([(False, False)] if dtype == "bfloat16" and max(lens) == 1 else []):
+            K.use_linear_attention_step = step_kernel
             state = rnd(5, H, DV, D, seed=1, scale=0.5)
             sd = state.cuda()
             for step in range(2):
@@ -251,6 +252,7 @@ def test_linear_attention(K, dtype, H, D, DV):
                 close(got, want, "float32", f"{lens} step {step} activated {activated}", scale=size, f32=3e-5 if activated else 4e-6)
                 close(sd, state, "float32", f"states after {lens} step {step}", scale=float(state.abs().max()), f32=3e-5 if activated else 4e-6)
             assert torch.equal(sd[4].cpu(), state[4])
+            K.use_linear_attention_step = True
 
 
 def test_linear_attention_remembers_the_first_token(K):
