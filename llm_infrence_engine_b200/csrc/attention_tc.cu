@@ -117,6 +117,12 @@ __device__ __forceinline__ float fast_exp2(float x) {
     return y;
 }
 
+__device__ __forceinline__ float fast_rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
+
 // Three-input maximum and the packed 32-bit forms of sm_100a (two independent float32 operations per instruction): the
 // softmax step is bound by issue slots, and these halve the slots of its maxima, scalings and sums.
 __device__ __forceinline__ float max3(float a, float b, float c) {
@@ -468,7 +474,7 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                 const float add = (p.cap > 0.f ? p.cap * LOG2E : 0.f) + (all_far ? rel_last : 0.f);
                 const uint64_t zero2 = pair_of(0.f, 0.f), x2 = pair_of(p.x_scale, p.x_scale), add2_ = pair_of(add, add);
                 if (p.cap > 0.f) {
-                    // cap tanh(v) = cap - 2 cap / (e^(2 v) + 1), two of them per division; e^(2 v) is bounded so that the product stays finite
+                    // cap tanh(v) = cap - 2 cap / (e^(2 v) + 1); an e^(2 v) beyond the largest number has the reciprocal zero, as it should
                     const float m2cap = -2.f * LOG2E * p.cap;
                     const uint64_t one2 = pair_of(1.f, 1.f), m2cap2 = pair_of(m2cap, m2cap);
 #pragma unroll
@@ -481,9 +487,8 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                             uint64_t v = pair_of(__uint_as_float(s[j + i]), __uint_as_float(s[j + i + 1]));
                             if (SHARED) v = fma2(v, pair_of(kk[i], kk[i + 1]), zero2);
                             unpair(fma2(v, x2, zero2), a, b);
-                            unpair(add2(pair_of(fast_exp2(fminf(a, 60.f)), fast_exp2(fminf(b, 60.f))), one2), t0, t1);
-                            const float r = __fdividef(1.0f, t0 * t1);
-                            unpair(fma2(pair_of(r * t1, r * t0), m2cap2, add2_), a, b);
+                            unpair(add2(pair_of(fast_exp2(a), fast_exp2(b)), one2), t0, t1);
+                            unpair(fma2(pair_of(fast_rcp(t0), fast_rcp(t1)), m2cap2, add2_), a, b);
                             s[j + i] = __float_as_uint(a);
                             s[j + i + 1] = __float_as_uint(b);
                         }
@@ -509,7 +514,12 @@ __global__ void __launch_bounds__(THREADS, 2) attn_tc_prefill_kernel(const __gri
                     // (A key behind the row's position reads what lies before the table in shared memory: the ring; see above.)
                     const float* tb = bias_s + (pos0 - key0) * G + (row_ok ? row : 0);
 #pragma unroll
-                    for (int j = 0; j < BN; ++j) s[j] = __float_as_uint(__uint_as_float(s[j]) + tb[-j * G]);
+                    for (int j = 0; j < BN; j += 2) {
+                        float a, b;
+                        unpair(add2(pair_of(__uint_as_float(s[j]), __uint_as_float(s[j + 1])), pair_of(tb[-j * G], tb[-(j + 1) * G])), a, b);
+                        s[j] = __float_as_uint(a);
+                        s[j + 1] = __float_as_uint(b);
+                    }
                 } else if (p.rel && !all_far && p.rows_s) {
                     const float* val = bias_s + p.table * G + (row_ok ? row % G : 0);
                     const unsigned short* row_of = reinterpret_cast<const unsigned short*>(bias_s + (p.table + p.rel_rows) * G);

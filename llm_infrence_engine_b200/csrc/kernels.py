@@ -55,6 +55,7 @@ class CudaKernels:
         self.sample_single_block = False   # sampling by one block per row instead of a cluster per row (the slower, older kernel)
         self.use_tc_attention = True   # prompt portions of head size 64 or 128: scores and outputs through tcgen05 and tensor memory
         self.cluster_merge = True      # decode attention: the key slices of a token form a cluster and merge in shared memory
+        self.tc_ext_pieces = 5             # (pieces in quarters of what fits at once)
         self.use_tc_attention_ext = True   # ... also with chunks, a soft cap, a bias by distance, a gate per head, keys that are values
         self.use_tc_gemm = True
         self.use_cluster_gate_up = False  # ... by pairs of blocks that share their weight rows (TMA multicast within a cluster of two)
@@ -693,6 +694,10 @@ class CudaKernels:
         # long tiles into slices, as many pieces as fit on the device at once, and starts long pieces first.
         fixed = int(num_splits or 0)
         capacity = max(1, 2 * self.num_sms // num_kv_heads)   # two blocks per SM
+        if chunk or softcap or rel is not None or key_scale is not None:
+            # a chunk with these extras takes half as long again, so a slice weighs less against it: more, shorter pieces than fit at
+            # once (the long ones start first, the short ones fill the gaps)
+            capacity = capacity * self.tc_ext_pieces // 4
         # (tiles of up to 16 chunks are never cut: a slice costs about 8 chunks' time and is at least 8 chunks long)
         max_items = tiles * fixed if fixed else max(tiles, min(capacity, 16 * tiles)) if span > 16 * 64 else tiles
         key = ("tcgen05 attention plan", group, num_kv_heads, page_size, int(window), int(chunk), fixed)
